@@ -32,7 +32,7 @@ def model_numbers(engine: Engine) -> Dict[str, object]:
             if isinstance(leaf, PagedKV):
                 mixer = m.blocks[entry.layer].parts.get("mixer")
                 # how many keys the query at a position sees: the mixer's own rule (a window, a chunk) where it has one
-                seen = getattr(mixer, "keys_seen", None)
+                seen = getattr(mixer, "keys_seen" if leaf.pool == 1 else "blocks_seen", None)
                 window = getattr(mixer, "window", leaf.window)
                 paged.append((leaf.num_kv_heads * (leaf.head_dim + leaf.value_dim) * elt,
                               seen if seen is not None else (lambda pos, w=window: pos + 1 if w is None else min(pos + 1, w))))
@@ -40,7 +40,7 @@ def model_numbers(engine: Engine) -> Dict[str, object]:
             continue               # reads what another entry keeps: counted above as read, not below as kept
         for leaf in cache_leaves(req):
             if isinstance(leaf, PagedKV):
-                kv_per_token += leaf.num_kv_heads * (leaf.head_dim + leaf.value_dim) * elt
+                kv_per_token += leaf.num_kv_heads * (leaf.head_dim + leaf.value_dim) * elt / leaf.pool
             elif isinstance(leaf, SlotState):
                 n = 1
                 for d in leaf.shape:

@@ -5,7 +5,10 @@ it keeps: keys and values in pages (``PagedKV``), a fixed-size state per request
 (``SlotState``), or nothing.  Paged entries with the same retention rule (all
 keys, or a window of W) form one *page group*: they share block tables, so one
 page id means the same token range in each of their pools, and every group has
-pages of its own.  Each paged entry owns two pools
+pages of its own.  Entries that keep one row per block of P tokens
+(``PagedKV.pool``) form groups of their own too: a page holds as many rows, which
+stand for P times as many tokens, and that is the page size the manager counts in.
+Each paged entry owns two pools
 ``[num_pages, kv_heads, page_size, head_dim]`` (a KV head's tokens of one page
 are contiguous, so the attention kernels stream whole pages per head); the
 reference lays a page out as ``[page, kv_heads, head_dim]`` per token
@@ -28,19 +31,20 @@ from .manager import PageGroup
 def group_name(request: PagedKV) -> str:
     """Paged entries with the same retention rule share block tables (a page id means the same token range
     in each of their pools); the rule is all a group is known by."""
-    return "kv_all" if request.window is None else f"kv_window_{request.window}"
+    name = "kv_all" if request.window is None else f"kv_window_{request.window}"
+    return name if request.pool == 1 else f"{name}_pool_{request.pool}"
 
 
 def group_page_bytes(requests: List[Optional[object]], cache_of: List[Optional[int]], page_size: int,
                      element_size: int) -> Dict[str, int]:
     """Bytes that one page id of each group stands for: the K and V pages of every schedule entry of the group
-    that keeps a cache of its own."""
+    that keeps a cache of its own (of a group with a row per P tokens, the P-th part: it has so many fewer pages)."""
     out: Dict[str, int] = {}
     for top, src in zip(requests, cache_of):
         for req in cache_leaves(top):
             if isinstance(req, PagedKV) and src is None:
                 name = group_name(req)
-                out[name] = out.get(name, 0) + req.num_kv_heads * page_size * (req.head_dim + req.value_dim) * element_size
+                out[name] = out.get(name, 0) + -(-req.num_kv_heads * page_size * (req.head_dim + req.value_dim) * element_size // req.pool)
     return out
 
 
@@ -55,9 +59,9 @@ def plan_groups(requests: List[Optional[object]], page_size: int, num_pages: int
                 max_slots: Optional[int] = None, step_tokens: Optional[int] = None) -> List[PageGroup]:
     """One page group per distinct retention rule among the paged requests.  ``num_pages`` is the pool of a
     group that keeps every key; a group with a window gets no more pages than it can ever use
-    (``window_group_pages``) when ``max_slots`` and ``step_tokens`` are known."""
+    (``window_group_pages``) when ``max_slots`` and ``step_tokens`` are known; a group with a row per P tokens gets the
+    P-th part, and a page more per request."""
     groups: Dict[str, PageGroup] = {}
-    width = -(-max_context // page_size)
     for r in (leaf for top in requests for leaf in cache_leaves(top)):
         if isinstance(r, PagedKV):
             name = group_name(r)
@@ -65,7 +69,10 @@ def plan_groups(requests: List[Optional[object]], page_size: int, num_pages: int
                 pages = num_pages
                 if r.window is not None and max_slots is not None and step_tokens is not None:
                     pages = min(pages, window_group_pages(r.window, page_size, max_slots, min(step_tokens, max_context)))
-                groups[name] = PageGroup(name, page_size, pages, r.window, width)
+                if r.pool > 1 and max_slots is not None:
+                    pages = min(pages, -(-pages // r.pool) + max_slots)
+                covered = page_size * r.pool          # tokens that a page stands for
+                groups[name] = PageGroup(name, covered, pages, r.window, -(-max_context // covered))
     return list(groups.values())
 
 
@@ -106,8 +113,9 @@ class CacheStorage:
             return {name: self._allocate(i, sub) for name, sub in req.items()}
         if isinstance(req, PagedKV):
             g = self._by_name[group_name(req)]
-            k = torch.empty((g.num_pages, req.num_kv_heads, g.page_size, req.head_dim), dtype=self._dtype, device=self._device)
-            v = torch.empty((g.num_pages, req.num_kv_heads, g.page_size, req.value_dim), dtype=self._dtype, device=self._device)
+            rows = g.page_size // req.pool
+            k = torch.empty((g.num_pages, req.num_kv_heads, rows, req.head_dim), dtype=self._dtype, device=self._device)
+            v = torch.empty((g.num_pages, req.num_kv_heads, rows, req.value_dim), dtype=self._dtype, device=self._device)
             self.bytes += k.numel() * k.element_size() + v.numel() * v.element_size()
             return PagedKVCache(k, v, g.name)
         if isinstance(req, SlotState):

@@ -13,7 +13,11 @@
 //   S <- cap * tanh(S / cap)                                            (cap > 0 only)
 //   O = softmax(S) V, or with a sink: exp(S_j) / (exp(z_h) + sum_i exp(S_i)) V  (a key of score z_h and no value;
 //   z_h = sink_logits[h], or 0 without that array)
-//   O <- O * sigmoid(gate[t, h, :])                                     (gate given only)
+//   O <- O * sigmoid(gate[t, h, :]), or * sigmoid(gate[t, h])           (gate given only)
+//   S <- S + rel[h][min(pos - j, rel_len - 1)]                          (a bias per distance, given only)
+// Pooled blocks (pool P > 0, with a window): beside the keys of the window a position sees one key and value for every
+// block of P positions that lies wholly before it, blocks b < floor((pos - window + 1) / P); they come from pools of
+// their own (entry b of the request's block table over entries) and share the softmax with the window's keys.
 // Values may have a head size of their own (hsv).
 // Mask by absolute position: yalis/attention/backend_impl/sdpa_and_flex.py:15-19, 301-307.
 // KV head of query head h: h / (nh / g)                                 (:59-67).
@@ -25,74 +29,88 @@ constexpr int kWarps = 4;
 constexpr int kMaxPerLane = 8;  // head size <= 256
 
 template <typename T>
-__global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_stride, T* __restrict__ out,
-                                               int out_stride, const T* __restrict__ k_pool,
-                                               const T* __restrict__ v_pool, const int32_t* __restrict__ positions,
-                                               const int32_t* __restrict__ req_of_token,
-                                               const int32_t* __restrict__ block_table, int table_width,
-                                               int page_size, int num_pages, int nh, int g, int hs, int hsv,
-                                               float scale, int window, float softcap, int sink,
-                                               float out_scale, int chunk, const float* __restrict__ sink_logits,
-                                               const float* __restrict__ slopes, const T* __restrict__ gate,
-                                               int gate_stride) {
+struct GenericParams {
+  const T* q; int q_stride;
+  T* out; int out_stride;
+  const T* k_pool; const T* v_pool;
+  const int32_t* positions; const int32_t* req_of_token; const int32_t* block_table;
+  int table_width, page_size, num_pages, nh, g, hs, hsv;
+  float scale; int window; float softcap; int sink; float out_scale; int chunk;
+  const float* sink_logits; const float* slopes;
+  const float* rel; int rel_len;                 // [nh, rel_len] or null
+  const T* gate; int gate_stride, gate_per_head; // [N, nh * hsv], or [N, nh] per head
+  int pool;                                      // P > 0: pooled blocks before the window
+  const T* pk_pool; const T* pv_pool; const int32_t* pool_table;
+  int pool_table_width, pool_page_size, pool_num_pages;   // in entries (one per block)
+};
+
+template <typename T>
+__global__ void paged_attention_generic_kernel(const GenericParams<T> p) {
   extern __shared__ float smem[];  // [kWarps][hsv] accumulators, then m[kWarps], l[kWarps]
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
-  const int req = req_of_token[t];
+  const int req = p.req_of_token[t];
   if (req < 0) return;
-  const int pos = positions[t];
-  const int kvh = h / (nh / g);
+  const int pos = p.positions[t];
+  const int kvh = h / (p.nh / p.g);
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-  const int per_lane = (hs + 31) >> 5, per_lane_v = (hsv + 31) >> 5;
+  const int per_lane = (p.hs + 31) >> 5, per_lane_v = (p.hsv + 31) >> 5;
 
   float qr[kMaxPerLane], acc[kMaxPerLane];
-  const T* qp = q + (size_t)t * q_stride + (size_t)h * hs;
+  const T* qp = p.q + (size_t)t * p.q_stride + (size_t)h * p.hs;
 #pragma unroll
   for (int i = 0; i < kMaxPerLane; ++i) {
     const int d = lane + 32 * i;
-    qr[i] = (i < per_lane && d < hs) ? to_f32<T>(qp[d]) : 0.f;
+    qr[i] = (i < per_lane && d < p.hs) ? to_f32<T>(qp[d]) : 0.f;
     acc[i] = 0.f;
   }
   float m = -INFINITY, l = 0.f;
-  int lo = (window > 0 && pos - window + 1 > 0) ? pos - window + 1 : 0;
-  if (chunk > 0) lo = max(lo, (pos / chunk) * chunk);
-  const float slope = slopes ? slopes[h] : 0.f;
-  const int32_t* bt = block_table + (size_t)req * table_width;
-  for (int j = lo + warp; j <= pos; j += kWarps) {
-    const int pi = j / page_size;
-    const int page = pi < table_width ? bt[pi] : -1;
-    if (page < 0 || page >= num_pages) continue;  // unmapped: treated as masked
-    const size_t row = ((size_t)page * g + kvh) * page_size + (j - pi * page_size);
-    const T* kp = k_pool + row * hs;
-    const T* vp = v_pool + row * hsv;
+  int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
+  if (p.chunk > 0) lo = max(lo, (pos / p.chunk) * p.chunk);
+  const float slope = p.slopes ? p.slopes[h] : 0.f;
+  const int32_t* bt = p.block_table + (size_t)req * p.table_width;
+  // the pooled blocks first, then the window's keys: one row of places, of which each warp walks every fourth
+  const int blocks = (p.pool > 0 && p.window > 0 && pos - p.window + 1 > 0) ? (pos - p.window + 1) / p.pool : 0;
+  for (int at = warp; at < blocks + pos - lo + 1; at += kWarps) {
+    const bool pooled = at < blocks;
+    const int j = pooled ? at : lo + (at - blocks);
+    const int ps = pooled ? p.pool_page_size : p.page_size;
+    const int pi = j / ps;
+    const int32_t* table = pooled ? p.pool_table + (size_t)req * p.pool_table_width : bt;
+    const int page = pi < (pooled ? p.pool_table_width : p.table_width) ? table[pi] : -1;
+    if (page < 0 || page >= (pooled ? p.pool_num_pages : p.num_pages)) continue;  // unmapped: treated as masked
+    const size_t row = ((size_t)page * p.g + kvh) * ps + (j - pi * ps);
+    const T* kp = (pooled ? p.pk_pool : p.k_pool) + row * p.hs;
+    const T* vp = (pooled ? p.pv_pool : p.v_pool) + row * p.hsv;
     float dot = 0.f;
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
       const int d = lane + 32 * i;
-      if (i < per_lane && d < hs) dot += qr[i] * to_f32<T>(kp[d]);
+      if (i < per_lane && d < p.hs) dot += qr[i] * to_f32<T>(kp[d]);
     }
-    float s = warp_sum(dot) * scale;
-    if (slopes) s -= slope * (float)(pos - j);
-    if (softcap > 0.f) s = softcap * tanhf(s / softcap);
+    float s = warp_sum(dot) * p.scale;
+    if (p.slopes && !pooled) s -= slope * (float)(pos - j);
+    if (p.rel && !pooled) s += p.rel[(size_t)h * p.rel_len + min(pos - j, p.rel_len - 1)];
+    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
     const float m_new = fmaxf(m, s);
     const float corr = expf(m - m_new);
-    const float p = expf(s - m_new);
-    l = l * corr + p;
+    const float e = expf(s - m_new);
+    l = l * corr + e;
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
       const int d = lane + 32 * i;
-      if (i < per_lane_v && d < hsv) acc[i] = acc[i] * corr + p * to_f32<T>(vp[d]);
+      if (i < per_lane_v && d < p.hsv) acc[i] = acc[i] * corr + e * to_f32<T>(vp[d]);
     }
     m = m_new;
   }
   float* acc_s = smem;
-  float* m_s = smem + kWarps * hsv;
+  float* m_s = smem + kWarps * p.hsv;
   float* l_s = m_s + kWarps;
 #pragma unroll
   for (int i = 0; i < kMaxPerLane; ++i) {
     const int d = lane + 32 * i;
-    if (i < per_lane_v && d < hsv) acc_s[warp * hsv + d] = acc[i];
+    if (i < per_lane_v && d < p.hsv) acc_s[warp * p.hsv + d] = acc[i];
   }
   if (lane == 0) {
     m_s[warp] = m;
@@ -102,28 +120,32 @@ __global__ void paged_attention_generic_kernel(const T* __restrict__ q, int q_st
   float mm = -INFINITY;
 #pragma unroll
   for (int w = 0; w < kWarps; ++w) mm = fmaxf(mm, m_s[w]);
-  const float sink_z = (sink && sink_logits) ? sink_logits[h] : 0.f;
-  if (sink) mm = fmaxf(mm, sink_z);
-  float ll = sink ? expf(sink_z - mm) : 0.f;
+  const float sink_z = (p.sink && p.sink_logits) ? p.sink_logits[h] : 0.f;
+  if (p.sink) mm = fmaxf(mm, sink_z);
+  float ll = p.sink ? expf(sink_z - mm) : 0.f;
   float wgt[kWarps];
 #pragma unroll
   for (int w = 0; w < kWarps; ++w) {
     wgt[w] = (m_s[w] == -INFINITY) ? 0.f : expf(m_s[w] - mm);
     ll += l_s[w] * wgt[w];
   }
-  T* op = out + (size_t)t * out_stride + (size_t)h * hsv;
-  for (int d = threadIdx.x; d < hsv; d += blockDim.x) {
+  T* op = p.out + (size_t)t * p.out_stride + (size_t)h * p.hsv;
+  for (int d = threadIdx.x; d < p.hsv; d += blockDim.x) {
     float o = 0.f;
 #pragma unroll
-    for (int w = 0; w < kWarps; ++w) o += acc_s[w * hsv + d] * wgt[w];
-    float res = ll > 0.f ? o / ll * out_scale : 0.f;
-    if (gate) res *= 1.0f / (1.0f + expf(-to_f32<T>(gate[(size_t)t * gate_stride + (size_t)h * hsv + d])));
+    for (int w = 0; w < kWarps; ++w) o += acc_s[w * p.hsv + d] * wgt[w];
+    float res = ll > 0.f ? o / ll * p.out_scale : 0.f;
+    if (p.gate) {
+      const size_t at = (size_t)t * p.gate_stride + (p.gate_per_head ? (size_t)h : (size_t)h * p.hsv + d);
+      res *= 1.0f / (1.0f + expf(-to_f32<T>(p.gate[at])));
+    }
     op[d] = from_f32<T>(res);
   }
 }
 
 }  // namespace
 
+// rel null: no bias per distance.  pool 0: no pooled blocks (the pool_* arguments are not read).
 YALIS_API int yalis_paged_attention_generic(const void* q, int q_stride, void* out, int out_stride,
                                             const void* k_pool, const void* v_pool, int dtype,
                                             const int32_t* positions, const int32_t* req_of_token,
@@ -131,17 +153,30 @@ YALIS_API int yalis_paged_attention_generic(const void* q, int q_stride, void* o
                                             int num_pages, int n_tokens, int nh, int g, int hs, int hsv,
                                             float scale, int window, float softcap, int sink, float out_scale,
                                             int chunk, const float* sink_logits, const float* slopes, const void* gate,
-                                            int gate_stride, cudaStream_t stream) {
+                                            int gate_stride, int gate_per_head, const float* rel, int rel_len, int pool,
+                                            const void* pk_pool, const void* pv_pool, const int32_t* pool_table,
+                                            int pool_table_width, int pool_page_size, int pool_num_pages,
+                                            cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
   if (hs <= 0 || hs > 32 * kMaxPerLane || hsv <= 0 || hsv > 32 * kMaxPerLane || g <= 0 || nh % g != 0 || nh > 65535)
     return YALIS_ERR_SHAPE;
+  if ((rel && rel_len < 1) || pool < 0 || (pool > 0 && (window <= 0 || chunk > 0 || !pk_pool || !pv_pool || !pool_table || pool_page_size < 1)))
+    return YALIS_ERR_SHAPE;
   const size_t smem = ((size_t)kWarps * hsv + 2 * kWarps) * sizeof(float);
   dim3 grid(n_tokens, nh);
-  YALIS_DISPATCH_DTYPE(dtype, T,
-                       return yalis_launch(paged_attention_generic_kernel<T>, grid, dim3(kWarps * 32), smem, stream,
-                                           (const T*)q, q_stride, (T*)out, out_stride, (const T*)k_pool,
-                                           (const T*)v_pool, positions, req_of_token, block_table, table_width,
-                                           page_size, num_pages, nh, g, hs, hsv, scale, window, softcap, sink, out_scale, chunk,
-                                           sink_logits, slopes, (const T*)gate, gate_stride));
+  YALIS_DISPATCH_DTYPE(dtype, T, {
+    GenericParams<T> p;
+    p.q = (const T*)q; p.q_stride = q_stride; p.out = (T*)out; p.out_stride = out_stride;
+    p.k_pool = (const T*)k_pool; p.v_pool = (const T*)v_pool;
+    p.positions = positions; p.req_of_token = req_of_token; p.block_table = block_table;
+    p.table_width = table_width; p.page_size = page_size; p.num_pages = num_pages;
+    p.nh = nh; p.g = g; p.hs = hs; p.hsv = hsv;
+    p.scale = scale; p.window = window; p.softcap = softcap; p.sink = sink; p.out_scale = out_scale; p.chunk = chunk;
+    p.sink_logits = sink_logits; p.slopes = slopes; p.rel = rel; p.rel_len = rel_len;
+    p.gate = (const T*)gate; p.gate_stride = gate_stride; p.gate_per_head = gate_per_head;
+    p.pool = pool; p.pk_pool = (const T*)pk_pool; p.pv_pool = (const T*)pv_pool; p.pool_table = pool_table;
+    p.pool_table_width = pool_table_width; p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
+    return yalis_launch(paged_attention_generic_kernel<T>, grid, dim3(kWarps * 32), smem, stream, p);
+  });
   return YALIS_OK;
 }

@@ -33,6 +33,13 @@
 // a factor on the result, and weights that meet V with 16 bits of mantissa instead of 8:
 // P is split into its bfloat16 rounding and the bfloat16 rounding of the rest, and both
 // halves go through the tensor cores (the sum of the weights is float32 in either form).
+//
+// The extended form (FORM 2) is the general form with head sizes that are known at launch only
+// (keys and values may differ; both multiples of 8, padded to one of three tile widths), a
+// learned bias per head and distance added to the scaled score, and pooled blocks: beside the
+// keys of its window a row sees one key and value for every block of P positions that lies
+// wholly before the window.  The blocks have pools and a block table of their own; their tiles
+// come first, then those of the window, in one softmax.
 #include "common.cuh"
 
 namespace {
@@ -66,6 +73,14 @@ struct AttnParams {
   const float* slopes;         // GEN: [nh] slope_h * (p - key) is taken off the score (null: none)
   const __nv_bfloat16* gate;   // GEN: [N, gate_stride] the result is multiplied by sigmoid(gate[t, head, :]) (null: not)
   int gate_stride;
+  int gate_per_head;           // GEN: the gate is [N, nh], one number per head
+  int hs, vs;                  // FORM 2: sizes of a key and a value (multiples of 8, at most HS)
+  const float* rel;            // FORM 2: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
+  int rel_len;
+  int pool;                    // FORM 2: P > 0: pooled blocks of P positions before the window
+  const __nv_bfloat16* pk_pool; const __nv_bfloat16* pv_pool;   // [pages, g, pool_page_size, HS / VS], an entry per block
+  const int32_t* pool_table;
+  int pool_table_width, pool_page_size, pool_num_pages;
   int n_splits;
   float* part_o;               // [N, nh, n_splits, HS] (split mode)
   float* part_ml;              // [N, nh, n_splits, 2]
@@ -142,6 +157,44 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* k_dst, __nv_bfloat16
   }
 }
 
+// The same for the extended form: keys and values of sizes known at launch, columns past them zero, from the token
+// pages or (`pooled`) from the pages of the pooled blocks.
+template <int HS>
+__device__ __forceinline__ void load_kv_tile_sized(__nv_bfloat16* k_dst, __nv_bfloat16* v_dst, const AttnParams& p, int req,
+                                                   int kvh, int key0, int lo_key, int hi_key, bool pooled) {
+  constexpr int CHUNKS = HS / 8, LD = HS + 8;
+  const int width = pooled ? p.pool_table_width : p.table_width;
+  const int32_t* bt = (pooled ? p.pool_table : p.block_table) + (size_t)req * width;
+  const int ps = pooled ? p.pool_page_size : p.page_size, pages = pooled ? p.pool_num_pages : p.num_pages;
+  const __nv_bfloat16* kp = pooled ? p.pk_pool : p.k_pool;
+  const __nv_bfloat16* vp = pooled ? p.pv_pool : p.v_pool;
+  constexpr int ITERS = BN * CHUNKS / (NWARPS * 32);
+  static_assert(BN * CHUNKS % (NWARPS * 32) == 0, "tile chunks must divide among the threads");
+  long long at[ITERS];                                    // row of the pool, -1: none
+#pragma unroll
+  for (int i = 0; i < ITERS; ++i) {
+    const int c = threadIdx.x + i * (NWARPS * 32);
+    const int key = key0 + c / CHUNKS;
+    at[i] = -1;
+    if (key >= lo_key && key <= hi_key) {
+      const int pi = key / ps;
+      const int page = pi < width ? bt[pi] : -1;
+      if (page >= 0 && page < pages) at[i] = ((long long)page * p.g + kvh) * ps + (key - pi * ps);
+    }
+  }
+#pragma unroll
+  for (int i = 0; i < ITERS; ++i) {
+    const int c = threadIdx.x + i * (NWARPS * 32);
+    const int row = c / CHUNKS, ch = c - row * CHUNKS;
+    __nv_bfloat16* kd = k_dst + row * LD + ch * 8;
+    __nv_bfloat16* vd = v_dst + row * LD + ch * 8;
+    if (at[i] >= 0 && ch * 8 < p.hs) cp_async16(kd, kp + at[i] * p.hs + ch * 8);
+    else *reinterpret_cast<uint4*>(kd) = make_uint4(0u, 0u, 0u, 0u);
+    if (at[i] >= 0 && ch * 8 < p.vs) cp_async16(vd, vp + at[i] * p.vs + ch * 8);
+    else *reinterpret_cast<uint4*>(vd) = make_uint4(0u, 0u, 0u, 0u);
+  }
+}
+
 // DEC: the block has at most 16 rows; warps split the keys of a tile instead of the rows.
 // A score in the exp2 domain: s * scale * log2(e), or with a cap c: c * tanh(s * scale / c) * log2(e).
 // `bias_log2`: what is taken off the scaled score before the cap, in the exp2 domain (the distance bias).
@@ -162,7 +215,8 @@ __device__ __forceinline__ float sink_log2(const AttnParams& p, int head) {
 }
 // sigmoid of the gate that belongs to out[tok, head, d].
 __device__ __forceinline__ float gate_factor(const AttnParams& p, int tok, int head, int hs, int d) {
-  return 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[(size_t)tok * p.gate_stride + (size_t)head * hs + d])));
+  const size_t at = (size_t)tok * p.gate_stride + (p.gate_per_head ? (size_t)head : (size_t)head * hs + d);
+  return 1.0f / (1.0f + __expf(-__bfloat162float(p.gate[at])));
 }
 // The first key a row at position `pos` sees.
 template <bool GEN>
@@ -170,6 +224,11 @@ __device__ __forceinline__ int first_visible(const AttnParams& p, int pos) {
   int lo = p.window > 0 ? max(0, pos - p.window + 1) : 0;
   if (GEN && p.chunk > 0) lo = max(lo, (pos / p.chunk) * p.chunk);
   return lo;
+}
+
+// How many pooled blocks a row at position `pos` sees: those that end at or before pos - window.
+__device__ __forceinline__ int blocks_seen(const AttnParams& p, int pos) {
+  return (p.pool > 0 && pos - p.window + 1 > 0) ? (pos - p.window + 1) / p.pool : 0;
 }
 
 // Normalisation of a finished row: with a sink the denominator gains exp2(0 - m) for the row's maximum m
@@ -184,8 +243,11 @@ __device__ __forceinline__ float finish_factor(const AttnParams& p, float m, flo
   return l > 0.f ? (GEN ? p.out_scale : 1.0f) / l : 0.f;
 }
 
-template <int HS, bool DEC, bool GEN>
+// FORM: 0 plain, 1 general, 2 extended (HS is then the padded size; p.hs and p.vs are the real ones).
+template <int HS, bool DEC, int FORM>
 __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const AttnParams p) {
+  constexpr bool GEN = FORM >= 1, EXT = FORM == 2;
+  const int hs = EXT ? p.hs : HS, vs = EXT ? p.vs : HS;
   constexpr int LD = HS + 8;            // padded row: ldmatrix rows fall into distinct banks
   constexpr int KSTEPS = HS / 16;       // k-steps of Q K^T
   constexpr int DT = HS / 8;            // n8 tiles of the output along the head dimension
@@ -228,7 +290,29 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     tile_lo = tile_lo + split * per_split;
     tile_hi = min(tile_hi, tile_lo + per_split);
   }
+  // Extended form: the tiles of the pooled blocks come first, `pool_tiles` of them; tile v < pool_tiles holds blocks
+  // [v * BN, ...), tile v >= pool_tiles the keys of tile first_key_tile + v - pool_tiles.
+  int pool_tiles = 0, first_key_tile = tile_lo, nb_last = 0;
+  if (EXT) {
+    first_key_tile = lo_key / BN;
+    nb_last = blocks_seen(p, pos_last);
+    pool_tiles = (nb_last + BN - 1) / BN;
+    const int total = pool_tiles + hi_key / BN + 1 - first_key_tile;
+    const int per_split = (total + p.n_splits - 1) / p.n_splits;
+    tile_lo = split * per_split;
+    tile_hi = min(total, tile_lo + per_split);
+  }
   const int n_tiles = max(0, tile_hi - tile_lo);
+  auto load_tile = [&](int buf, int tile) {       // tile: counted from the block's first (extended: over both kinds)
+    __nv_bfloat16* kd = k_s + buf * BN * LD;
+    __nv_bfloat16* vd = v_s + buf * BN * LD;
+    if constexpr (EXT) {
+      if (tile < pool_tiles) load_kv_tile_sized<HS>(kd, vd, p, req, kvh, tile * BN, 0, nb_last - 1, true);
+      else load_kv_tile_sized<HS>(kd, vd, p, req, kvh, (first_key_tile + tile - pool_tiles) * BN, lo_key, hi_key, false);
+    } else {
+      load_kv_tile<HS>(kd, vd, bt, p, kvh, tile * BN, lo_key, hi_key);
+    }
+  };
 
   // ---- Q tile -> shared memory, then this warp's A fragments ----------------------
   {
@@ -237,9 +321,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       const int r = c / CHUNKS, ch = c - r * CHUNKS;
       const int row = row0 + r;
       __nv_bfloat16* d = q_s + r * LD + ch * 8;
-      if (row < n_rows) {
+      if (row < n_rows && (!EXT || ch * 8 < hs)) {
         const int t = row / p.per, h = row - t * p.per;
-        cp_async16(d, p.q + (size_t)(tok0 + t) * p.q_stride + (size_t)(kvh * p.per + h) * HS + ch * 8);
+        cp_async16(d, p.q + (size_t)(tok0 + t) * p.q_stride + (size_t)(kvh * p.per + h) * hs + ch * 8);
       } else {
         *reinterpret_cast<uint4*>(d) = make_uint4(0u, 0u, 0u, 0u);
       }
@@ -248,8 +332,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   // Prologue: Q and the first tile form one group, then NST-2 further tiles one group each.
 #pragma unroll
   for (int t = 0; t < NST - 1; ++t) {
-    if (t < n_tiles)
-      load_kv_tile<HS>(k_s + t * BN * LD, v_s + t * BN * LD, bt, p, kvh, (tile_lo + t) * BN, lo_key, hi_key);
+    if (t < n_tiles) load_tile(t, tile_lo + t);
     cp_async_commit();
   }
   cp_async_wait<NST - 2>();     // the group with Q and tile 0 has landed
@@ -266,6 +349,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   int row_pos[2], row_lo[2];
   bool row_ok[2];
   float row_slope[2] = {0.f, 0.f};      // in the exp2 domain
+  int row_blocks[2] = {0, 0};           // extended: pooled blocks the row sees
+  const float* row_rel[2] = {nullptr, nullptr};
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int row = row0 + wrow + gid + i * 8;
@@ -273,7 +358,12 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     row_pos[i] = row_ok[i] ? p.positions[tok0 + row / p.per] : -1;
     row_lo[i] = row_ok[i] ? first_visible<GEN>(p, row_pos[i]) : 0;
     if (GEN && p.slopes && row_ok[i]) row_slope[i] = p.slopes[kvh * p.per + row % p.per] * 1.4426950408889634f;
+    if (EXT && row_ok[i]) {
+      row_blocks[i] = blocks_seen(p, row_pos[i]);
+      if (p.rel) row_rel[i] = p.rel + (size_t)(kvh * p.per + row % p.per) * p.rel_len;
+    }
   }
+  const int nb_first = EXT ? blocks_seen(p, pos_first) : 0;
 
   float o[DT][4];
 #pragma unroll
@@ -282,12 +372,10 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 
   for (int it = 0; it < n_tiles; ++it) {
     const int buf = it % NST;
-    const int key0 = (tile_lo + it) * BN;
+    const bool pooled = EXT && tile_lo + it < pool_tiles;
+    const int key0 = (EXT && !pooled ? first_key_tile - pool_tiles + tile_lo + it : tile_lo + it) * BN;
     // prefetch tile it + NST - 1 into the buffer that tile it - 1 has left
-    if (it + NST - 1 < n_tiles) {
-      const int nb = (it + NST - 1) % NST;
-      load_kv_tile<HS>(k_s + nb * BN * LD, v_s + nb * BN * LD, bt, p, kvh, key0 + (NST - 1) * BN, lo_key, hi_key);
-    }
+    if (it + NST - 1 < n_tiles) load_tile((it + NST - 1) % NST, tile_lo + it + NST - 1);
     cp_async_commit();
     const __nv_bfloat16* kt = k_s + buf * BN * LD;
     const __nv_bfloat16* vt = v_s + buf * BN * LD;
@@ -298,6 +386,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     for (int j = 0; j < ST; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < KSTEPS; ++ks) {
+      if (EXT && ks * 16 >= hs) continue;
 #pragma unroll
       for (int j = 0; j < ST; j += 2) {
         unsigned kb[4];
@@ -311,7 +400,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     // ---- mask, online softmax (exp2 domain) -----------------------------------------
     float m_new[2] = {m_run[0], m_run[1]};
     // A tile strictly inside every row's visible range needs no mask (the common case in decode).
-    const bool inner = key0 + BN - 1 <= pos_first && key0 >= lo_last && row0 + RB <= n_rows && !(GEN && p.slopes);
+    const bool inner = pooled ? key0 + BN <= nb_first && row0 + RB <= n_rows
+                              : key0 + BN - 1 <= pos_first && key0 >= lo_last && row0 + RB <= n_rows &&
+                                    !(GEN && p.slopes) && !(EXT && p.rel);
     if (inner) {
 #pragma unroll
       for (int j = 0; j < ST; ++j) {
@@ -328,8 +419,17 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
         for (int e = 0; e < 4; ++e) {
           const int i = e >> 1;
           const int key = key0 + wkey + j * 8 + tig * 2 + (e & 1);
-          const bool vis = row_ok[i] && key <= row_pos[i] && key >= row_lo[i];
-          const float v = vis ? score_log2<GEN>(p, s[j][e], row_slope[i] * (float)(row_pos[i] - key)) : -INFINITY;
+          bool vis = row_ok[i] && key <= row_pos[i] && key >= row_lo[i];
+          float off = row_slope[i] * (float)(row_pos[i] - key);
+          if (EXT) {
+            if (pooled) {
+              vis = key < row_blocks[i];
+              off = 0.f;
+            } else if (vis && p.rel) {
+              off -= __ldg(row_rel[i] + min(row_pos[i] - key, p.rel_len - 1)) * 1.4426950408889634f;
+            }
+          }
+          const float v = vis ? score_log2<GEN>(p, s[j][e], off) : -INFINITY;
           s[j][e] = v;
           m_new[i] = fmaxf(m_new[i], v);
         }
@@ -370,6 +470,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       for (int kk = 0; kk < ST / 2; ++kk) {
 #pragma unroll
         for (int d = 0; d < DT; d += 2) {
+          if (EXT && d * 8 >= vs) continue;
           unsigned vb[4];
           const int key = wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
           const int dim = d * 8 + (lane >> 4) * 8;
@@ -411,6 +512,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
         }
 #pragma unroll
         for (int d = 0; d < DT; d += 2) {
+          if (EXT && d * 8 >= vs) continue;
           unsigned vb[4];
           const int key = wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
           const int dim = d * 8 + (lane >> 4) * 8;
@@ -451,8 +553,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     }
     __syncthreads();
     const int rows_here = min(16, n_rows - row0);
-    for (int e = threadIdx.x; e < rows_here * HS; e += NWARPS * 32) {
-      const int r = e / HS, d = e - r * HS;
+    for (int e = threadIdx.x; e < rows_here * vs; e += NWARPS * 32) {
+      const int r = e / vs, d = e - r * vs;
       float mm = -INFINITY;
 #pragma unroll
       for (int w = 0; w < NWARPS; ++w) mm = fmaxf(mm, mml[(w * 16 + r) * 2]);
@@ -477,11 +579,11 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
           mm = up;
         }
         float res = acc * finish_factor<GEN>(p, mm, ll, sz);
-        if (GEN && p.gate) res *= gate_factor(p, tok, head, HS, d);
-        p.out[(size_t)tok * p.out_stride + (size_t)head * HS + d] = __float2bfloat16_rn(res);
+        if (GEN && p.gate) res *= gate_factor(p, tok, head, vs, d);
+        p.out[(size_t)tok * p.out_stride + (size_t)head * vs + d] = __float2bfloat16_rn(res);
       } else {
         const size_t slot = ((size_t)tok * p.nh + head) * p.n_splits + split;
-        p.part_o[slot * HS + d] = acc;
+        p.part_o[slot * vs + d] = acc;
         if (d == 0) {
           p.part_ml[slot * 2] = mm;
           p.part_ml[slot * 2 + 1] = ll;
@@ -497,8 +599,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       __syncthreads();
       if (s_last) {
         __threadfence();
-        for (int e = threadIdx.x; e < rows_here * HS; e += NWARPS * 32) {
-          const int r = e / HS, d = e - r * HS;
+        for (int e = threadIdx.x; e < rows_here * vs; e += NWARPS * 32) {
+          const int r = e / vs, d = e - r * vs;
           const int row = row0 + r;
           const int t = row / p.per, h = row - t * p.per;
           const int tok = tok0 + t, head = kvh * p.per + h;
@@ -512,7 +614,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
             const float m = ml[(base + sp) * 2];
             const float f = (m == -INFINITY) ? 0.f : exp2f(m - mm);
             ll += ml[(base + sp) * 2 + 1] * f;
-            acc += po[(base + sp) * HS + d] * f;
+            acc += po[(base + sp) * vs + d] * f;
           }
           float sz = 0.f;
           if (GEN && p.sink) {
@@ -523,8 +625,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
             mm = up;
           }
           float res = acc * finish_factor<GEN>(p, mm, ll, sz);
-          if (GEN && p.gate) res *= gate_factor(p, tok, head, HS, d);
-          p.out[(size_t)tok * p.out_stride + (size_t)head * HS + d] = __float2bfloat16_rn(res);
+          if (GEN && p.gate) res *= gate_factor(p, tok, head, vs, d);
+          p.out[(size_t)tok * p.out_stride + (size_t)head * vs + d] = __float2bfloat16_rn(res);
         }
         if (threadIdx.x == 0) p.tickets[blockIdx.y] = 0;
       }
@@ -545,13 +647,14 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     } else {
       inv = finish_factor<GEN>(p, m_run[i], l_run[i]);
     }
-    __nv_bfloat16* dst = p.out + (size_t)tok * p.out_stride + (size_t)head * HS;
+    __nv_bfloat16* dst = p.out + (size_t)tok * p.out_stride + (size_t)head * vs;
 #pragma unroll
     for (int d = 0; d < DT; ++d) {
+      if (EXT && d * 8 >= vs) continue;
       float v0 = o[d][i * 2] * inv, v1 = o[d][i * 2 + 1] * inv;
       if (GEN && p.gate) {
-        v0 *= gate_factor(p, tok, head, HS, d * 8 + tig * 2);
-        v1 *= gate_factor(p, tok, head, HS, d * 8 + tig * 2 + 1);
+        v0 *= gate_factor(p, tok, head, vs, d * 8 + tig * 2);
+        v1 *= gate_factor(p, tok, head, vs, d * 8 + tig * 2 + 1);
       }
       *reinterpret_cast<__nv_bfloat162*>(dst + d * 8 + tig * 2) = __floats2bfloat162_rn(v0, v1);
     }
@@ -559,31 +662,37 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   }
 }
 
-template <int HS, bool DEC, bool GEN>
+template <int HS, bool DEC, int FORM>
 int launch_mode(const AttnParams& p, int n_requests, int max_rows, cudaStream_t stream) {
   constexpr int LD = HS + 8;
   constexpr int RB = DEC ? 16 : BM, NST = DEC ? 3 : 2;
   const size_t smem = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
   static bool configured = false;
   if (!configured) {
-    if (cudaFuncSetAttribute(paged_attention_mma_kernel<HS, DEC, GEN>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+    if (cudaFuncSetAttribute(paged_attention_mma_kernel<HS, DEC, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize,
                              (int)smem) != cudaSuccess)
       return YALIS_ERR_LAUNCH;
     configured = true;
   }
   dim3 grid((max_rows + RB - 1) / RB, n_requests * p.g, p.n_splits);
   if (grid.y > 65535 || grid.z > 65535) return YALIS_ERR_SHAPE;
-  return yalis_launch(paged_attention_mma_kernel<HS, DEC, GEN>, grid, dim3(NWARPS * 32), smem, stream, p);
+  return yalis_launch(paged_attention_mma_kernel<HS, DEC, FORM>, grid, dim3(NWARPS * 32), smem, stream, p);
 }
 
 template <int HS>
 int launch(const AttnParams& p, int n_requests, int max_rows, cudaStream_t stream) {
   const bool general = p.cap_log2 > 0.f || p.sink || p.out_scale != 1.0f || p.exact_weights || p.chunk > 0 || p.slopes || p.gate;
   if (general)
-    return max_rows <= 16 ? launch_mode<HS, true, true>(p, n_requests, max_rows, stream)
-                          : launch_mode<HS, false, true>(p, n_requests, max_rows, stream);
-  return max_rows <= 16 ? launch_mode<HS, true, false>(p, n_requests, max_rows, stream)
-                        : launch_mode<HS, false, false>(p, n_requests, max_rows, stream);
+    return max_rows <= 16 ? launch_mode<HS, true, 1>(p, n_requests, max_rows, stream)
+                          : launch_mode<HS, false, 1>(p, n_requests, max_rows, stream);
+  return max_rows <= 16 ? launch_mode<HS, true, 0>(p, n_requests, max_rows, stream)
+                        : launch_mode<HS, false, 0>(p, n_requests, max_rows, stream);
+}
+
+template <int HS>
+int launch_extended(const AttnParams& p, int n_requests, int max_rows, cudaStream_t stream) {
+  return max_rows <= 16 ? launch_mode<HS, true, 2>(p, n_requests, max_rows, stream)
+                        : launch_mode<HS, false, 2>(p, n_requests, max_rows, stream);
 }
 
 }  // namespace
@@ -598,13 +707,20 @@ YALIS_API int yalis_attention_mma_supports(int hs) {
   }
 }
 
-// Scratch floats needed for n_splits > 1: part_o then part_ml.  Besides, `tickets` needs
+// Whether the extended form takes keys of size hs and values of size vs.
+YALIS_API int yalis_attention_mma_extended_supports(int hs, int vs) {
+  return hs >= 8 && vs >= 8 && hs <= 256 && vs <= 256 && hs % 8 == 0 && vs % 8 == 0;
+}
+
+// Scratch floats (hs: the size of a value) needed for n_splits > 1: part_o then part_ml.  Besides, `tickets` needs
 // n_requests * g int32 that are zero before the first launch (each launch leaves them zero).
 YALIS_API long long yalis_attention_mma_scratch_floats(int n_tokens, int nh, int hs, int n_splits) {
   return n_splits > 1 ? (long long)n_tokens * nh * n_splits * (hs + 2) : 0;
 }
 
-// softcap 0: none.  With a cap, a sink, a factor other than 1 or exact_weights the general form of the kernel runs.
+// softcap 0: none.  With a cap, a sink, a factor other than 1 or exact_weights the general form of the kernel runs;
+// with vs != hs, a bias per distance (rel), pooled blocks (pool > 0) or a head size that has no kernel of its own the
+// extended form.
 YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                                 const void* v_pool, const int32_t* positions, const int32_t* q_start,
                                                 const int32_t* req_of_token, const int32_t* block_table, int table_width,
@@ -613,6 +729,9 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
                                                 int32_t* tickets, float softcap, int sink, float out_scale,
                                                 int exact_weights, int chunk, const float* sink_logits,
                                                 const float* slopes, const void* gate, int gate_stride,
+                                                int gate_per_head, int vs, const float* rel, int rel_len, int pool,
+                                                const void* pk_pool, const void* pv_pool, const int32_t* pool_table,
+                                                int pool_table_width, int pool_page_size, int pool_num_pages,
                                                 cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return YALIS_OK;
   if (softcap < 0.f) return YALIS_ERR_SHAPE;
@@ -635,16 +754,32 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
   p.sink = sink; p.out_scale = out_scale; p.exact_weights = exact_weights;
   p.window = window; p.n_splits = n_splits;
   p.chunk = chunk; p.sink_logits = sink ? sink_logits : nullptr; p.slopes = slopes;
-  p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride;
+  p.gate = (const __nv_bfloat16*)gate; p.gate_stride = gate_stride; p.gate_per_head = gate_per_head;
+  p.hs = hs; p.vs = vs; p.rel = rel; p.rel_len = rel_len; p.pool = pool;
+  p.pk_pool = (const __nv_bfloat16*)pk_pool; p.pv_pool = (const __nv_bfloat16*)pv_pool; p.pool_table = pool_table;
+  p.pool_table_width = pool_table_width; p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
+  const bool extended = vs != hs || rel != nullptr || pool > 0 || !yalis_attention_mma_supports(hs);
+  if (pool < 0 || (rel && rel_len < 1)) return YALIS_ERR_SHAPE;
+  if (pool > 0) {
+    if (window <= 0 || chunk > 0 || !pk_pool || !pv_pool || !pool_table || pool_page_size < 1) return YALIS_ERR_SHAPE;
+    if (((uintptr_t)pk_pool | (uintptr_t)pv_pool) & 15) return YALIS_ERR_ALIGN;
+  }
+  if (extended && !yalis_attention_mma_extended_supports(hs, vs)) return YALIS_ERR_SHAPE;
   if (chunk < 0) return YALIS_ERR_SHAPE;
   p.part_o = nullptr; p.part_ml = nullptr; p.tickets = tickets;
   if (n_splits > 1) {
     if (scratch == nullptr || tickets == nullptr || max_q_len * p.per > 16) return YALIS_ERR_SHAPE;
     p.part_o = scratch;
-    p.part_ml = scratch + (size_t)n_tokens * nh * n_splits * hs;
+    p.part_ml = scratch + (size_t)n_tokens * nh * n_splits * vs;
   }
   const int max_rows = max_q_len * p.per;
   int st;
+  if (extended) {
+    const int widest = hs > vs ? hs : vs;
+    if (widest <= 64) return launch_extended<64>(p, n_requests, max_rows, stream);
+    if (widest <= 128) return launch_extended<128>(p, n_requests, max_rows, stream);
+    return launch_extended<256>(p, n_requests, max_rows, stream);
+  }
   switch (hs) {
     case 16: st = launch<16>(p, n_requests, max_rows, stream); break;
     case 32: st = launch<32>(p, n_requests, max_rows, stream); break;
@@ -706,7 +841,7 @@ YALIS_API int yalis_paged_attention_mma(const void* q, int q_stride, void* out, 
   return yalis_paged_attention_mma_general(q, q_stride, out, out_stride, k_pool, v_pool, positions, q_start, req_of_token,
                                            block_table, table_width, page_size, num_pages, n_tokens, n_requests, max_q_len,
                                            nh, g, hs, scale, window, n_splits, scratch, tickets, 0.f, 0, 1.0f, 0, 0, nullptr, nullptr,
-                                           nullptr, 0, stream);
+                                           nullptr, 0, 0, hs, nullptr, 0, 0, nullptr, nullptr, nullptr, 0, 0, 0, stream);
 }
 
 YALIS_API long long yalis_paged_attention_mma_noalloc_needed(int n_tokens, int n_requests, int nh, int g, int hs,

@@ -370,17 +370,47 @@ YALIS_API int yalis_add_rmsnorm(float* x, const void* delta, int delta_dtype, in
 // The same with a sub-layer's result that is itself normed (and may carry a bias) before it joins the stream:
 //   d = sum_s delta[s][r] (+ bias)                       float32
 //   d <- d * rsqrt(mean(d^2) + d_eps) * d_w             (only with d_w)
+//   with a second result d2 = sum_s delta2[s][r] of its own norm:  d <- d + d2 * rsqrt(mean(d2^2) + d2_eps) * d2_w
+//   d <- d * factor * scale                              (scale: a learned vector, or absent)
 //   h = x[r] + d;  x[r] = h (when write_back);  y[i] = (h * rsqrt(mean(h^2) + eps)) * w  (only with w)
 // One block per row; the row waits in shared memory between the passes, so every value is read once.
 // --------------------------------------------------------------------------
+// What may stand behind the first result: a factor and a vector on the sum, and a second normed result.
+struct SumTail {
+  const float* scale;                 // [width] or null
+  float factor;
+  const void* d2; int d2_f32;         // [n2][rows][width] in float32 or bfloat16, or null
+  int n2; size_t stride2;
+  const float* d2_w; float d2_eps;
+};
+__device__ __forceinline__ float tail_value(const SumTail& t, size_t row_off) {
+  return t.d2_f32 ? sum_parts<float>(reinterpret_cast<const float*>(t.d2) + row_off, t.n2, t.stride2)
+                  : sum_parts<__nv_bfloat16>(reinterpret_cast<const __nv_bfloat16*>(t.d2) + row_off, t.n2, t.stride2);
+}
+__device__ __forceinline__ float4 tail_value4(const SumTail& t, size_t row_off) {
+  if (!t.d2_f32) return load4_f32(reinterpret_cast<const __nv_bfloat16*>(t.d2) + row_off);     // a bfloat16 result has one part
+  const float* p = reinterpret_cast<const float*>(t.d2) + row_off;
+  float4 acc = make_float4(0.f, 0.f, 0.f, 0.f);
+  for (int s0 = 0; s0 < t.n2; s0 += 4) {
+    float4 v[4];
+#pragma unroll
+    for (int j = 0; j < 4; ++j) v[j] = s0 + j < t.n2 ? load4_f32(p + (size_t)(s0 + j) * t.stride2) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int j = 0; j < 4; ++j) {
+      acc.x += v[j].x; acc.y += v[j].y; acc.z += v[j].z; acc.w += v[j].w;
+    }
+  }
+  return acc;
+}
+
 template <typename T, typename TD>
 __global__ void __launch_bounds__(1024) add_normed_rmsnorm_kernel(float* __restrict__ x, const TD* __restrict__ delta, int n_delta,
                                                                   size_t delta_stride, const float* __restrict__ bias,
                                                                   const float* __restrict__ d_w, float d_eps,
                                                                   const float* __restrict__ w, T* __restrict__ y,
                                                                   const int32_t* __restrict__ rows, int width, float eps,
-                                                                  int write_back) {
-  extern __shared__ float row_s[];        // [width]
+                                                                  int write_back, const SumTail tail) {
+  extern __shared__ float row_s[];        // [width], with a second result [2 * width]
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -398,9 +428,22 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_kernel(float* __restr
   }
   float d_inv = 1.0f;
   if (d_w) d_inv = rsqrtf(block_sum(ss, scratch) / (float)width + d_eps);
+  float d2_inv = 0.f;
+  if (tail.d2) {
+    ss = 0.f;
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float d2 = tail_value(tail, (size_t)r * width + c);
+      row_s[width + c] = d2;
+      ss = __fmaf_rn(d2, d2, ss);
+    }
+    d2_inv = rsqrtf(block_sum(ss, scratch) / (float)width + tail.d2_eps);
+  }
   ss = 0.f;
   for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float d = d_w ? (row_s[c] * d_inv) * d_w[c] : row_s[c];
+    float d = d_w ? (row_s[c] * d_inv) * d_w[c] : row_s[c];
+    if (tail.d2) d += (row_s[width + c] * d2_inv) * tail.d2_w[c];
+    d *= tail.factor;
+    if (tail.scale) d *= tail.scale[c];
     const float h = xr[c] + d;
     if (write_back) xr[c] = h;
     row_s[c] = h;
@@ -416,14 +459,15 @@ __global__ void __launch_bounds__(1024) add_normed_rmsnorm_kernel(float* __restr
 // groups of four columns in registers from the first load to the last store (no shared-memory row), and the three
 // weight vectors are fetched before the wait for the preceding kernel.  Same order of sums per element as above
 // except inside the two means, which are fixed-order block reductions in both.
-template <typename T, typename TD, int NV>
+// TAIL: a second result, a factor or a vector on the sum may follow (their loads are left where they are used).
+template <typename T, typename TD, int NV, bool TAIL>
 __global__ void __launch_bounds__(NV == 1 ? 1024 : 256, NV == 2 ? 3 : 1) add_normed_rmsnorm_vec_kernel(float* __restrict__ x, const TD* __restrict__ delta,
                                                                       int n_delta, size_t delta_stride,
                                                                       const float* __restrict__ bias,
                                                                       const float* __restrict__ d_w, float d_eps,
                                                                       const float* __restrict__ w, T* __restrict__ y,
                                                                       const int32_t* __restrict__ rows, int width, float eps,
-                                                                      int write_back) {
+                                                                      int write_back, const SumTail tail) {
   __shared__ float scratch[32];
   pdl_launch_dependents();
   const int n4 = width >> 2;
@@ -483,6 +527,34 @@ __global__ void __launch_bounds__(NV == 1 ? 1024 : 256, NV == 2 ? 3 : 1) add_nor
       d[v].z = (d[v].z * d_inv) * dwv[v].z; d[v].w = (d[v].w * d_inv) * dwv[v].w;
     }
   }
+  if constexpr (TAIL) {
+    if (tail.d2) {
+      float4 e[NV];
+      ss = 0.f;
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int c = threadIdx.x + v * blockDim.x;
+        e[v] = c < n4 ? tail_value4(tail, (size_t)r * width + 4 * c) : zero4;
+        ss += (e[v].x * e[v].x + e[v].y * e[v].y) + (e[v].z * e[v].z + e[v].w * e[v].w);
+      }
+      const float inv2 = rsqrtf(block_sum(ss, scratch) / (float)width + tail.d2_eps);
+#pragma unroll
+      for (int v = 0; v < NV; ++v) {
+        const int c = threadIdx.x + v * blockDim.x;
+        const float4 w2 = c < n4 ? load4_f32(tail.d2_w + 4 * c) : zero4;
+        d[v].x += (e[v].x * inv2) * w2.x; d[v].y += (e[v].y * inv2) * w2.y;
+        d[v].z += (e[v].z * inv2) * w2.z; d[v].w += (e[v].w * inv2) * w2.w;
+      }
+    }
+#pragma unroll
+    for (int v = 0; v < NV; ++v) {
+      const int c = threadIdx.x + v * blockDim.x;
+      float4 sc = make_float4(1.f, 1.f, 1.f, 1.f);
+      if (tail.scale && c < n4) sc = load4_f32(tail.scale + 4 * c);
+      d[v].x = d[v].x * tail.factor * sc.x; d[v].y = d[v].y * tail.factor * sc.y;
+      d[v].z = d[v].z * tail.factor * sc.z; d[v].w = d[v].w * tail.factor * sc.w;
+    }
+  }
   ss = 0.f;
 #pragma unroll
   for (int v = 0; v < NV; ++v) {
@@ -506,45 +578,63 @@ __global__ void __launch_bounds__(NV == 1 ? 1024 : 256, NV == 2 ? 3 : 1) add_nor
 template <typename T, typename TD>
 int launch_add_normed_rmsnorm(float* x, const void* delta, int n_delta, size_t delta_stride, const float* bias, const float* d_w,
                               float d_eps, const float* w, void* y, const int32_t* rows, int n_out_rows, int width, float eps,
-                              int write_back, cudaStream_t stream) {
-  const uintptr_t ptrs = (uintptr_t)x | (uintptr_t)delta | (uintptr_t)bias | (uintptr_t)d_w | (uintptr_t)w | (uintptr_t)y;
-  if (width % 4 == 0 && width <= 16384 && (ptrs & 15) == 0 && delta_stride % 4 == 0) {
+                              int write_back, const SumTail& tail, cudaStream_t stream) {
+  const uintptr_t ptrs = (uintptr_t)x | (uintptr_t)delta | (uintptr_t)bias | (uintptr_t)d_w | (uintptr_t)w | (uintptr_t)y |
+                         (uintptr_t)tail.scale | (uintptr_t)tail.d2 | (uintptr_t)tail.d2_w;
+  const bool has_tail = tail.scale || tail.d2 || tail.factor != 1.0f;
+  if (width % 4 == 0 && width <= 16384 && (ptrs & 15) == 0 && delta_stride % 4 == 0 && tail.stride2 % 4 == 0) {
     const int n4 = width / 4;
     // few rows: a thread per group of four where a block can hold them; otherwise 256 threads a row with up to four
     // groups each (more rows in flight per SM, registers to spare); wider rows take the shared-memory form below
     const int cap = (n_out_rows < 256 && n4 <= 1024) ? 1024 : 256;
     const int vthreads = n4 >= cap ? cap : (n4 + 31) / 32 * 32;
     const int nv = (n4 + vthreads - 1) / vthreads;
-#define YALIS_NNORM_VEC(V)                                                                                           \
-  return yalis_launch(add_normed_rmsnorm_vec_kernel<T, TD, V>, dim3(n_out_rows), dim3(vthreads), 0, stream, x,       \
-                      (const TD*)delta, n_delta, delta_stride, bias, d_w, d_eps, w, (T*)y, rows, width, eps, write_back)
+#define YALIS_NNORM_VEC_T(V, TAIL)                                                                                   \
+  return yalis_launch(add_normed_rmsnorm_vec_kernel<T, TD, V, TAIL>, dim3(n_out_rows), dim3(vthreads), 0, stream, x, \
+                      (const TD*)delta, n_delta, delta_stride, bias, d_w, d_eps, w, (T*)y, rows, width, eps, write_back, tail)
+#define YALIS_NNORM_VEC(V)                \
+  do {                                    \
+    if (has_tail) YALIS_NNORM_VEC_T(V, true); \
+    else YALIS_NNORM_VEC_T(V, false);     \
+  } while (0)
     if (nv == 1) YALIS_NNORM_VEC(1);
     else if (nv == 2) YALIS_NNORM_VEC(2);
     else if (nv <= 4) YALIS_NNORM_VEC(4);
 #undef YALIS_NNORM_VEC
+#undef YALIS_NNORM_VEC_T
   }
-  if (width > 48 * 1024 / 4) return YALIS_ERR_SHAPE;
+  const size_t smem = (size_t)width * (tail.d2 ? 2 : 1) * sizeof(float);
+  if (smem > 200 * 1024) return YALIS_ERR_SHAPE;
+  if (smem > 48 * 1024 && cudaFuncSetAttribute(add_normed_rmsnorm_kernel<T, TD>, cudaFuncAttributeMaxDynamicSharedMemorySize,
+                                               200 * 1024) != cudaSuccess)
+    return YALIS_ERR_LAUNCH;
   const int threads = width >= 2048 ? 512 : (width >= 512 ? 256 : 128);
-  return yalis_launch(add_normed_rmsnorm_kernel<T, TD>, dim3(n_out_rows), dim3(threads), (size_t)width * sizeof(float), stream, x,
-                      (const TD*)delta, n_delta, delta_stride, bias, d_w, d_eps, w, (T*)y, rows, width, eps, write_back);
+  return yalis_launch(add_normed_rmsnorm_kernel<T, TD>, dim3(n_out_rows), dim3(threads), smem, stream, x, (const TD*)delta, n_delta,
+                      delta_stride, bias, d_w, d_eps, w, (T*)y, rows, width, eps, write_back, tail);
 }
 
-// delta: [n_delta][rows_total][width] in delta_dtype; bias, d_w, w float32 [width] or null; y in out_dtype (unused
-// without w).
+// delta: [n_delta][rows_total][width] in delta_dtype; bias, d_w, w, scale float32 [width] or null; y in out_dtype (unused
+// without w).  delta2: a second result [n2][rows_total][width] in delta2_dtype with its own norm (d2_w, d2_eps), or null.
 YALIS_API int yalis_add_normed_rmsnorm(float* x, const void* delta, int delta_dtype, int n_delta, long long delta_stride,
                                        const float* bias, const float* d_w, float d_eps, const float* w, void* y,
                                        int out_dtype, const int32_t* rows, int n_out_rows, int width, float eps,
-                                       int write_back, cudaStream_t stream) {
+                                       int write_back, const float* scale, float factor, const void* delta2, int delta2_dtype,
+                                       int n2, long long stride2, const float* d2_w, float d2_eps, cudaStream_t stream) {
   if (n_out_rows <= 0) return YALIS_OK;
   if (delta == nullptr || n_delta <= 0 || width <= 0) return YALIS_ERR_SHAPE;
+  if (delta2 != nullptr && (n2 <= 0 || d2_w == nullptr || (delta2_dtype != YALIS_F32 && (delta2_dtype != YALIS_BF16 || n2 != 1))))
+    return YALIS_ERR_SHAPE;
+  SumTail tail;
+  tail.scale = scale; tail.factor = factor; tail.d2 = delta2; tail.d2_f32 = delta2_dtype == YALIS_F32;
+  tail.n2 = n2; tail.stride2 = (size_t)stride2; tail.d2_w = d2_w; tail.d2_eps = d2_eps;
   YALIS_DISPATCH_DTYPE(
       out_dtype, T,
       if (delta_dtype == YALIS_F32) {
         return launch_add_normed_rmsnorm<T, float>(x, delta, n_delta, (size_t)delta_stride, bias, d_w, d_eps, w, y, rows,
-                                                   n_out_rows, width, eps, write_back, stream);
+                                                   n_out_rows, width, eps, write_back, tail, stream);
       } else if (delta_dtype == YALIS_BF16) {
         return launch_add_normed_rmsnorm<T, __nv_bfloat16>(x, delta, n_delta, (size_t)delta_stride, bias, d_w, d_eps, w, y, rows,
-                                                           n_out_rows, width, eps, write_back, stream);
+                                                           n_out_rows, width, eps, write_back, tail, stream);
       } else { return YALIS_ERR_DTYPE; });
   return YALIS_OK;
 }

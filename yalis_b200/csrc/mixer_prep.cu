@@ -1,8 +1,9 @@
 // What lies between a mixer's input projection and its core, for mixers whose heads are
 // prepared in more ways than a full rotation: an added bias, a norm over the head with a
-// learned scale, a rotation of only the first `rot_dims` sizes, a constant factor, value heads
-// of a size of their own.  Queries go to a plain matrix; keys and values go to the pages of a
-// cache or to plain matrices (for mixers that keep a state instead of keys).  Also the
+// learned scale (or over all heads at once), a rotation of only the first `rot_dims` sizes, a
+// constant factor, value heads of a size of their own.  Queries go to a plain matrix; keys and values go to the pages of a
+// cache or to plain matrices (for mixers that keep a state instead of keys); blocks of P
+// consecutive cached keys and values may be kept as their means besides.  Also the
 // element-wise activations of dense feed-forwards and the row-wise additions of looped layers.
 // All arithmetic is float32; sines and cosines come from sincosf of a float32 angle.
 #include "common.cuh"
@@ -18,6 +19,8 @@ struct PrepParams {
   const float* q_norm; const float* k_norm; float norm_eps;       // scale over dim, or null: no norm
   const float* inv_freq; int rot_dims;                            // [rot_dims / 2], or null: no rotation
   int rot_interleaved;                                            // pair i is (2i, 2i + 1) instead of (i, i + rot_dims / 2)
+  float rot_scale;                                                // factor on cosine and sine
+  int norm_all;                                                   // the norm is over all heads of q (of k) at once, scales [heads * dim]
   float q_scale, k_scale;
   float q_temp_coef; int q_temp_every;                            // every > 0: q *= 1 + coef * ln(floor((pos + 1) / every) + 1)
   void* q_out; int q_out_stride;             // [N, nq * dim]
@@ -28,85 +31,178 @@ struct PrepParams {
   const int32_t* positions; const int32_t* req_of_token;
   int nq, nk, dim, vdim;
   int32_t* bad_page;
+  int pool;                                  // P > 0: the warp that stores the last row of a block of P positions stores their mean
+  void* pk_pool; void* pv_pool;              // [pages, nk, pool_page_size, dim] and [..., vdim], an entry per block
+  const int32_t* pool_table; int pool_table_width, pool_page_size, pool_num_pages;
 };
 
-// One warp per (token, head): heads [0, nq) are queries, [nq, nq + nk) keys, [nq + nk, nq + 2 nk) values.
+// Where a request's cached row `at` lies in pages of `page_size` rows: its index among the rows of one head, or -1.
+__device__ __forceinline__ long long paged_row(const int32_t* table, int width, int page_size, int num_pages, int nk, int head,
+                                               int at) {
+  const int pi = at / page_size;
+  const int page = pi < width ? table[pi] : -1;
+  return page < 0 || page >= num_pages ? -1 : ((long long)page * nk + head) * page_size + (at - pi * page_size);
+}
+
+// The mean of a head's cached rows at positions pos - P + 1 .. pos, added in order in float32, goes to entry pos / P.
+// One warp; every row must be stored and visible to it.
+template <typename T>
+__device__ void store_block_mean(const PrepParams& p, int req, int pos, int head, bool is_v, int lane) {
+  const int width = is_v ? p.vdim : p.dim;
+  const T* rows = reinterpret_cast<const T*>(is_v ? p.v_pool : p.k_pool);
+  const int32_t* table = p.block_table + (size_t)req * p.table_width;
+  const long long entry = paged_row(p.pool_table + (size_t)req * p.pool_table_width, p.pool_table_width, p.pool_page_size,
+                                    p.pool_num_pages, p.nk, head, pos / p.pool);
+  if (entry < 0) {
+    if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
+    return;
+  }
+  T* dst = reinterpret_cast<T*>(is_v ? p.pv_pool : p.pk_pool) + entry * width;
+  for (int d0 = 0; d0 < width; d0 += 128) {      // up to four sizes a lane at a time
+    float sum[4] = {0.f, 0.f, 0.f, 0.f};
+    for (int at = pos - p.pool + 1; at <= pos; ++at) {
+      const long long row = paged_row(table, p.table_width, p.page_size, p.num_pages, p.nk, head, at);
+      if (row < 0) {
+        if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
+        return;
+      }
+#pragma unroll
+      for (int i = 0; i < 4; ++i) {
+        const int d = d0 + lane + 32 * i;
+        if (d < width) sum[i] += to_f32<T>(rows[row * width + d]);
+      }
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const int d = d0 + lane + 32 * i;
+      if (d < width) dst[d] = from_f32<T>(sum[i] / (float)p.pool);
+    }
+  }
+}
+
+// For steps in which a request brings several tokens: after qkv_prepare has stored them, a warp per (token, key or value
+// head) stores the mean of the block that ends at the token, if one does.
+template <typename T>
+__global__ void store_block_means_kernel(const PrepParams p) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = blockIdx.x, head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  if (head >= 2 * p.nk) return;
+  const int req = p.req_of_token[n];
+  if (req < 0) return;
+  const int pos = p.positions[n];
+  if ((pos + 1) % p.pool) return;
+  store_block_mean<T>(p, req, pos, head >= p.nk ? head - p.nk : head, head >= p.nk, threadIdx.x & 31);
+}
+
+// Sum over the block of the squares of `count` values (plus a bias) of a row.
+template <typename T>
+__device__ __forceinline__ float row_squares(const T* row, const T* bias, int count, float* scratch) {
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < count; c += blockDim.x) {
+    float x = to_f32<T>(row[c]);
+    if (bias) x += to_f32<T>(bias[c]);
+    ss = __fmaf_rn(x, x, ss);
+  }
+  return block_sum(ss, scratch);
+}
+
+// One warp per (token, head): heads [0, nq) are queries, [nq, nq + nk) keys, [nq + nk, nq + 2 nk) values.  A warp goes on
+// to further heads of its token where the grid has fewer warps than heads.
 template <typename T, typename TO>
 __global__ void qkv_prepare_kernel(const PrepParams p) {
   extern __shared__ float xs_all[];           // a row of `width_max` floats per warp
+  __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
-  const int n = blockIdx.x, head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
-  if (head >= p.nq + 2 * p.nk) return;
+  const int n = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   float* xs = xs_all + (size_t)(threadIdx.x >> 5) * (p.dim > p.vdim ? p.dim : p.vdim);
   const int req = p.req_of_token[n];
   if (req < 0) return;
   const int pos = p.positions[n];
-  const bool is_q = head < p.nq, is_v = head >= p.nq + p.nk;
-  const int hh = is_q ? head : (is_v ? head - p.nq - p.nk : head - p.nq);
-  const int width = is_v ? p.vdim : p.dim;
-  const T* src = reinterpret_cast<const T*>(p.src) + (size_t)n * p.src_stride + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) +
-                 (size_t)hh * width;
-  const T* bias = reinterpret_cast<const T*>(is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias));
-  TO* dst;
-  if (is_q) {
-    dst = reinterpret_cast<TO*>(p.q_out) + (size_t)n * p.q_out_stride + (size_t)hh * width;
-  } else if (p.k_pool != nullptr) {
-    const int page_idx = pos / p.page_size;
-    const int page = page_idx < p.table_width ? p.block_table[(size_t)req * p.table_width + page_idx] : -1;
-    if (page < 0 || page >= p.num_pages) {
-      if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
-      return;
+  const T* row = reinterpret_cast<const T*>(p.src) + (size_t)n * p.src_stride;
+  float all_q = 1.f, all_k = 1.f;             // norm over all heads: 1 / root mean square of the whole of q and of k
+  if (p.norm_all) {
+    if (p.q_norm) all_q = 1.0f / sqrtf(row_squares(row + p.q_off, reinterpret_cast<const T*>(p.q_bias), p.nq * p.dim, scratch) /
+                                           (float)(p.nq * p.dim) + p.norm_eps);
+    if (p.k_norm) all_k = 1.0f / sqrtf(row_squares(row + p.k_off, reinterpret_cast<const T*>(p.k_bias), p.nk * p.dim, scratch) /
+                                           (float)(p.nk * p.dim) + p.norm_eps);
+  }
+  for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < p.nq + 2 * p.nk; head += gridDim.y * warps) {
+    const bool is_q = head < p.nq, is_v = head >= p.nq + p.nk;
+    const int hh = is_q ? head : (is_v ? head - p.nq - p.nk : head - p.nq);
+    const int width = is_v ? p.vdim : p.dim;
+    const T* src = row + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + (size_t)hh * width;
+    const T* bias = reinterpret_cast<const T*>(is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias));
+    TO* dst;
+    if (is_q) {
+      dst = reinterpret_cast<TO*>(p.q_out) + (size_t)n * p.q_out_stride + (size_t)hh * width;
+    } else if (p.k_pool != nullptr) {
+      const long long at = paged_row(p.block_table + (size_t)req * p.table_width, p.table_width, p.page_size, p.num_pages, p.nk,
+                                     hh, pos);
+      if (at < 0) {
+        if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
+        continue;
+      }
+      dst = reinterpret_cast<TO*>(is_v ? p.v_pool : p.k_pool) + at * width;
+    } else {
+      if (p.k_out == nullptr) continue;            // nothing keeps this layer's keys and values: queries only
+      dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
+                 : reinterpret_cast<TO*>(p.k_out) + (size_t)n * p.k_out_stride + (size_t)hh * width;
     }
-    dst = reinterpret_cast<TO*>(is_v ? p.v_pool : p.k_pool) +
-          (((size_t)page * p.nk + hh) * p.page_size + (pos - page_idx * p.page_size)) * width;
-  } else {
-    if (p.k_out == nullptr) return;              // nothing keeps this layer's keys and values: queries only
-    dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
-               : reinterpret_cast<TO*>(p.k_out) + (size_t)n * p.k_out_stride + (size_t)hh * width;
+    __syncwarp();                                  // the warp is done with the row of its last head
+    float ss = 0.f;
+    for (int d = lane; d < width; d += 32) {
+      float x = to_f32<T>(src[d]);
+      if (bias) x += to_f32<T>(bias[(size_t)hh * width + d]);
+      xs[d] = x;
+      ss = __fmaf_rn(x, x, ss);
+    }
+    if (is_v) {
+      for (int d = lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d]);
+    } else {
+      const float* nw = is_q ? p.q_norm : p.k_norm;
+      if (nw && p.norm_all) {
+        const float r = is_q ? all_q : all_k;
+        for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[(size_t)hh * width + d];
+      } else if (nw) {
+        ss = warp_sum(ss);
+        const float r = 1.0f / sqrtf(ss / (float)width + p.norm_eps);
+        for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[d];
+      }
+      __syncwarp();
+      float factor = is_q ? p.q_scale : p.k_scale;
+      if (is_q && p.q_temp_every > 0) factor *= 1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1));
+      const int half = p.inv_freq ? p.rot_dims >> 1 : 0;
+      for (int i = lane; i < half; i += 32) {
+        float sn, cs, o1, o2;
+        sincosf((float)pos * p.inv_freq[i], &sn, &cs);
+        const int a = p.rot_interleaved ? 2 * i : i, b = p.rot_interleaved ? 2 * i + 1 : i + half;
+        rotate_pair(xs[a], xs[b], cs * p.rot_scale, sn * p.rot_scale, o1, o2);
+        dst[a] = from_f32<TO>(o1 * factor);
+        dst[b] = from_f32<TO>(o2 * factor);
+      }
+      for (int d = 2 * half + lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d] * factor);
+    }
+    if (p.pool > 0 && !is_q && (pos + 1) % p.pool == 0) {
+      __syncwarp();                                // the row that this warp has just stored ends a block
+      store_block_mean<TO>(p, req, pos, hh, is_v, lane);
+    }
   }
-  float ss = 0.f;
-  for (int d = lane; d < width; d += 32) {
-    float x = to_f32<T>(src[d]);
-    if (bias) x += to_f32<T>(bias[(size_t)hh * width + d]);
-    xs[d] = x;
-    ss = __fmaf_rn(x, x, ss);
-  }
-  if (is_v) {
-    for (int d = lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d]);
-    return;
-  }
-  const float* nw = is_q ? p.q_norm : p.k_norm;
-  if (nw) {
-    ss = warp_sum(ss);
-    const float r = 1.0f / sqrtf(ss / (float)width + p.norm_eps);
-    for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[d];
-  }
-  __syncwarp();
-  float factor = is_q ? p.q_scale : p.k_scale;
-  if (is_q && p.q_temp_every > 0) factor *= 1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1));
-  const int half = p.inv_freq ? p.rot_dims >> 1 : 0;
-  for (int i = lane; i < half; i += 32) {
-    float sn, cs, o1, o2;
-    sincosf((float)pos * p.inv_freq[i], &sn, &cs);
-    const int a = p.rot_interleaved ? 2 * i : i, b = p.rot_interleaved ? 2 * i + 1 : i + half;
-    rotate_pair(xs[a], xs[b], cs, sn, o1, o2);
-    dst[a] = from_f32<TO>(o1 * factor);
-    dst[b] = from_f32<TO>(o2 * factor);
-  }
-  for (int d = 2 * half + lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d] * factor);
 }
 
 // ACT: 0 gelu with erf, 1 gelu with tanh, 2 silu, 3 the square of relu, 4 tanh.
+// With `bias` (float32, one per column) it is added to x first.
 template <typename T>
 __global__ void activation_kernel(const T* __restrict__ x, int x_stride, T* __restrict__ y, int y_stride, int rows,
-                                  int cols, int act) {
+                                  int cols, int act, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   const size_t total = (size_t)rows * cols;
   for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
     const size_t r = e / cols, c = e - r * cols;
-    const float z = to_f32<T>(x[r * x_stride + c]);
+    float z = to_f32<T>(x[r * x_stride + c]);
+    if (bias) z += bias[c];
     float o;
     if (act == 0) o = 0.5f * z * (1.0f + erff(z * 0.70710678118654752440f));
     else if (act == 1) o = 0.5f * z * (1.0f + tanhf(0.79788456080286535588f * (z + 0.044715f * z * z * z)));
@@ -128,7 +224,7 @@ __device__ __forceinline__ float act_value(float z, int act) {
 }
 
 __global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ x, int x_stride, __nv_bfloat16* __restrict__ y,
-                                         int y_stride, int cols, int act) {
+                                         int y_stride, int cols, int act, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
   const int c = (blockIdx.x * blockDim.x + threadIdx.x) * 8;
@@ -138,7 +234,12 @@ __global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ x, in
   __nv_bfloat162* h = reinterpret_cast<__nv_bfloat162*>(&raw);
 #pragma unroll
   for (int i = 0; i < 4; ++i) {
-    const float2 z = __bfloat1622float2(h[i]);
+    float2 z = __bfloat1622float2(h[i]);
+    if (bias) {
+      const float2 b = *reinterpret_cast<const float2*>(bias + c + 2 * i);
+      z.x += b.x;
+      z.y += b.y;
+    }
     h[i] = __floats2bfloat162_rn(act_value(z.x, act), act_value(z.y, act));
   }
   *reinterpret_cast<uint4*>(y + r * y_stride + c) = raw;
@@ -216,17 +317,23 @@ __global__ void add_rows_vector_kernel(float* __restrict__ x, const float* __res
 
 }  // namespace
 
+// pool > 0: the means of blocks of `pool` keys and values go to pk_pool / pv_pool.  With single_tokens (no request brings
+// more than one token) the warp that stores a block's last row does it; otherwise a second kernel does, once all rows of
+// the step are stored.
 // out_dtype: the dtype of q_out and of the plain k_out / v_out (pools always have the model dtype `dtype`).
 YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int q_off, int k_off, int v_off,
                                 const void* q_bias, const void* k_bias, const void* v_bias, const float* q_norm,
                                 const float* k_norm, float norm_eps, const float* inv_freq, int rot_dims,
-                                int rot_interleaved, float q_scale, float k_scale, float q_temp_coef, int q_temp_every,
+                                int rot_interleaved, float rot_scale, int norm_all, float q_scale, float k_scale, float q_temp_coef, int q_temp_every,
                                 void* q_out, int q_out_stride, void* k_out, int k_out_stride, void* v_out,
                                 int v_out_stride, int out_dtype, void* k_pool, void* v_pool,
                                 const int32_t* block_table, int table_width, int page_size, int num_pages,
                                 const int32_t* positions, const int32_t* req_of_token, int n_tokens, int nq, int nk,
-                                int dim, int vdim, int32_t* bad_page, cudaStream_t stream) {
+                                int dim, int vdim, int32_t* bad_page, int pool, void* pk_pool, void* pv_pool,
+                                const int32_t* pool_table, int pool_table_width, int pool_page_size, int pool_num_pages,
+                                int single_tokens, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
+  if (pool < 0 || (pool > 0 && (!k_pool || !pk_pool || !pv_pool || !pool_table || pool_page_size < 1))) return YALIS_ERR_SHAPE;
   if (dim <= 0 || dim > kMaxHeadDim || vdim <= 0 || vdim > kMaxHeadDim || nq <= 0 || nk <= 0 || nq + 2 * nk > 65535)
     return YALIS_ERR_SHAPE;
   if (inv_freq && (rot_dims <= 0 || (rot_dims & 1) || rot_dims > dim)) return YALIS_ERR_SHAPE;
@@ -234,37 +341,50 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   PrepParams p;
   p.src = src; p.src_stride = src_stride; p.q_off = q_off; p.k_off = k_off; p.v_off = v_off;
   p.q_bias = q_bias; p.k_bias = k_bias; p.v_bias = v_bias; p.q_norm = q_norm; p.k_norm = k_norm; p.norm_eps = norm_eps;
-  p.inv_freq = inv_freq; p.rot_dims = rot_dims; p.rot_interleaved = rot_interleaved; p.q_scale = q_scale; p.k_scale = k_scale;
+  p.inv_freq = inv_freq; p.rot_dims = rot_dims; p.rot_interleaved = rot_interleaved;
+  p.rot_scale = rot_scale; p.norm_all = norm_all; p.q_scale = q_scale; p.k_scale = k_scale;
   p.q_temp_coef = q_temp_coef; p.q_temp_every = q_temp_every;
   p.q_out = q_out; p.q_out_stride = q_out_stride; p.k_out = k_out; p.k_out_stride = k_out_stride;
   p.v_out = v_out; p.v_out_stride = v_out_stride; p.k_pool = k_pool; p.v_pool = v_pool; p.block_table = block_table;
   p.table_width = table_width; p.page_size = page_size; p.num_pages = num_pages; p.positions = positions;
   p.req_of_token = req_of_token; p.nq = nq; p.nk = nk; p.dim = dim; p.vdim = vdim; p.bad_page = bad_page;
+  p.pool = single_tokens ? pool : 0;
+  p.pk_pool = pk_pool; p.pv_pool = pv_pool; p.pool_table = pool_table; p.pool_table_width = pool_table_width;
+  p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
   const int warps = 4;
-  const dim3 grid(n_tokens, (nq + 2 * nk + warps - 1) / warps);
+  // a norm over all heads is summed by every block anew: with tokens enough to fill the GPU one block walks all heads
+  const int by = norm_all && n_tokens >= 2 * yalis_sm_count() ? 1 : (nq + 2 * nk + warps - 1) / warps;
+  const dim3 grid(n_tokens, by);
   const size_t smem = (size_t)warps * (dim > vdim ? dim : vdim) * sizeof(float);
+  int st;
   if (dtype == YALIS_F32 && out_dtype == YALIS_F32)
-    return yalis_launch(qkv_prepare_kernel<float, float>, grid, dim3(32 * warps), smem, stream, p);
-  if (dtype == YALIS_BF16 && out_dtype == YALIS_BF16)
-    return yalis_launch(qkv_prepare_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(32 * warps), smem, stream, p);
-  if (dtype == YALIS_BF16 && out_dtype == YALIS_F32)
-    return yalis_launch(qkv_prepare_kernel<__nv_bfloat16, float>, grid, dim3(32 * warps), smem, stream, p);
-  return YALIS_ERR_DTYPE;
+    st = yalis_launch(qkv_prepare_kernel<float, float>, grid, dim3(32 * warps), smem, stream, p);
+  else if (dtype == YALIS_BF16 && out_dtype == YALIS_BF16)
+    st = yalis_launch(qkv_prepare_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(32 * warps), smem, stream, p);
+  else if (dtype == YALIS_BF16 && out_dtype == YALIS_F32)
+    st = yalis_launch(qkv_prepare_kernel<__nv_bfloat16, float>, grid, dim3(32 * warps), smem, stream, p);
+  else
+    return YALIS_ERR_DTYPE;
+  if (st != YALIS_OK || pool == 0 || single_tokens) return st;
+  p.pool = pool;
+  const dim3 means(n_tokens, (2 * nk + warps - 1) / warps);
+  YALIS_DISPATCH_DTYPE(dtype, T, return yalis_launch(store_block_means_kernel<T>, means, dim3(32 * warps), 0, stream, p));
+  return YALIS_OK;
 }
 
 YALIS_API int yalis_activation(const void* x, int x_stride, void* y, int y_stride, int dtype, int rows, int cols,
-                               int act, cudaStream_t stream) {
+                               int act, const float* bias, cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return YALIS_OK;
   if (act < 0 || act > 4) return YALIS_ERR_SHAPE;
   const size_t total = (size_t)rows * cols;
   const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
   if (dtype == YALIS_BF16 && cols % 8 == 0 && x_stride % 8 == 0 && y_stride % 8 == 0 && !((uintptr_t)x & 15) &&
-      !((uintptr_t)y & 15) && rows <= 65535)
+      !((uintptr_t)y & 15) && !((uintptr_t)bias & 7) && rows <= 65535)
     return yalis_launch(activation_bf16x8_kernel, dim3((cols / 8 + 127) / 128, rows), dim3(128), 0, stream,
-                        (const __nv_bfloat16*)x, x_stride, (__nv_bfloat16*)y, y_stride, cols, act);
+                        (const __nv_bfloat16*)x, x_stride, (__nv_bfloat16*)y, y_stride, cols, act, bias);
   YALIS_DISPATCH_DTYPE(dtype, T,
                        return yalis_launch(activation_kernel<T>, dim3(blocks), dim3(256), 0, stream, (const T*)x, x_stride,
-                                           (T*)y, y_stride, rows, cols, act));
+                                           (T*)y, y_stride, rows, cols, act, bias));
   return YALIS_OK;
 }
 

@@ -6,6 +6,10 @@
 //   S <- S + k_t u^T
 //   o_t = S^T q_t                         (the read-out sees the token's own write)
 //
+// the selective form, with a step size in front of the write and the token's own value beside the read-out,
+//
+//   S <- g_t S + k_t (beta_t v_t)^T,   o_t = S^T q_t + D v_t
+//
 // and the generalized delta rule, whose decay and removal both read the OLD state,
 //
 //   S <- diag(g_t) S - (a_t * u_t)(u_t^T S) + k_t v_t^T,   o_t = S^T q_t
@@ -34,7 +38,8 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 // With kv_heads > 0 the first 2 * kv_heads * dim channels are the heads of q and then of k: each head is
 // brought to unit length, x / sqrt(sum x^2 + eps), and q multiplied by q_scale.  With a_raw the decay
 // g = exp(-exp(a_log[h]) * softplus(a_raw + dt_bias)) (per head, or per head and key channel) and the write
-// strength beta = sigmoid(b_raw) are computed beside it, in float32.
+// strength are computed beside it, in float32: beta = sigmoid(b_raw), or without b_raw (one column of a_raw per
+// head) the step size itself, beta = softplus(a_raw + dt_bias).  With conv_bias y_t[c] = silu(conv_bias[c] + ...).
 constexpr int kMaxTaps = 16;
 
 template <typename T>
@@ -46,7 +51,7 @@ __global__ void delta_prepare_kernel(const T* __restrict__ x, int x_stride, cons
                                      const T* __restrict__ a_raw, int a_stride, int a_cols,
                                      const float* __restrict__ a_log, const float* __restrict__ dt_bias,
                                      const T* __restrict__ b_raw, int b_stride, int heads, float* __restrict__ g_out,
-                                     float* __restrict__ beta_out) {
+                                     float* __restrict__ beta_out, const float* __restrict__ conv_bias) {
   pdl_launch_dependents();
   pdl_wait();
   const int n = blockIdx.x;
@@ -63,15 +68,16 @@ __global__ void delta_prepare_kernel(const T* __restrict__ x, int x_stride, cons
       else xv = tl[(size_t)c * (taps - 1) + (taps - 1 + i - j)];
       acc = __fmaf_rn(w[(size_t)c * taps + (taps - 1 - j)], xv, acc);
     }
-    row[c] = silu_exact(acc);
+    row[c] = silu_exact(conv_bias ? acc + conv_bias[c] : acc);
   }
   if (a_raw != nullptr) {
     const int per = a_cols / heads;               // 1, or dim
     for (int c = threadIdx.x; c < a_cols; c += blockDim.x) {
-      const float a = to_f32<T>(a_raw[(size_t)n * a_stride + c]) + dt_bias[c];
-      g_out[(size_t)n * a_cols + c] = expf(-expf(a_log[c / per]) * softplus_f(a));
+      const float step = softplus_f(to_f32<T>(a_raw[(size_t)n * a_stride + c]) + dt_bias[c]);
+      g_out[(size_t)n * a_cols + c] = expf(-expf(a_log[c / per]) * step);
+      if (b_raw == nullptr) beta_out[(size_t)n * heads + c] = step;
     }
-    for (int h = threadIdx.x; h < heads; h += blockDim.x)
+    for (int h = threadIdx.x; b_raw != nullptr && h < heads; h += blockDim.x)
       beta_out[(size_t)n * heads + h] = sigmoid_f(to_f32<T>(b_raw[(size_t)n * b_stride + h]));
   }
   if (kv_heads > 0) {
@@ -124,7 +130,8 @@ struct ScanParams {
   const float* k; int k_stride;
   const float* v; int v_stride;      // [N, heads * vdim]
   const float* decay;                // DECAY 0: [heads]; 1: [N, heads]; 2: [N, heads * dim]
-  const float* beta;                 // RULE 1: [N, heads]
+  const float* beta;                 // RULE 1, 3: [N, heads]
+  const float* skip;                 // RULE 3: [heads] or null: skip_h v_t is added to the read-out
   const float* unit;                 // RULE 2: unit keys u [N, heads * dim]
   const float* removal;              // RULE 2: a * u [N, heads * dim]
   float* state; size_t slot_stride;  // per slot: [heads][vdim][dim_padded]
@@ -144,7 +151,8 @@ __device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.com
 template <int N>
 __device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group %0;\n" ::"n"(N)); }
 
-// RULE: 0 plain outer-product write, 1 delta rule, 2 generalized delta rule (needs DECAY 2).
+// RULE: 0 plain outer-product write, 1 delta rule, 2 generalized delta rule (needs DECAY 2), 3 plain write of beta v
+// with skip_h v beside the read-out.
 // DECAY: 0 constant per head, 1 scalar per token and head, 2 vector per token, head and key channel.
 // ROWS: rows of a column that a thread keeps (8: twice the warps, which hide each other's waits; 16: dim up to 512).
 // The tokens of a request are staged through two buffers in shared memory: while one tile is walked, the
@@ -226,7 +234,7 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const ScanPara
     }
     if (tid < tt) {
       const size_t n = (size_t)(t_begin + t0 + tid);
-      if (DELTA) copy_async4(bs + tid, p.beta + n * p.heads + h);
+      if (DELTA || RULE == 3) copy_async4(bs + tid, p.beta + n * p.heads + h);
       if (DECAY == 1) copy_async4(gs + tid, p.decay + n * p.heads + h);
     }
     copy_async_commit();
@@ -242,6 +250,7 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const ScanPara
     S[4 * i] = x.x; S[4 * i + 1] = x.y; S[4 * i + 2] = x.z; S[4 * i + 3] = x.w;
   }
   const float g_const = DECAY == 0 ? p.decay[h] : 1.f;
+  const float skip = (RULE == 3 && p.skip) ? p.skip[h] : 0.f;
 
   issue(0, 0);
   int b = 0;
@@ -335,6 +344,7 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const ScanPara
         for (int o = 1; o < L; o <<= 1) dot += __shfl_xor_sync(0xffffffffu, dot, o);
         u = bs[t] * (u - dot);
       }
+      if (RULE == 3) u *= bs[t];
       float part[ROWS / 2];
 #pragma unroll
       for (int i = 0; i < ROWS / 2; ++i) {
@@ -346,6 +356,9 @@ __global__ void __launch_bounds__(kScanThreads) state_scan_kernel(const ScanPara
       for (int w = ROWS / 4; w >= 1; w >>= 1)
 #pragma unroll
         for (int i = 0; i < w; ++i) part[i] += part[i + w];
+      // (the token's own value joins the first lane's share here: the copies of the next tile may already be
+      // overwriting this one while the shares are added)
+      if (RULE == 3 && l == 0) part[0] = __fmaf_rn(skip, vs[t * cols + c], part[0]);
       shares[(t * cols + c) * (L + 1) + l] = part[0];
     }
     __syncthreads();                // the next round's copies overwrite the other buffer, which the round after reads
@@ -395,6 +408,32 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, int o_stride,
     }
     y[(size_t)n * y_stride + (size_t)h * vdim + d] = from_f32<T>(val * out_scale);
   }
+}
+
+// ---- gate, then norm in equal parts -----------------------------------------------------------------------------
+//   y = o * silu(z);   y[part] <- y / sqrt(mean(y^2 over the part) + eps) * weight * out_scale
+// A block per (token, part); a part waits in shared memory between the two passes.
+template <typename T>
+__global__ void gate_norm_kernel(const float* __restrict__ o, int o_stride, const T* __restrict__ z, int z_stride,
+                                 const float* __restrict__ weight, T* __restrict__ y, int y_stride,
+                                 const int32_t* __restrict__ req_of_token, int width, float eps, float out_scale) {
+  extern __shared__ float part_s[];               // [width]
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int n = blockIdx.x, c0 = blockIdx.y * width;
+  if (req_of_token[n] < 0) return;
+  const float* op = o + (size_t)n * o_stride + c0;
+  const T* zp = z + (size_t)n * z_stride + c0;
+  float ss = 0.f;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) {
+    const float v = op[c] * silu_exact(to_f32<T>(zp[c]));
+    part_s[c] = v;
+    ss = __fmaf_rn(v, v, ss);
+  }
+  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+  T* yp = y + (size_t)n * y_stride + c0;
+  for (int c = threadIdx.x; c < width; c += blockDim.x) yp[c] = from_f32<T>(part_s[c] * r * weight[c0 + c] * out_scale);
 }
 
 // ---- what the generalized delta rule reads ------------------------------------------------------------
@@ -457,6 +496,7 @@ YALIS_API int yalis_general_delta_prepare(const void* q, const void* k, const vo
   return YALIS_OK;
 }
 
+// b_raw null (with a_raw [N, heads]): beta_out receives the step sizes softplus(a_raw + dt_bias).
 // a_raw null: no decay and write strength are computed.  kv_heads 0: no head is brought to unit length.
 YALIS_API int yalis_delta_prepare(const void* x, int dtype, int x_stride, const float* w, float* tail,
                                   int64_t slot_stride, const int32_t* req_of_token, const int32_t* q_start,
@@ -464,17 +504,17 @@ YALIS_API int yalis_delta_prepare(const void* x, int dtype, int x_stride, const 
                                   int channels, int taps, int kv_heads, int dim, float q_scale, float unit_eps,
                                   const void* a_raw, int a_stride, int a_cols, const float* a_log, const float* dt_bias,
                                   const void* b_raw, int b_stride, int heads, float* g_out, float* beta_out,
-                                  cudaStream_t stream) {
+                                  const float* conv_bias, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
   if (taps < 1 || taps > kMaxTaps || channels <= 0 || kv_heads < 0 || 2 * kv_heads * dim > channels) return YALIS_ERR_SHAPE;
-  if (a_raw && (heads <= 0 || a_cols % heads || !a_log || !dt_bias || !b_raw || !g_out || !beta_out)) return YALIS_ERR_SHAPE;
+  if (a_raw && (heads <= 0 || a_cols % heads || !a_log || !dt_bias || (!b_raw && a_cols != heads) || !g_out || !beta_out)) return YALIS_ERR_SHAPE;
   const int by = (channels + 127) / 128;
   const int threads = channels >= 1024 ? 256 : 128;
   YALIS_DISPATCH_DTYPE(dtype, T, {
     int st = yalis_launch(delta_prepare_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (const T*)x, x_stride, w,
                           (const float*)tail, (size_t)slot_stride, req_of_token, q_start, slots, out, out_stride, channels,
                           taps, kv_heads, dim, q_scale, unit_eps, (const T*)a_raw, a_stride, a_cols, a_log, dt_bias,
-                          (const T*)b_raw, b_stride, heads, g_out, beta_out);
+                          (const T*)b_raw, b_stride, heads, g_out, beta_out, conv_bias);
     if (st != YALIS_OK || taps == 1) return st;
     return yalis_launch(short_conv_tail_kernel<T>, dim3(n_requests, by), dim3(128), 0, stream, (const T*)x, x_stride,
                         tail, (size_t)slot_stride, q_start, slots, channels, taps);
@@ -507,6 +547,7 @@ static int launch_scan(const ScanParams& p, dim3 grid, size_t smem, cudaStream_t
 template <int ROWS, int LANES>
 static int launch_scan_kind(const ScanParams& p, dim3 grid, size_t smem, int delta, int decay_kind, cudaStream_t stream) {
   if (delta == 2) return launch_scan<ROWS, LANES, 2, 2>(p, grid, smem, stream);
+  if (delta == 3) return launch_scan<ROWS, LANES, 3, 1>(p, grid, smem, stream);
   if (delta && decay_kind == 1) return launch_scan<ROWS, LANES, 1, 1>(p, grid, smem, stream);
   if (delta && decay_kind == 2) return launch_scan<ROWS, LANES, 1, 2>(p, grid, smem, stream);
   if (delta) return launch_scan<ROWS, LANES, 1, 0>(p, grid, smem, stream);
@@ -517,10 +558,11 @@ static int launch_scan_kind(const ScanParams& p, dim3 grid, size_t smem, int del
 
 // decay_kind 0: decay [heads]; 1: decay [N, heads]; 2: decay [N, heads * dim].  delta 1: the delta rule with beta
 // [N, heads]; delta 2: the generalized delta rule with unit keys and removal vectors [N, heads * dim] (contiguous,
-// kv_heads = heads, decay_kind 2).
+// kv_heads = heads, decay_kind 2); delta 3: the selective form, beta [N, heads] the step sizes and skip [heads] (or null)
+// the token's own value in the read-out (decay_kind 1).
 // max_q_len: the longest portion of the step if the caller knows it (0: not known); it only bounds the staging tile.
 YALIS_API int yalis_state_scan(const float* q, int q_stride, const float* k, int k_stride, const float* v, int v_stride,
-                               const float* decay, int decay_kind, const float* beta, const float* unit,
+                               const float* decay, int decay_kind, const float* beta, const float* skip, const float* unit,
                                const float* removal, float* state, int64_t slot_stride,
                                float* out, int out_stride, const int32_t* q_start, const int32_t* slots, int n_requests,
                                int heads, int kv_heads, int dim, int vdim, int delta, int max_q_len, cudaStream_t stream) {
@@ -529,7 +571,8 @@ YALIS_API int yalis_state_scan(const float* q, int q_stride, const float* k, int
     return YALIS_ERR_SHAPE;
   const int lanes = yalis_state_scan_lanes(dim);
   if (lanes > 32) return YALIS_ERR_SHAPE;           // dim <= 512
-  if (decay_kind < 0 || decay_kind > 2 || !decay || delta < 0 || delta > 2 || (delta == 1 && !beta)) return YALIS_ERR_SHAPE;
+  if (decay_kind < 0 || decay_kind > 2 || !decay || delta < 0 || delta > 3 || (delta == 1 && !beta)) return YALIS_ERR_SHAPE;
+  if (delta == 3 && (decay_kind != 1 || !beta)) return YALIS_ERR_SHAPE;
   if (delta == 2 && (decay_kind != 2 || !unit || !removal || kv_heads != heads)) return YALIS_ERR_SHAPE;
   const int dim_padded = (dim + 3) & ~3;
   if ((slot_stride & 3) || ((uintptr_t)state & 15)) return YALIS_ERR_ALIGN;
@@ -541,7 +584,7 @@ YALIS_API int yalis_state_scan(const float* q, int q_stride, const float* k, int
   if (max_q_len > 0 && tile > max_q_len) tile = max_q_len;      // single tokens: small blocks, many of them per SM
   ScanParams p;
   p.q = q; p.q_stride = q_stride; p.k = k; p.k_stride = k_stride; p.v = v; p.v_stride = v_stride;
-  p.decay = decay; p.beta = beta; p.unit = unit; p.removal = removal; p.state = state; p.slot_stride = (size_t)slot_stride; p.out = out;
+  p.decay = decay; p.beta = beta; p.skip = skip; p.unit = unit; p.removal = removal; p.state = state; p.slot_stride = (size_t)slot_stride; p.out = out;
   p.out_stride = out_stride; p.q_start = q_start; p.slots = slots; p.heads = heads; p.kv_heads = kv_heads;
   p.dim = dim; p.dim_padded = dim_padded; p.vdim = vdim; p.lanes = lanes; p.tile = tile;
   p.wide = (dim % 4 == 0 && q_stride % 4 == 0 && k_stride % 4 == 0 && !((uintptr_t)q & 15) && !((uintptr_t)k & 15) &&
@@ -572,5 +615,24 @@ YALIS_API int yalis_head_norm_gate(const float* o, int o_stride, const float* we
                                            dim3(32 * warps), 0, stream, o, o_stride, weight, (const T*)gate, gate_stride,
                                            gate_kind, (T*)y, y_stride, req_of_token, heads, vdim, eps, out_scale,
                                            weight_per_head ? vdim : 0));
+  return YALIS_OK;
+}
+
+// o float32 [N, parts * width]; z (model dtype) the gate's input; weight float32 [parts * width]; y in the model dtype.
+YALIS_API int yalis_gate_norm(const float* o, int o_stride, const void* z, int z_stride, const float* weight, void* y,
+                              int y_stride, int dtype, const int32_t* req_of_token, int n_tokens, int parts, int width,
+                              float eps, float out_scale, cudaStream_t stream) {
+  if (n_tokens <= 0) return YALIS_OK;
+  if (parts <= 0 || parts > 65535 || width <= 0) return YALIS_ERR_SHAPE;
+  const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
+  const size_t smem = (size_t)width * sizeof(float);
+  if (smem > 200 * 1024) return YALIS_ERR_SHAPE;
+  YALIS_DISPATCH_DTYPE(dtype, T, {
+    if (smem > 48 * 1024 &&
+        cudaFuncSetAttribute(gate_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+      return YALIS_ERR_LAUNCH;
+    return yalis_launch(gate_norm_kernel<T>, dim3(n_tokens, parts), dim3(threads), smem, stream, o, o_stride, (const T*)z, z_stride,
+                        weight, (T*)y, y_stride, req_of_token, width, eps, out_scale);
+  });
   return YALIS_OK;
 }

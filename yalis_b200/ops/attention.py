@@ -6,6 +6,7 @@ import collections
 import ctypes
 import math
 import os
+from dataclasses import dataclass
 from typing import Optional
 
 import numpy as np
@@ -42,7 +43,8 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
                             v_head_dim: Optional[int] = None, softcap: Optional[float] = None, sink: bool = False,
                             out_scale: float = 1.0, chunk: Optional[int] = None,
                             sink_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                            gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                            gate: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None,
+                            pool: Optional["PooledBlocks"] = None) -> torch.Tensor:
     """Exact attention of every token over the cached keys of its request.
 
     ``q`` may be the fused qkv matrix (only its first heads*head_dim columns are
@@ -50,7 +52,9 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
     p - window < j <= p, and with ``chunk`` C only j >= floor(p / C) * C.  ``slopes`` (float32 [heads]) take
     slope_h * (p - j) off the scaled score.  ``softcap`` c turns a score s into c * tanh(s / c); ``sink``
     adds exp(z_h) to the softmax's denominator (a key of score z_h that has no value; z = ``sink_logits`` float32
-    [heads], 0 without them); ``gate`` [N, heads * v_head_dim] multiplies the result by its sigmoid;
+    [heads], 0 without them); ``gate`` [N, heads * v_head_dim], or [N, heads] for one number per head, multiplies the
+    result by its sigmoid; ``rel`` (float32 [heads, L]) adds rel[h, min(p - j, L - 1)] to the scaled score; ``pool``
+    (with a window) lets p see, beside its window, the pooled blocks that lie wholly before it (``PooledBlocks``);
     ``v_head_dim`` is the head size of the values when it is not the keys'.  The result,
     times ``out_scale``, is [N, heads*v_head_dim] in q's dtype (``out`` may be a
     column block of a wider matrix).
@@ -65,7 +69,8 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
         out = torch.empty((n, num_heads * vd), dtype=q.dtype, device=q.device)
     need(out.shape == (n, num_heads * vd) and out.dtype == q.dtype and out.stride(1) == 1, name, "bad out tensor")
     need(softcap is None or softcap > 0, name, "the soft cap must be positive")
-    _check_extras(name, q, num_heads, vd, chunk, sink, sink_logits, slopes, gate)
+    _check_extras(name, q, num_heads, vd, chunk, sink, sink_logits, slopes, gate, rel)
+    pooled = _pool_arguments(name, pool, k_pool, v_pool, window, chunk)
     if scale is None:
         scale = 1.0 / math.sqrt(head_dim)
     check(lib().yalis_paged_attention_generic(
@@ -73,19 +78,55 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
         ptr(positions), ptr(req_of_token), ptr(block_table), i32(block_table.shape[1]), i32(k_pool.shape[2]),
         i32(k_pool.shape[0]), i32(n), i32(num_heads), i32(num_kv_heads), i32(head_dim), i32(vd), f32(scale),
         i32(window or 0), f32(softcap or 0.0), i32(int(sink)), f32(out_scale), i32(chunk or 0), ptr(sink_logits), ptr(slopes),
-        ptr(gate), i32(gate.stride(0) if gate is not None else 0), stream()), name)
+        ptr(gate), i32(gate.stride(0) if gate is not None else 0), i32(_per_head(gate, num_heads, vd)), ptr(rel),
+        i32(rel.shape[1] if rel is not None else 0), *pooled, stream()), name)
     return out
 
 
-def _check_extras(name, q, num_heads, vd, chunk, sink, sink_logits, slopes, gate):
-    need_cuda(name, sink_logits, slopes, gate)
+@dataclass(frozen=True)
+class PooledBlocks:
+    """One mean key and mean value per block of ``size`` consecutive positions, in pages of their own: ``k``
+    [pages, kv_heads, entries, head_dim], ``v`` [.., v_head_dim], ``table`` int32 [R, width] (page of entry b at column
+    b // entries).  A query at position p with a window W sees block b if its last position, b * size + size - 1, is at
+    most p - W; blocks and the window's keys share one softmax."""
+
+    size: int
+    k: torch.Tensor
+    v: torch.Tensor
+    table: torch.Tensor
+
+
+def _pool_arguments(name, pool: Optional[PooledBlocks], k_pool, v_pool, window, chunk):
+    if pool is None:
+        return i32(0), ptr(None), ptr(None), ptr(None), i32(0), i32(0), i32(0)
+    need_cuda(name, pool.k, pool.v, pool.table)
+    need(pool.size > 0 and window is not None and chunk is None, name, "pooled blocks come with a window and without chunks")
+    need(pool.k.dim() == pool.v.dim() == 4 and pool.k.shape[:3] == pool.v.shape[:3] and pool.k.shape[1] == k_pool.shape[1]
+         and pool.k.shape[3] == k_pool.shape[3] and pool.v.shape[3] == v_pool.shape[3] and pool.k.is_contiguous()
+         and pool.v.is_contiguous() and pool.k.dtype == pool.v.dtype == k_pool.dtype, name,
+         "pools of blocks must be contiguous [pages, kv_heads, entries, head size] like the pools of keys and values")
+    need(pool.table.dtype == torch.int32 and pool.table.dim() == 2 and pool.table.is_contiguous(), name,
+         "the blocks' table must be contiguous int32 [R, width]")
+    return (i32(pool.size), ptr(pool.k), ptr(pool.v), ptr(pool.table), i32(pool.table.shape[1]), i32(pool.k.shape[2]),
+            i32(pool.k.shape[0]))
+
+
+def _per_head(gate, num_heads: int, vd: int) -> int:
+    return int(gate is not None and gate.shape[1] == num_heads and vd != 1)
+
+
+def _check_extras(name, q, num_heads, vd, chunk, sink, sink_logits, slopes, gate, rel):
+    need_cuda(name, sink_logits, slopes, gate, rel)
+    need(rel is None or (rel.dtype == torch.float32 and rel.dim() == 2 and rel.shape[0] == num_heads and rel.shape[1] >= 1
+                         and rel.is_contiguous()), name, "the bias per distance must be contiguous float32 [heads, L]")
     need(chunk is None or chunk > 0, name, "the chunk size must be positive")
     need(sink_logits is None or sink, name, "sink scores come with a sink")
     for v in (sink_logits, slopes):
         need(v is None or (v.dtype == torch.float32 and v.shape == (num_heads,) and v.is_contiguous()), name,
              "sink scores and slopes must be float32 [heads]")
-    need(gate is None or (gate.dtype == q.dtype and gate.shape == (q.shape[0], num_heads * vd) and gate.stride(1) == 1), name,
-         "the gate must be [N, heads * v_head_dim] in q's dtype with unit inner stride")
+    need(gate is None or (gate.dtype == q.dtype and gate.shape in ((q.shape[0], num_heads * vd), (q.shape[0], num_heads))
+                          and gate.stride(1) == 1), name,
+         "the gate must be [N, heads * v_head_dim] or [N, heads] in q's dtype with unit inner stride")
 
 
 SM_COUNT: Optional[int] = None    # set to override what the device reports (tests pretend a small GPU)
@@ -120,6 +161,12 @@ USE_PREFILL_TCGEN05 = os.environ.get("YALIS_B200_NO_PREFILL_TCGEN05", "0") != "1
 def mma_supports(head_dim: int) -> bool:
     """Whether the tensor-core kernel is built for this head size (multiples of 16 up to 128, of 32 up to 256)."""
     return bool(lib().yalis_attention_mma_supports(i32(head_dim)))
+
+
+def mma_extended_supports(head_dim: int, v_head_dim: int) -> bool:
+    """Whether the extended form of the tensor-core kernel (a value size of its own, a bias per distance, pooled blocks)
+    takes these sizes: multiples of 8 up to 256."""
+    return bool(lib().yalis_attention_mma_extended_supports(i32(head_dim), i32(v_head_dim)))
 
 
 def decode_splits(n_requests: int, num_kv_heads: int) -> int:
@@ -185,7 +232,8 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
                         out: Optional[torch.Tensor] = None, softcap: Optional[float] = None, sink: bool = False,
                         out_scale: float = 1.0, exact_weights: bool = False, chunk: Optional[int] = None,
                         sink_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
-                        gate: Optional[torch.Tensor] = None) -> torch.Tensor:
+                        gate: Optional[torch.Tensor] = None, v_head_dim: Optional[int] = None,
+                        rel: Optional[torch.Tensor] = None, pool: Optional[PooledBlocks] = None) -> torch.Tensor:
     """Tensor-core attention (bfloat16) of the step's tokens over the cache; the same
     semantics as ``paged_attention_generic``.  ``q_start`` int32 [R+1] gives each request's
     token range; ``max_q_len`` bounds the launch grid.  ``n_splits`` > 1 divides the keys of
@@ -193,22 +241,28 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
     ``softcap``, ``sink``, ``out_scale``, ``chunk``, ``sink_logits``, ``slopes`` and ``gate`` as in
     ``paged_attention_generic``; with any of them, or with
     ``exact_weights``, the softmax weights meet the values with 16 bits of mantissa (in two bfloat16 halves)
-    instead of 8.  ``out`` may be a column block of a wider matrix if it starts on a 16-byte boundary.
+    instead of 8.  ``v_head_dim``, ``rel`` and ``pool`` as there too; they, and head sizes the other forms are not built
+    for, take the kernel's extended form.  ``out`` may be a column block of a wider matrix if it starts on a 16-byte
+    boundary.
     """
     name = "paged_attention_mma"
     LAUNCHED["mma"] += 1
-    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads, head_dim)
+    vd = head_dim if v_head_dim is None else int(v_head_dim)
+    extended = vd != head_dim or rel is not None or pool is not None or not mma_supports(head_dim)
+    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads, head_dim, vd)
     need(q.dtype == torch.bfloat16, name, "bfloat16 only (float32 goes to the generic kernel)")
-    need(mma_supports(head_dim), name, f"head_dim {head_dim} is not built (multiples of 16 to 128, of 32 to 256)")
+    need(mma_extended_supports(head_dim, vd) if extended else mma_supports(head_dim), name,
+         f"head sizes {head_dim}, {vd} are not built (equal: multiples of 16 to 128, of 32 to 256; extended form: of 8 to 256)")
     n, r = q.shape[0], q_start.numel() - 1
     need(q_start.dtype == torch.int32 and q_start.is_contiguous() and q_start.is_cuda, name, "q_start must be int32 [R+1]")
     need(block_table.shape[0] >= r, name, "block_table has fewer rows than requests")
     if out is None:
-        out = torch.empty((n, num_heads * head_dim), dtype=q.dtype, device=q.device)
-    need(out.shape == (n, num_heads * head_dim) and out.dtype == q.dtype and out.stride(1) == 1
+        out = torch.empty((n, num_heads * vd), dtype=q.dtype, device=q.device)
+    need(out.shape == (n, num_heads * vd) and out.dtype == q.dtype and out.stride(1) == 1
          and out.stride(0) % 2 == 0 and out.data_ptr() % 16 == 0, name, "bad out tensor")
     need(softcap is None or softcap > 0, name, "the soft cap must be positive")
-    _check_extras(name, q, num_heads, head_dim, chunk, sink, sink_logits, slopes, gate)
+    _check_extras(name, q, num_heads, vd, chunk, sink, sink_logits, slopes, gate, rel)
+    pooled = _pool_arguments(name, pool, k_pool, v_pool, window, chunk)
     if scale is None:
         scale = 1.0 / math.sqrt(head_dim)
     scratch = tickets = None
@@ -216,7 +270,7 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
         need(max_q_len * (num_heads // num_kv_heads) <= 16, name, "splitting the keys is for decode steps only")
         floats = lib().yalis_attention_mma_scratch_floats
         floats.restype = ctypes.c_longlong
-        scratch = torch.empty(int(floats(i32(n), i32(num_heads), i32(head_dim), i32(n_splits))), dtype=torch.float32,
+        scratch = torch.empty(int(floats(i32(n), i32(num_heads), i32(vd), i32(n_splits))), dtype=torch.float32,
                               device=q.device)
         tickets = _tickets(q.device, r * num_kv_heads)
     check(lib().yalis_paged_attention_mma_general(
@@ -225,7 +279,8 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
         i32(n), i32(r), i32(max_q_len), i32(num_heads), i32(num_kv_heads), i32(head_dim), f32(scale), i32(window or 0),
         i32(n_splits), ptr(scratch), ptr(tickets), f32(softcap or 0.0), i32(int(sink)), f32(out_scale),
         i32(int(exact_weights)), i32(chunk or 0), ptr(sink_logits), ptr(slopes), ptr(gate),
-        i32(gate.stride(0) if gate is not None else 0), stream()), name)
+        i32(gate.stride(0) if gate is not None else 0), i32(_per_head(gate, num_heads, vd)), i32(vd), ptr(rel),
+        i32(rel.shape[1] if rel is not None else 0), *pooled, stream()), name)
     return out
 
 

@@ -89,13 +89,25 @@ def add_rmsnorm(x: torch.Tensor, delta: Optional[torch.Tensor], weight: torch.Te
     return out
 
 
+def _result_layout(name: str, y: Optional[torch.Tensor], n: int, width: int):
+    """(parts, stride between them) of a sub-layer's result [N, width] or of its float32 partial sums [S, N, width]."""
+    if y is None:
+        return 0, 0
+    need(y.is_contiguous() and (y.shape == (n, width) or (y.dim() == 3 and y.shape[1:] == (n, width))), name,
+         f"a result must be contiguous [N, width] or partial sums [S, N, width] of {(n, width)}, not {tuple(y.shape)}")
+    return (1, 0) if y.dim() == 2 else (y.shape[0], n * width)
+
+
 def add_normed_rmsnorm(x: torch.Tensor, delta: torch.Tensor, *, bias: Optional[torch.Tensor] = None,
                        delta_norm=None, weight: Optional[torch.Tensor] = None, eps: float = 0.0,
-                       out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                       out_dtype: Optional[torch.dtype] = None, rows: Optional[torch.Tensor] = None,
+                       scale: Optional[torch.Tensor] = None, factor: float = 1.0, second=None) -> Optional[torch.Tensor]:
     """A sub-layer's result that is normed on its way into the stream, and the norm that follows, in one pass:
 
         d = delta (the sum of split partial sums [S, N, width], in order) + bias
         d <- d / sqrt(mean(d^2) + e_d) * w_d          with ``delta_norm`` = (w_d, e_d)
+        d <- d + d2 / sqrt(mean(d2^2) + e_2) * w_2    with ``second`` = (delta2, (w_2, e_2)), delta2 like delta
+        d <- d * factor * scale                       ``scale`` a vector over the width
         x <- x + d;  returns rmsnorm(x) * weight in ``out_dtype``        (nothing without ``weight``)
 
     all float32.  With ``rows`` only those rows are computed and x is left untouched."""
@@ -104,16 +116,13 @@ def add_normed_rmsnorm(x: torch.Tensor, delta: torch.Tensor, *, bias: Optional[t
     need_cuda(name, x, delta, bias, d_w, weight, rows)
     need(x.dtype == torch.float32 and x.dim() == 2 and x.is_contiguous(), name, "x must be contiguous float32 [N, width]")
     n, width = x.shape
-    for v in (bias, d_w, weight):
+    second_y, (s_w, s_eps) = (None, (None, 0.0)) if second is None else second
+    need_cuda(name, scale, second_y, s_w)
+    for v in (bias, d_w, weight, scale, s_w):
         need(v is None or (v.dtype == torch.float32 and v.shape == (width,) and v.is_contiguous()), name,
              "bias and norm weights must be float32 [width]")
-    need(delta.is_contiguous(), name, "delta must be contiguous")
-    if delta.dim() == 2:
-        need(delta.shape == (n, width), name, f"delta shape {tuple(delta.shape)} != {(n, width)}")
-        n_delta, d_stride = 1, 0
-    else:
-        need(delta.dim() == 3 and delta.shape[1:] == (n, width), name, "split delta must be [S, N, width]")
-        n_delta, d_stride = delta.shape[0], n * width
+    (n_delta, d_stride), (n_second, second_stride) = _result_layout(name, delta, n, width), _result_layout(name, second_y, n, width)
+    need(second_y is None or s_w is not None, name, "the second result comes with its norm")
     n_out = n
     if rows is not None:
         need(rows.dtype == torch.int32 and rows.dim() == 1 and rows.is_contiguous(), name, "rows must be int32 [R]")
@@ -125,7 +134,9 @@ def add_normed_rmsnorm(x: torch.Tensor, delta: torch.Tensor, *, bias: Optional[t
     check(lib().yalis_add_normed_rmsnorm(ptr(x), ptr(delta), i32(dtype_code(delta.dtype)), i32(n_delta), i64(d_stride), ptr(bias),
                                          ptr(d_w), f32(d_eps), ptr(weight), ptr(out),
                                          i32(dtype_code(out_dtype if out is not None else torch.float32)), ptr(rows), i32(n_out),
-                                         i32(width), f32(eps), i32(0 if rows is not None else 1), stream()), name)
+                                         i32(width), f32(eps), i32(0 if rows is not None else 1), ptr(scale), f32(factor), ptr(second_y),
+                                         i32(dtype_code(second_y.dtype) if second_y is not None else 0), i32(n_second),
+                                         i64(second_stride), ptr(s_w), f32(s_eps), stream()), name)
     return out
 
 
@@ -240,8 +251,9 @@ ACTIVATIONS = {"gelu": ACT_GELU_ERF, "gelu_erf": ACT_GELU_ERF, "gelu_tanh": ACT_
                "relu2": ACT_RELU2, "tanh": ACT_TANH}
 
 
-def activation(x: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None) -> torch.Tensor:
-    """act(x) element by element in float32: ``gelu_erf`` 0.5 z (1 + erf(z / sqrt 2)), ``gelu_tanh``
+def activation(x: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None,
+               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+    """act(x), or act(x + bias) with ``bias`` float32 [C], element by element in float32: ``gelu_erf`` 0.5 z (1 + erf(z / sqrt 2)), ``gelu_tanh``
     0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), ``silu``, ``relu2`` (max(z, 0)^2) or ``tanh``.  ``x`` and ``out`` are [N, C] with unit inner
     stride (column blocks of wider matrices are fine)."""
     name = "activation"
@@ -251,8 +263,11 @@ def activation(x: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None) -
     if out is None:
         out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
     need(out.shape == x.shape and out.dtype == x.dtype and out.stride(1) == 1, name, "bad out tensor")
+    need_cuda(name, bias)
+    need(bias is None or (bias.dtype == torch.float32 and bias.shape == (x.shape[1],) and bias.is_contiguous()), name,
+         "the bias must be float32 [C]")
     check(lib().yalis_activation(ptr(x), i32(x.stride(0)), ptr(out), i32(out.stride(0)), i32(dtype_code(x.dtype)),
-                                 i32(x.shape[0]), i32(x.shape[1]), i32(ACTIVATIONS[kind]), stream()), name)
+                                 i32(x.shape[0]), i32(x.shape[1]), i32(ACTIVATIONS[kind]), ptr(bias), stream()), name)
     return out
 
 
@@ -274,18 +289,26 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
                 inv_freq: Optional[torch.Tensor] = None, q_scale: float = 1.0, k_scale: float = 1.0,
                 k_pool: Optional[torch.Tensor] = None, v_pool: Optional[torch.Tensor] = None,
                 block_table: Optional[torch.Tensor] = None, store: bool = True,
-                bad_flag: Optional[torch.Tensor] = None, interleaved: bool = False, q_temperature=None):
+                bad_flag: Optional[torch.Tensor] = None, interleaved: bool = False, q_temperature=None,
+                rot_scale: float = 1.0, norm_all: bool = False, pool: int = 0, pooled_k: Optional[torch.Tensor] = None,
+                pooled_v: Optional[torch.Tensor] = None, pooled_table: Optional[torch.Tensor] = None,
+                single_tokens: bool = False):
     """Prepares the heads of a mixer from its input projection ``src`` [N, ...] (model dtype), whose query,
     key and value heads start at the columns ``offsets`` = (q, k, v):
 
         x <- x + bias;  q, k <- x / sqrt(mean(x^2) + norm_eps) * norm (where a norm is given);
+        (with ``norm_all`` the mean is over all heads of q, and of k, at once and the norms are [heads * dim]);
         q, k <- rotation of their first 2 * len(inv_freq) sizes by the angle position * inv_freq (size i paired
-        with i + len(inv_freq); with ``interleaved`` size 2i with 2i + 1), the other sizes unchanged;
+        with i + len(inv_freq); with ``interleaved`` size 2i with 2i + 1), the other sizes unchanged, cosine and sine
+        times ``rot_scale``;
         q <- q * q_scale, k <- k * k_scale;  with ``q_temperature`` = (coef, every) also
         q <- q * (1 + coef * ln(floor((position + 1) / every) + 1)).
 
     With pools, keys [pages, nk, page_size, dim] and values [pages, nk, page_size, vdim] are written to the pages
-    of ``block_table`` (not at all when ``store`` is False) and the queries [N, nq * dim] are returned.  Without
+    of ``block_table`` (not at all when ``store`` is False) and the queries [N, nq * dim] are returned.  With ``pool``
+    P the means of every block of P positions that a token of the step completes (keys and values as the pages hold
+    them, float32 sums in order) are written to entry position // P of ``pooled_k`` [pages, nk, entries, dim] and
+    ``pooled_v`` [.., vdim] by ``pooled_table``; ``single_tokens``: no request brings more than one token.  Without
     pools (q, k, v) are returned as plain matrices in ``out_dtype``."""
     name = "qkv_prepare"
     need_cuda(name, src, positions, req_of_token, q_norm, k_norm, inv_freq, k_pool, v_pool, block_table, bad_flag, *biases)
@@ -298,9 +321,9 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
     for b, width in zip(biases, (nq * dim, nk * dim, nk * vdim)):
         need(b is None or (b.dtype == src.dtype and b.shape == (width,) and b.is_contiguous()), name,
              "a bias must be a contiguous vector over its heads in the dtype of src")
-    for w in (q_norm, k_norm):
-        need(w is None or (w.dtype == torch.float32 and w.shape == (dim,) and w.is_contiguous()), name,
-             "a norm scale must be float32 [dim]")
+    for w, heads in ((q_norm, nq), (k_norm, nk)):
+        need(w is None or (w.dtype == torch.float32 and w.shape == ((heads * dim if norm_all else dim),) and w.is_contiguous()),
+             name, "a norm scale must be float32 [dim], or [heads * dim] when the norm is over all heads")
     rot_dims = 0
     if inv_freq is not None:
         need(inv_freq.dtype == torch.float32 and inv_freq.dim() == 1 and inv_freq.is_contiguous()
@@ -324,16 +347,29 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
     else:
         k_out = torch.empty((n, nk * dim), dtype=out_dtype, device=src.device)
         v_out = torch.empty((n, nk * vdim), dtype=out_dtype, device=src.device)
+    pooled_width = pooled_page = pooled_pages = 0
+    if pool:
+        need_cuda(name, pooled_k, pooled_v, pooled_table)
+        need(paged and store and pool > 0, name, "pooled blocks need pages to store to")
+        need(pooled_k is not None and pooled_v is not None and pooled_k.shape[:3] == pooled_v.shape[:3]
+             and pooled_k.dim() == 4 and pooled_k.shape[1] == nk and pooled_k.shape[3] == dim and pooled_v.shape[3] == vdim
+             and pooled_k.dtype == pooled_v.dtype == src.dtype and pooled_k.is_contiguous() and pooled_v.is_contiguous(), name,
+             "pooled pools must be contiguous [pages, kv_heads, entries, dim] and [..., vdim] in the dtype of src")
+        need(pooled_table is not None and pooled_table.dtype == torch.int32 and pooled_table.dim() == 2
+             and pooled_table.is_contiguous(), name, "pooled_table must be contiguous int32 [R, width]")
+        pooled_pages, pooled_page, pooled_width = pooled_k.shape[0], pooled_k.shape[2], pooled_table.shape[1]
     # (with pools but ``store`` False - a layer that reads another entry's cache - the blocks of the key and
     # value heads find no destination and return)
     check(lib().yalis_qkv_prepare(
         ptr(src), i32(dtype_code(src.dtype)), i32(src.stride(0)), i32(q_off), i32(k_off), i32(v_off),
         ptr(biases[0]), ptr(biases[1]), ptr(biases[2]), ptr(q_norm), ptr(k_norm), f32(norm_eps), ptr(inv_freq),
-        i32(rot_dims), i32(int(interleaved)), f32(q_scale), f32(k_scale),
+        i32(rot_dims), i32(int(interleaved)), f32(rot_scale), i32(int(norm_all)), f32(q_scale), f32(k_scale),
         f32(q_temperature[0] if q_temperature is not None else 0.0), i32(q_temperature[1] if q_temperature is not None else 0),
         ptr(q_out), i32(q_out.stride(0)), ptr(k_out),
         i32(k_out.stride(0) if k_out is not None else 0), ptr(v_out), i32(v_out.stride(0) if v_out is not None else 0),
         i32(dtype_code(out_dtype)), ptr(k_pool if store else None), ptr(v_pool if store else None), ptr(block_table),
         i32(table_width), i32(page_size), i32(num_pages), ptr(positions), ptr(req_of_token), i32(n), i32(nq), i32(nk),
-        i32(dim), i32(vdim), ptr(bad_flag), stream()), name)
+        i32(dim), i32(vdim), ptr(bad_flag), i32(pool), ptr(pooled_k if pool else None), ptr(pooled_v if pool else None),
+        ptr(pooled_table if pool else None), i32(pooled_width), i32(pooled_page), i32(pooled_pages), i32(int(single_tokens)),
+        stream()), name)
     return q_out if paged else (q_out, k_out, v_out)

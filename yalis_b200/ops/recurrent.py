@@ -59,7 +59,7 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
                   req_of_token: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, *, unit_heads: int = 0,
                   dim: int = 0, q_scale: float = 1.0, unit_eps: float = 1e-6, a_raw: Optional[torch.Tensor] = None,
                   a_log: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None,
-                  b_raw: Optional[torch.Tensor] = None):
+                  b_raw: Optional[torch.Tensor] = None, conv_bias: Optional[torch.Tensor] = None):
     """What a delta rule reads, in one kernel: silu of a causal convolution over time, per channel, continuing each
     request from the tail its slot keeps; the heads of q and k brought to unit length; decay and write strength.
 
@@ -68,10 +68,13 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
     ``unit_heads`` = G > 0 the first 2 G ``dim`` channels are G heads of q and G of k: each becomes
     x / sqrt(sum x^2 + unit_eps), q times ``q_scale``.  With ``a_raw`` ([N, heads] or [N, heads * dim]), ``a_log``
     [heads], ``dt_bias`` (one per column of a_raw) and ``b_raw`` [N, heads]: g = exp(-exp(a_log) softplus(a_raw +
-    dt_bias)) and beta = sigmoid(b_raw).  Returns (float32 [N, C], g, beta), g and beta float32 or None; afterwards
+    dt_bias)) and beta = sigmoid(b_raw); without ``b_raw`` (``a_raw`` [N, heads]) beta is the step size softplus(a_raw +
+    dt_bias) itself.  ``conv_bias`` (float32 [C]) is added to the convolution before its silu.  Returns (float32 [N, C], g, beta), g and beta float32 or None; afterwards
     the tails hold the last ``taps - 1`` inputs of every request."""
     name = "delta_prepare"
-    need_cuda(name, x, weight, slot_rows, req_of_token, q_start, slots, a_raw, a_log, dt_bias, b_raw)
+    need_cuda(name, x, weight, slot_rows, req_of_token, q_start, slots, a_raw, a_log, dt_bias, b_raw, conv_bias)
+    need(conv_bias is None or (conv_bias.dtype == torch.float32 and conv_bias.shape == (x.shape[1],) and conv_bias.is_contiguous()),
+         name, "the convolution's bias must be float32 [C]")
     need(x.dim() == 2 and x.stride(1) == 1, name, "x must be [N, C] with unit inner stride")
     n, c = x.shape
     need(weight.dtype == torch.float32 and weight.dim() == 2 and weight.shape[0] == c and weight.is_contiguous(), name,
@@ -86,14 +89,15 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
     g = beta = None
     heads = a_cols = 0
     if a_raw is not None:
-        need(a_log is not None and dt_bias is not None and b_raw is not None, name, "a_raw comes with a_log, dt_bias and b_raw")
+        need(a_log is not None and dt_bias is not None, name, "a_raw comes with a_log and dt_bias")
+        need(b_raw is not None or a_raw.shape[1] == a_log.numel(), name, "without b_raw, a_raw must be [N, heads]")
         heads = a_log.numel()
         need(a_raw.dim() == 2 and a_raw.shape[0] == n and a_raw.stride(1) == 1 and a_raw.dtype == x.dtype
              and a_raw.shape[1] % heads == 0, name, "a_raw must be [N, heads] or [N, heads * dim] in the dtype of x")
         a_cols = a_raw.shape[1]
         need(a_log.dtype == torch.float32 and a_log.is_contiguous() and dt_bias.dtype == torch.float32
              and dt_bias.shape == (a_cols,) and dt_bias.is_contiguous(), name, "a_log float32 [heads], dt_bias float32 per column of a_raw")
-        need(b_raw.shape == (n, heads) and b_raw.stride(1) == 1 and b_raw.dtype == x.dtype, name, "b_raw must be [N, heads] in the dtype of x")
+        need(b_raw is None or b_raw.shape == (n, heads) and b_raw.stride(1) == 1 and b_raw.dtype == x.dtype, name, "b_raw must be [N, heads] in the dtype of x")
         g = torch.empty((n, a_cols), dtype=torch.float32, device=x.device)
         beta = torch.empty((n, heads), dtype=torch.float32, device=x.device)
     tail = slot_rows.view(-1)[tail_offset:]
@@ -102,7 +106,7 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
         ptr(req_of_token), ptr(q_start), ptr(slots), ptr(out), i32(c), i32(n), i32(slots.numel()), i32(c), i32(taps),
         i32(unit_heads), i32(dim), f32(q_scale), f32(unit_eps), ptr(a_raw), i32(a_raw.stride(0) if a_raw is not None else 0),
         i32(a_cols), ptr(a_log), ptr(dt_bias), ptr(b_raw), i32(b_raw.stride(0) if b_raw is not None else 0), i32(heads),
-        ptr(g), ptr(beta), stream()), name)
+        ptr(g), ptr(beta), ptr(conv_bias), stream()), name)
     return out, g, beta
 
 
@@ -115,7 +119,8 @@ def short_conv_silu(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tens
 def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_rows: torch.Tensor, layout: StateLayout,
                q_start: torch.Tensor, slots: torch.Tensor, *, kv_heads: int, decay: torch.Tensor,
                beta: Optional[torch.Tensor] = None, unit: Optional[torch.Tensor] = None,
-               removal: Optional[torch.Tensor] = None, max_q_len: int = 0) -> torch.Tensor:
+               removal: Optional[torch.Tensor] = None, max_q_len: int = 0, selective: bool = False,
+               skip: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Walks every request's tokens in order through the recurrence, from and to the state in its slot.
 
     Per head (S is [dim, vdim]):  S <- g S;  u = beta (v - S^T k) with ``beta`` (the delta rule), else u = v;
@@ -123,10 +128,11 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_rows: tor
     blocks are fine).  ``decay`` float32: [heads] (constant), [N, heads] (per token) or [N, heads * dim] (per key
     channel too); ``beta`` float32 [N, heads].  With ``unit`` and ``removal`` (float32 [N, heads * dim]) the rule is the generalized delta rule instead:
     S <- diag(g) S - removal (unit^T S) + k v^T, both terms reading the old state; it needs a decay per key channel
-    and kv_heads = heads, and ``decay``, ``unit``, ``removal`` contiguous.  ``max_q_len``: the longest portion of the step if known (it bounds
+    and kv_heads = heads, and ``decay``, ``unit``, ``removal`` contiguous.  ``selective``: S <- g S + k (beta v)^T and
+    o = S^T q + skip v with the step sizes ``beta``, a decay per token and ``skip`` float32 [heads] (None: 0).  ``max_q_len``: the longest portion of the step if known (it bounds
     the tile of tokens staged in shared memory, nothing else).  Returns float32 [N, heads * vdim]."""
     name = "state_scan"
-    need_cuda(name, q, k, v, slot_rows, q_start, slots, decay, beta)
+    need_cuda(name, q, k, v, slot_rows, q_start, slots, decay, beta, skip)
     h, d, vd = layout.heads, layout.dim, layout.vdim
     n = q.shape[0]
     for t, width, what in ((q, kv_heads * d, "q"), (k, kv_heads * d, "k"), (v, h * vd, "v")):
@@ -148,6 +154,12 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_rows: tor
     if beta is not None:
         need(beta.dtype == torch.float32 and beta.shape == (n, h) and beta.is_contiguous(), name, "beta must be float32 [N, heads]")
     rule = 1 if beta is not None else 0
+    need(skip is None or (selective and skip.dtype == torch.float32 and skip.shape == (h,) and skip.is_contiguous()), name,
+         "skip is float32 [heads] and belongs to the selective form")
+    if selective:
+        need(beta is not None and kind == DECAY_PER_TOKEN and unit is None and removal is None, name,
+             "the selective form takes a decay and a step size per token and head")
+        rule = 3
     if unit is not None or removal is not None:
         need(beta is None and unit is not None and removal is not None and kind == DECAY_PER_CHANNEL and kv_heads == h, name,
              "the generalized rule takes unit keys and removal vectors, a decay per key channel, kv_heads = heads and no beta")
@@ -157,7 +169,7 @@ def state_scan(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, slot_rows: tor
         rule = 2
     out = torch.empty((n, h * vd), dtype=torch.float32, device=q.device)
     check(lib().yalis_state_scan(
-        ptr(q), i32(q.stride(0)), ptr(k), i32(k.stride(0)), ptr(v), i32(v.stride(0)), ptr(decay), i32(kind), ptr(beta),
+        ptr(q), i32(q.stride(0)), ptr(k), i32(k.stride(0)), ptr(v), i32(v.stride(0)), ptr(decay), i32(kind), ptr(beta), ptr(skip),
         ptr(unit), ptr(removal), ptr(slot_rows), i64(slot_rows.stride(0)), ptr(out), i32(out.stride(0)), ptr(q_start), ptr(slots),
         i32(slots.numel()), i32(h), i32(kv_heads), i32(d), i32(vd), i32(rule), i32(max_q_len), stream()), name)
     return out
@@ -214,3 +226,24 @@ def general_delta_prepare(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a_r
                                             ptr(req_of_token), i32(n), i32(heads), i32(dim), i32(dtype_code(q.dtype)), ptr(out),
                                             stream()), name)
     return tuple(out[i] for i in range(6))
+
+
+def gate_norm(o: torch.Tensor, z: torch.Tensor, parts: int, weight: torch.Tensor, eps: float, req_of_token: torch.Tensor,
+              out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
+    """y = o * silu(z), then each of ``parts`` equal column ranges divided by its own root mean square
+    (sqrt(mean(y^2) + eps)), times ``weight`` and ``out_scale``.  ``o`` float32 [N, C]; ``z`` [N, C] in the dtype of
+    ``out``; ``weight`` float32 [C]; ``out`` [N, C] (column blocks of wider matrices are fine)."""
+    name = "gate_norm"
+    need_cuda(name, o, z, weight, req_of_token, out)
+    n, c = o.shape
+    need(o.dtype == torch.float32 and o.stride(1) == 1, name, "o must be float32 [N, C] with unit inner stride")
+    need(z.shape == (n, c) and z.stride(1) == 1 and z.dtype == out.dtype, name, "z must be [N, C] in the output's dtype")
+    need(out.shape == (n, c) and out.stride(1) == 1, name, "out must be [N, C] with unit inner stride")
+    need(parts > 0 and c % parts == 0, name, f"{c} columns do not divide into {parts} parts")
+    need(weight.dtype == torch.float32 and weight.shape == (c,) and weight.is_contiguous(), name, "weight must be float32 [C]")
+    need(req_of_token.dtype == torch.int32 and req_of_token.shape == (n,) and req_of_token.is_contiguous(), name,
+         "req_of_token must be int32 [N]")
+    check(lib().yalis_gate_norm(ptr(o), i32(o.stride(0)), ptr(z), i32(z.stride(0)), ptr(weight), ptr(out), i32(out.stride(0)),
+                                i32(dtype_code(out.dtype)), ptr(req_of_token), i32(n), i32(parts), i32(c // parts), f32(eps),
+                                f32(out_scale), stream()), name)
+    return out

@@ -11,6 +11,7 @@ model.py:544-557, which only serves its tensor-parallel split).
 from __future__ import annotations
 
 import math
+from fractions import Fraction
 from typing import Dict, Optional
 
 import torch
@@ -96,20 +97,56 @@ class PagedAttention(Mixer):
         return linear_partial(y, self.w_o)             # the residual stream adds the partial sums
 
 
+def distance_bucket(n: int, buckets: int, far: float) -> int:
+    """Which of ``buckets`` = B learned numbers the distance n >= 0 takes: n itself below h = B / 2, from there on
+    h + floor(ln(n / h) / ln(far / h) * (B - h)), at most B - 1.  The floor is taken exactly: it is at least k when
+    (n / h)^(B - h) >= (far / h)^k, a comparison of rational numbers (a logarithm in floating point falls short of whole
+    results now and then, ln(2) / ln(32) * 5 for one)."""
+    if buckets < 2 or buckets % 2:
+        raise ValueError(f"a bias per distance needs an even number of buckets, not {buckets}")
+    h = buckets // 2
+    if not far > h:
+        raise ValueError(f"the largest distance with a bucket of its own, {far}, must lie beyond {h}")
+    if n < h:
+        return n
+    grown, step = Fraction(n, h) ** (buckets - h), Fraction(far) / h
+    k, power = 0, step
+    while h + k < buckets - 1 and grown >= power:
+        k, power = k + 1, power * step
+    return h + k
+
+
+def distance_reach(buckets: int, far: float) -> int:
+    """The smallest L such that all distances from L - 1 on share a bucket, the last."""
+    lo, hi = 0, max(1, math.ceil(far))
+    while lo < hi:                           # buckets grow with the distance
+        mid = (lo + hi) // 2
+        lo, hi = (lo, mid) if distance_bucket(mid, buckets, far) == buckets - 1 else (mid + 1, hi)
+    return lo + 1
+
+
 class GeneralAttention(Mixer, Projected):
     """Grouped-query causal attention over the paged cache with the variations that the fast kernels of
     ``paged_attention`` do not take.  Parameters: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``
     (of q and k), ``v_head_dim`` (None: head_dim), ``bias`` (q, k, v = W x + b), ``qk_norm_eps`` (None: no norm;
     else q and k of every head become x / sqrt(mean(x^2) + eps) * scale before the rotation, one learned scale
-    [head_dim] for q and one for k), ``rotary`` ({"dims", "theta", "layout"}: the first ``dims`` sizes of a head turn,
-    size i paired with i + dims / 2, or with layout ``interleaved`` size 2i with 2i + 1; None: no rotation), ``scale``
+    [head_dim] for q and one for k), ``qk_norm_over`` (``head``, the default, or ``all``: the mean is over all heads of q,
+    and of k, at once, the learned scales are [heads * head_dim]), ``qk_norm_weight`` (False: a norm without learned
+    scales), ``values_from_keys`` (the values are the keys as projected, before their norm and rotation: no value matrix),
+    ``rotary`` ({"dims", "theta", "layout", "scaling"}: the first ``dims`` sizes of a head turn, size i paired with
+    i + dims / 2, or with layout ``interleaved`` size 2i with 2i + 1; ``scaling`` as the rotary part takes it, YaRN's
+    factor on cosine and sine included; None: no rotation), ``scale``
     (None: 1/sqrt(head_dim)), ``softcap`` (c: scores become c tanh(s / c)), ``sink`` (True: 1 is added to the
     softmax's denominator; ``"learned"``: exp(z_h) with a learned z per head, the tensor ``sink``), ``window`` (position
     p sees the W positions up to itself), ``chunk`` (position p sees only its own chunk of C positions, counted from
     position 0, up to itself), ``distance_slopes`` (one number per head: slope_h * (p - j) is taken off the scaled
-    score of key j), ``q_temperature`` ({"coef", "every"}: the query at position p is multiplied by
+    score of key j), ``distance_bias`` ({"buckets": B, "max": D}: rel[bucket(p - j), h] with a learned table ``rel``
+    [B, heads] is added to the scaled score, see ``distance_bucket``), ``pool`` (P, with a window: beside the window's
+    keys position p sees one key and one value for every block of P positions, counted from position 0, that lies wholly
+    before the window: the means of the block's keys and values as the cache holds them; tokens and blocks share one
+    softmax), ``q_temperature`` ({"coef", "every"}: the query at position p is multiplied by
     1 + coef ln(floor((p + 1) / every) + 1)), ``gate`` (the heads' results are multiplied by sigmoid(W_g x), one more
-    matrix over the mixer's input), ``out_bias`` (a bias on the output product), ``own_kv`` (False: the mixer has no
+    matrix over the mixer's input; ``"head"``: one number per head instead of one per element), ``out_bias`` (a bias on the output product), ``own_kv`` (False: the mixer has no
     key and value projections and reads the cache of the schedule entry it is pointed at; default True),
     ``cache_window`` (how many positions back the keys are kept, when that is not the mixer's own ``window`` or
     ``chunk``: the widest reach among this mixer and the mixers that read its cache), ``out_scale``.  Scores, weights
@@ -132,9 +169,16 @@ class GeneralAttention(Mixer, Projected):
         self.window = p.get("window")
         self.chunk = int(p["chunk"]) if p.get("chunk") is not None else None
         self.slopes_host = tuple(float(v) for v in p["distance_slopes"]) if p.get("distance_slopes") is not None else None
+        self.norm_all = str(p.get("qk_norm_over", "head")) == "all"
+        self.norm_weight = bool(p.get("qk_norm_weight", True))
+        self.values_from_keys = bool(p.get("values_from_keys", False))
+        db = p.get("distance_bias")
+        self.distance_bias = (int(db["buckets"]), db["max"]) if db is not None else None
+        self.pool = int(p["pool"]) if p.get("pool") is not None else None
         qt = p.get("q_temperature")
         self.q_temperature = (float(qt["coef"]), int(qt["every"])) if qt is not None else None
         self.gated = bool(p.get("gate", False))
+        self.gate_per_head = p.get("gate") == "head"
         self.out_bias = bool(p.get("out_bias", False))
         self.own_kv = bool(p.get("own_kv", True))
         self.cache_window = p.get("cache_window", self.window if self.window is not None else self.chunk)
@@ -145,13 +189,24 @@ class GeneralAttention(Mixer, Projected):
             raise ValueError(f"{len(self.slopes_host)} distance slopes for {self.nh} heads")
         if self.chunk is not None and self.chunk <= 0 or self.q_temperature is not None and self.q_temperature[1] <= 0:
             raise ValueError("chunk and the query temperature's period must be positive")
+        if self.distance_bias is not None:
+            distance_bucket(0, *self.distance_bias)           # refuses what has no buckets
+        if self.values_from_keys and (self.vd != self.hs or self.bias):
+            raise ValueError("values that are the keys have the keys' head size and no bias of their own")
+        if self.pool is not None:
+            if self.pool <= 0 or self.window is None or self.chunk is not None or not self.own_kv:
+                raise ValueError("pooled blocks need a window, a block size and keys of the mixer's own")
+            # a block's mean is taken when its last token arrives: its tokens must be kept until then
+            self.cache_window = max(self.cache_window, self.pool)
         if self.nh % self.g:
             raise ValueError(f"num_heads {self.nh} is not a multiple of num_kv_heads {self.g}")
         if max(self.hs, self.vd) > 256:
             raise ValueError(f"head sizes {self.hs}, {self.vd} are not supported (at most 256)")
         self.hidden_width = self.nh * self.vd
+        self.shares_projections = not self.out_bias
         self.w_in: Optional[torch.Tensor] = None
         self.w_out: Optional[torch.Tensor] = None
+        self.rel: Optional[torch.Tensor] = None
         self.biases = (None, None, None)
         self.q_norm = self.k_norm = None
         self.sink_logits = self.slopes = self.o_bias = None
@@ -160,27 +215,32 @@ class GeneralAttention(Mixer, Projected):
     def param_specs(self) -> Dict[str, ParamSpec]:
         specs = {"q_proj": ParamSpec((self.nh * self.hs, self.hidden)), "o_proj": ParamSpec((self.hidden, self.nh * self.vd))}
         if self.own_kv:
-            specs.update({"k_proj": ParamSpec((self.g * self.hs, self.hidden)), "v_proj": ParamSpec((self.g * self.vd, self.hidden))})
+            specs["k_proj"] = ParamSpec((self.g * self.hs, self.hidden))
+            if not self.values_from_keys:
+                specs["v_proj"] = ParamSpec((self.g * self.vd, self.hidden))
         if self.bias:
             specs["q_bias"] = ParamSpec((self.nh * self.hs,), init="zeros")
             if self.own_kv:
                 specs.update({"k_bias": ParamSpec((self.g * self.hs,), init="zeros"), "v_bias": ParamSpec((self.g * self.vd,), init="zeros")})
-        if self.norm_eps is not None:
-            specs["q_norm"] = ParamSpec((self.hs,), init="ones", keep_float32=True)
+        if self.norm_eps is not None and self.norm_weight:
+            specs["q_norm"] = ParamSpec((self.nh * self.hs if self.norm_all else self.hs,), init="ones", keep_float32=True)
             if self.own_kv:
-                specs["k_norm"] = ParamSpec((self.hs,), init="ones", keep_float32=True)
+                specs["k_norm"] = ParamSpec((self.g * self.hs if self.norm_all else self.hs,), init="ones", keep_float32=True)
+        if self.distance_bias is not None:
+            specs["rel"] = ParamSpec((self.distance_bias[0], self.nh), init="zeros", keep_float32=True)
         if self.learned_sink:
             specs["sink"] = ParamSpec((self.nh,), init="zeros", keep_float32=True)
         if self.gated:
-            specs["g_proj"] = ParamSpec((self.nh * self.vd, self.hidden))
+            specs["g_proj"] = ParamSpec((self.nh if self.gate_per_head else self.nh * self.vd, self.hidden))
         if self.out_bias:
             specs["o_bias"] = ParamSpec((self.hidden,), init="zeros", keep_float32=True)
         return specs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         # the input matrices stacked, each block of the product's columns on a 16-byte boundary
-        names = ["q_proj"] + (["k_proj", "v_proj"] if self.own_kv else []) + (["g_proj"] if self.gated else [])
-        plain = not self.gated and self.own_kv
+        names = ["q_proj"] + (["k_proj"] if self.own_kv else []) + (["v_proj"] if "v_proj" in t else []) \
+            + (["g_proj"] if self.gated else [])
+        plain = not self.gated and self.own_kv and not self.values_from_keys
         if plain:
             self.w_in = torch.cat([t[n] for n in names], dim=0).contiguous()
             qd, kd = self.nh * self.hs, self.g * self.hs
@@ -193,8 +253,16 @@ class GeneralAttention(Mixer, Projected):
         if self.bias:
             self.biases = tuple(t[n].to(self.w_in.dtype).contiguous() if n in t else None for n in ("q_bias", "k_bias", "v_bias"))
         if self.norm_eps is not None:
-            self.q_norm = t["q_norm"].contiguous()
-            self.k_norm = t["k_norm"].contiguous() if self.own_kv else None
+            sizes = (self.nh * self.hs, self.g * self.hs) if self.norm_all else (self.hs, self.hs)
+            unit = [torch.ones(n, dtype=torch.float32, device=self.w_in.device) for n in sizes] if not self.norm_weight else None
+            self.q_norm = unit[0] if unit else t["q_norm"].contiguous()
+            self.k_norm = (unit[1] if unit else t["k_norm"].contiguous()) if self.own_kv else None
+        if self.distance_bias is not None:
+            # the table by distance, up to the window or to where every further distance shares the last number
+            reach = distance_reach(*self.distance_bias)
+            length = min(reach, self.window) if self.window is not None else reach
+            index = torch.tensor([distance_bucket(n, *self.distance_bias) for n in range(length)], device=self.w_in.device)
+            self.rel = t["rel"].float()[index].t().contiguous()
         if self.learned_sink:
             self.sink_logits = t["sink"].float().contiguous()
         if self.slopes_host is not None:
@@ -213,14 +281,21 @@ class GeneralAttention(Mixer, Projected):
             raise ValueError("an arrangement that adds several output products into one cannot carry this mixer's output bias")
         self.w_in = self.w_out = None
 
-    def cache_request(self) -> PagedKV:
-        return PagedKV(self.g, self.hs, self.cache_window, v_head_dim=None if self.vd == self.hs else self.vd)
+    def cache_request(self):
+        vd = None if self.vd == self.hs else self.vd
+        tokens = PagedKV(self.g, self.hs, self.cache_window, v_head_dim=vd)
+        if self.pool is None:
+            return tokens
+        return {"tokens": tokens, "blocks": PagedKV(self.g, self.hs, None, v_head_dim=vd, pool=self.pool)}
 
     def _tensor_core_form(self, dtype: torch.dtype) -> bool:
-        """bfloat16 steps whose keys and values have one head size the kernel is built for go to the tensor cores
-        (scores and the sum of weights in float32, the weights against V in two bfloat16 halves); float32 steps
-        and other shapes go to the exact kernel."""
-        return dtype == torch.bfloat16 and self.vd == self.hs and attn_ops.mma_supports(self.hs)
+        """bfloat16 steps with head sizes the kernel is built for go to the tensor cores (scores and the sum of weights
+        in float32, the weights against V in two bfloat16 halves); float32 steps and other shapes go to the exact
+        kernel."""
+        if dtype != torch.bfloat16:
+            return False
+        plain = self.vd == self.hs and self.distance_bias is None and self.pool is None and attn_ops.mma_supports(self.hs)
+        return plain or attn_ops.mma_extended_supports(self.hs, self.vd)
 
     def _launch_shape(self, host):
         """(longest portion, key splits): a step in which a request's rows fill at most one tile of 16 (single
@@ -239,33 +314,45 @@ class GeneralAttention(Mixer, Projected):
             lo = max(lo, position // self.chunk * self.chunk)
         return position - lo + 1
 
+    def blocks_seen(self, position: int) -> int:
+        """How many pooled blocks the query at ``position`` sees."""
+        return max(0, position - self.window + 1) // self.pool if self.pool else 0
+
     def mixing_flops(self, q_len: int, ctx_before: int) -> float:
-        keys = sum(self.keys_seen(ctx_before + t) for t in range(q_len)) if self.window or self.chunk \
+        keys = sum(self.keys_seen(ctx_before + t) + self.blocks_seen(ctx_before + t) for t in range(q_len)) if self.window or self.chunk \
             else q_len * ctx_before + q_len * (q_len + 1) / 2
         return 2.0 * self.nh * (self.hs + self.vd) * keys
 
-    def mix(self, z: torch.Tensor, ctx, cache: PagedKVCache, y: torch.Tensor) -> None:
+    def mix(self, z: torch.Tensor, ctx, cache, y: torch.Tensor) -> None:
         if self.position is None:
-            freq, interleaved = None, False
+            freq, interleaved, magnitude = None, False, 1.0
         else:
             interleaved = bool(getattr(self.position, "interleaved", False))
-            freq = self.position.frequencies(self.position.head_dim, z.device) if interleaved \
-                else self.position.rotary_frequencies(self.position.head_dim, z.device)
+            magnitude = float(getattr(self.position, "magnitude", 1.0))
+            freq = self.position.frequencies(self.position.head_dim, z.device)
+        blocks = None
+        if self.pool is not None:
+            cache, blocks = cache["tokens"], cache["blocks"]
+            blocks = attn_ops.PooledBlocks(self.pool, blocks.k, blocks.v, ctx.block_tables[blocks.group])
         table = ctx.block_tables[cache.group]
         if self.own_kv != cache.writable:
             raise ValueError("a mixer with key and value projections writes its own cache; one without reads another's")
         q_at = self.spans["q_proj"][0]
-        k_at, v_at = (self.spans["k_proj"][0], self.spans["v_proj"][0]) if self.own_kv else (q_at, q_at)
+        k_at = self.spans["k_proj"][0] if self.own_kv else q_at
+        v_at = self.spans["v_proj"][0] if "v_proj" in self.spans else k_at
+        pooling = {} if blocks is None else dict(pool=blocks.size, pooled_k=blocks.k, pooled_v=blocks.v, pooled_table=blocks.table,
+                                                 single_tokens=ctx.host.max_q_len == 1)
         q = qkv_prepare(z, (q_at, k_at, v_at), self.nh, self.g, self.hs, self.vd, ctx.positions, ctx.req_of_token,
                         out_dtype=z.dtype, biases=self.biases, q_norm=self.q_norm, k_norm=self.k_norm,
                         norm_eps=self.norm_eps or 0.0, inv_freq=freq, k_pool=cache.k, v_pool=cache.v, block_table=table,
                         store=cache.writable, bad_flag=ctx.error_flag, interleaved=interleaved,
-                        q_temperature=self.q_temperature)
+                        q_temperature=self.q_temperature, rot_scale=magnitude, norm_all=self.norm_all, **pooling)
         gate = None
         if self.gated:
             a, b = self.spans["g_proj"]
             gate = z[:, a:b]
-        extras = dict(chunk=self.chunk, sink_logits=self.sink_logits, slopes=self.slopes, gate=gate)
+        extras = dict(chunk=self.chunk, sink_logits=self.sink_logits, slopes=self.slopes, gate=gate, rel=self.rel, pool=blocks,
+                      v_head_dim=self.vd)
         if self._tensor_core_form(z.dtype):
             longest, splits = self._launch_shape(ctx.host)
             direct = y.data_ptr() % 16 == 0 and y.stride(0) % 2 == 0
@@ -277,7 +364,7 @@ class GeneralAttention(Mixer, Projected):
                 y.copy_(out)
             return
         attn_ops.paged_attention_generic(q, cache.k, cache.v, ctx.positions, ctx.req_of_token, table, self.nh, self.g, self.hs,
-                                         scale=self.scale, window=self.window, out=y, v_head_dim=self.vd,
+                                         scale=self.scale, window=self.window, out=y,
                                          softcap=self.softcap, sink=self.sink, out_scale=self.out_scale, **extras)
 
     def forward(self, x: torch.Tensor, ctx, cache: PagedKVCache):

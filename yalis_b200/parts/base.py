@@ -74,12 +74,14 @@ class ParamSpec:
 @dataclass(frozen=True)
 class PagedKV:
     """Keys and values in pages. ``window`` None keeps every key; W keeps, for a
-    query at position p, the keys at positions > p - W."""
+    query at position p, the keys at positions > p - W.  ``pool`` P > 1: not a row per token but one entry per block of
+    P consecutive tokens (a mean of theirs, say); a page of as many entries then covers P times as many tokens."""
 
     num_kv_heads: int
     head_dim: int
     window: Optional[int] = None
     v_head_dim: Optional[int] = None      # head size of the values when it is not the keys'
+    pool: int = 1                         # tokens that one entry stands for
 
     @property
     def value_dim(self) -> int:
@@ -155,12 +157,25 @@ class PendingWrite:
 class NormedSum:
     """A sub-layer's result that is not added as it is: ``bias`` (float32 [hidden]) is added to it, and with ``norm`` =
     (weight float32 [hidden], eps) the sum is normed, d / sqrt(mean(d^2) + eps) * weight, before it joins the stream
-    (an arrangement with a norm behind each sub-layer).  ``y`` is [N, hidden] in the model dtype or float32 partial
-    sums [P, N, hidden].  All of it is float32 arithmetic inside the pass that adds it."""
+    (an arrangement with a norm behind each sub-layer).  ``second`` = (another result, its norm) is normed by itself and
+    added; the sum is multiplied by ``factor`` and, element by element, by ``scale`` (float32 [hidden]).  ``y`` is
+    [N, hidden] in the model dtype or float32 partial sums [P, N, hidden], and so is the second result.  All of it is
+    float32 arithmetic inside the pass that adds it."""
 
     y: torch.Tensor
     bias: Optional[torch.Tensor] = None
     norm: Optional[Tuple[torch.Tensor, float]] = None
+    scale: Optional[torch.Tensor] = None
+    factor: float = 1.0
+    second: Optional[Tuple[torch.Tensor, Tuple[torch.Tensor, float]]] = None
+
+    @property
+    def plain(self) -> bool:
+        """Nothing but ``y``."""
+        return self.bias is None and self.norm is None and self.scale is None and self.factor == 1.0 and self.second is None
+
+    def arguments(self) -> Dict[str, Any]:
+        return {"bias": self.bias, "delta_norm": self.norm, "scale": self.scale, "factor": self.factor, "second": self.second}
 
 
 class ResidualStream:
@@ -204,7 +219,7 @@ class ResidualStream:
         self.flush()
         if self.x.dim() == 3 and not isinstance(delta, PendingWrite):
             raise ValueError("a stream kept in several copies takes a PendingWrite, not a plain sum")
-        if isinstance(delta, NormedSum) and delta.bias is None and delta.norm is None:
+        if isinstance(delta, NormedSum) and delta.plain:
             delta = delta.y
         self.pending = delta
 
@@ -216,7 +231,7 @@ class ResidualStream:
             stream_step(self.x, read=False, source=self.take_source(), **self.pending.arguments())
         elif isinstance(self.pending, NormedSum):
             from yalis_b200.ops.elementwise import add_normed_rmsnorm
-            add_normed_rmsnorm(self.x, self.pending.y, bias=self.pending.bias, delta_norm=self.pending.norm)
+            add_normed_rmsnorm(self.x, self.pending.y, **self.pending.arguments())
         else:
             from yalis_b200.ops.elementwise import residual_add
             residual_add(self.x, self.pending)
@@ -371,6 +386,7 @@ class Projected:
     """
 
     hidden_width = 0
+    shares_projections = True        # False: what stands behind the output product cannot be shared (a norm, a bias)
 
     def in_weight(self) -> torch.Tensor:
         raise NotImplementedError

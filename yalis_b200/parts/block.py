@@ -39,8 +39,8 @@ class PreNormResidualBlock(Block):
             return result
         if not isinstance(result, NormedSum):
             result = NormedSum(result)
-        if result.norm is not None:
-            raise ValueError("the result already carries a norm")
+        if result.norm is not None or result.second is not None or result.scale is not None or result.factor != 1.0:
+            raise ValueError("the result already carries a norm or a factor")
         params = norm.rms_parameters()
         if params is not None:
             return NormedSum(result.y, result.bias, params)
@@ -81,7 +81,7 @@ class ParallelResidualBlock(Block):
         if self.w_in is not None:
             return True
         shared = [p for p in (self.mixer, self.ff) if p is not None]
-        if len(shared) < 2 or not all(isinstance(p, Projected) for p in shared):
+        if len(shared) < 2 or not all(isinstance(p, Projected) and p.shares_projections for p in shared):
             return False
         if any(p.in_weight().dtype != shared[0].in_weight().dtype or p.out_weight().dtype != shared[0].out_weight().dtype
                for p in shared):

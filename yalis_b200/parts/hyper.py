@@ -5,6 +5,9 @@ all copies at once, x_t <- sum_s mix[s, t] x_s + out_t y.  Before the write y ma
 by a learned vector (``layer_scale``) and by a gate sigmoid(W_g h + b_g) computed from what the sub-layer read
 (``gate``).  With one copy and no mixing this is the plain residual sum with those two factors.
 
+``scaled_sum`` (category ``connection``): the plain residual sum of a stream of one copy with a learned vector on the
+sub-layer's result, x += y * scale; the vector rides along with the result into the pass that adds it.
+
 ``pre_norm_connected`` (category ``block``): x <- write_1(mixer(norm_1(read_1 x))), then the same with the
 feed-forward, if the layer has one.  The norm reads the copies, applies the pending write of the sub-layer before
 and norms in one pass (``ops/streams.stream_step``).
@@ -12,6 +15,7 @@ and norms in one pass (``ops/streams.stream_step``).
 
 from __future__ import annotations
 
+from dataclasses import replace
 from typing import Dict, Optional
 
 import torch
@@ -19,7 +23,7 @@ import torch
 from yalis_b200.config.spec import PartSpec
 from yalis_b200.ops.linear import linear
 from yalis_b200.ops.streams import MAX_COPIES
-from .base import Block, Connection, ParamSpec, PendingWrite, ResidualStream, register_part
+from .base import Block, Connection, NormedSum, ParamSpec, PendingWrite, ResidualStream, register_part
 
 
 class HyperConnection(Connection):
@@ -73,6 +77,30 @@ class HyperConnection(Connection):
         return None
 
 
+class ScaledSum(Connection):
+    """x += y * scale.  Parameters: ``hidden_size``.  The scale is held in float32."""
+
+    def __init__(self, spec: PartSpec):
+        super().__init__(spec)
+        self.hidden = int(spec.params["hidden_size"])
+        self.scale: Optional[torch.Tensor] = None
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"scale": ParamSpec((self.hidden,), init="ones", keep_float32=True)}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        self.scale = t["scale"].contiguous()
+
+    def write(self, h: torch.Tensor, y) -> NormedSum:
+        result = y if isinstance(y, NormedSum) else NormedSum(y)
+        if result.scale is not None:
+            raise ValueError("the result already carries a scale")
+        return replace(result, scale=self.scale)
+
+    def capture_key(self, host):
+        return None
+
+
 class PreNormConnectedBlock(Block):
     """h = norm_1(read_1(x)); x <- write_1(h, mixer(h)); h = norm_2(read_2(x)); x <- write_2(h, feed_forward(h)).
     Reads and writes are the layer's ``connection`` parts; the norms must read a stream of several copies with
@@ -103,4 +131,5 @@ class PreNormConnectedBlock(Block):
 
 
 register_part("connection", "hyper_connection", HyperConnection)
+register_part("connection", "scaled_sum", ScaledSum)
 register_part("block", "pre_norm_connected", PreNormConnectedBlock)

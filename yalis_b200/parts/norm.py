@@ -14,20 +14,23 @@ from .base import Norm, NormedSum, ParamSpec, PendingWrite, ResidualStream, regi
 
 class RMSNorm(Norm):
     """Parameters: ``size`` (width of the stream), ``eps``, ``one_plus`` (the stored tensor w lies around
-    zero and the scale is 1 + w; default False: the tensor is the scale).  The scale is held in float32."""
+    zero and the scale is 1 + w; default False: the tensor is the scale), ``scalar`` (the stored tensor is one number,
+    the scale of every coordinate).  The scale is held in float32."""
 
     def __init__(self, spec: PartSpec):
         super().__init__(spec)
         self.size = int(spec.params["size"])
         self.eps = float(spec.params["eps"])
         self.one_plus = bool(spec.params.get("one_plus", False))
+        self.scalar = bool(spec.params.get("scalar", False))
         self.weight: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {"weight": ParamSpec((self.size,), init="zeros" if self.one_plus else "ones", keep_float32=True)}
+        return {"weight": ParamSpec(() if self.scalar else (self.size,), init="zeros" if self.one_plus else "ones", keep_float32=True)}
 
     def load(self, tensors: Dict[str, torch.Tensor]) -> None:
-        w = tensors["weight"].contiguous()
+        w = tensors["weight"]
+        w = w.reshape(1).expand(self.size).contiguous() if self.scalar else w.contiguous()
         self.weight = (1.0 + w) if self.one_plus else w       # float32: the sum is exact to one rounding
 
     def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
@@ -38,8 +41,8 @@ class RMSNorm(Norm):
             stream.flush()
         if isinstance(stream.pending, NormedSum):      # a result with a bias or a norm of its own: the same single pass
             pend = stream.pending
-            y = add_normed_rmsnorm(stream.x, pend.y, bias=pend.bias, delta_norm=pend.norm, weight=self.weight, eps=self.eps,
-                                   out_dtype=stream.dtype, rows=rows)
+            y = add_normed_rmsnorm(stream.x, pend.y, weight=self.weight, eps=self.eps, out_dtype=stream.dtype, rows=rows,
+                                   **pend.arguments())
         else:
             y = add_rmsnorm(stream.x, stream.pending, self.weight, self.eps, stream.dtype, rows=rows)
         if rows is None:

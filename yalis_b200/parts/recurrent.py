@@ -8,9 +8,13 @@
 ``general_delta``  S <- diag(w_t) S - (a_t * u_t)(u_t^T S) + k_t v_t^T (both terms read the old S);  o_t = S^T r_t  with
                  the unit key u_t = k_t / |k_t|, a decay w_t per head and key channel through a low-rank product and a
                  removal rate a_t per head and key channel; a normed, sigmoid-gated read-out.
-``sum_of_mixers``  several mixers that read the same input; their results are added, each times its factor.
+``state_space``  S_t = exp(-exp(A) s_t) S_(t-1) + s_t B_t x_t^T,  y_t = S_t^T C_t + D x_t  with a step size s_t per
+                 token and head, B and C shared by groups of heads, a short convolution before and a gate and a norm
+                 in equal parts behind (Mamba-2).
+``sum_of_mixers``  several mixers that read the same input; their results are added, each times its factor or each
+                 through a norm of its own.
 
-All three are ``Projected``: an arrangement may run their input and output products together with those of its
+All of them are ``Projected``: an arrangement may run their input and output products together with those of its
 other parts.  What the recurrences keep (state matrices in float32, the convolution's last inputs) is one row
 of slot memory per request; the kernels walk a request's tokens in order, so the result at a position does not
 depend on how the request was cut into steps.
@@ -25,18 +29,18 @@ import torch
 from yalis_b200.config.spec import PartSpec
 from yalis_b200.ops import recurrent as rec_ops
 from yalis_b200.ops.elementwise import activation, qkv_prepare
-from yalis_b200.ops.linear import linear
-from .base import Mixer, ParamSpec, PositionEncoding, Projected, SlotState, SlotStateCache, make_part, register_part, stack_rows
+from yalis_b200.ops.linear import linear, linear_partial
+from .base import Mixer, NormedSum, ParamSpec, PositionEncoding, Projected, SlotState, SlotStateCache, make_part, register_part, stack_rows
 
 
 def position_part(params) -> Optional[PositionEncoding]:
     """The position part a mixer builds for itself from its ``rotary`` parameter ({"dims", "theta"} and optionally
-    "layout"; None: none)."""
+    "layout" and "scaling", as the rotary part takes them; None: none)."""
     rot = params.get("rotary")
     if rot is None:
         return None
     return make_part("position", PartSpec("rotary", {"head_dim": int(rot["dims"]), "theta": float(rot["theta"]),
-                                                     "scaling": None, "exact_powers": True,
+                                                     "scaling": rot.get("scaling"), "exact_powers": True,
                                                      "layout": rot.get("layout", "half")}))
 
 
@@ -260,10 +264,80 @@ class GeneralDelta(_ProjectedMixer):
                                gate_kind=rec_ops.GATE_SIGMOID, out_scale=self.out_scale)
 
 
+class StateSpace(_ProjectedMixer):
+    """Selective state space with a scalar decay per head (Mamba-2, "state space duality").  Parameters: ``hidden_size``,
+    ``heads``, ``vdim`` (of x, per head), ``state`` (N, the size of B and C), ``groups`` (of B and C; head h uses group
+    h // (heads / groups)), ``conv`` (taps), ``norm_groups`` (equal parts of the read-out with a norm each), ``eps``,
+    ``out_scale``.  With inner = heads * vdim,
+
+        [z: inner | x: inner | B: groups N | C: groups N | s: heads] = W_in h
+        x, B, C <- silu(causal convolution per channel + bias)           s <- softplus(s + dt_bias)
+        S <- exp(-exp(A_log) s) S + B (s x)^T                             y = S^T C + D x          per head
+        y <- y silu(z), every part divided by its root mean square, * norm;   result W_o y
+
+    Everything between the two products is float32; the state [heads, N, vdim] and the convolution's last inputs are a
+    float32 slot row."""
+
+    def __init__(self, spec: PartSpec, position: Optional[PositionEncoding] = None):
+        super().__init__(spec, position)
+        p = spec.params
+        self.hidden, self.h, self.vd, self.n = int(p["hidden_size"]), int(p["heads"]), int(p["vdim"]), int(p["state"])
+        self.g, self.taps, self.parts, self.eps = int(p["groups"]), int(p["conv"]), int(p["norm_groups"]), float(p["eps"])
+        self.inner = self.h * self.vd
+        if self.h % self.g:
+            raise ValueError(f"state_space: heads {self.h} is not a multiple of groups {self.g}")
+        if self.inner % self.parts:
+            raise ValueError(f"state_space: {self.inner} columns do not divide into {self.parts} parts")
+        self.channels = self.inner + 2 * self.g * self.n
+        self.layout = rec_ops.StateLayout(self.h, self.n, self.vd, self.channels, self.taps)
+        self.hidden_width = self.inner
+        self.spans: Dict[str, tuple] = {}
+
+    def param_specs(self) -> Dict[str, ParamSpec]:
+        return {"in_proj": ParamSpec((self.inner + self.channels + self.h, self.hidden)),
+                "conv": ParamSpec((self.channels, self.taps), keep_float32=True),
+                "conv_bias": ParamSpec((self.channels,), init="zeros", keep_float32=True),
+                "dt_bias": ParamSpec((self.h,), init="zeros", keep_float32=True),
+                "A_log": ParamSpec((self.h,), init="zeros", keep_float32=True),
+                "D": ParamSpec((self.h,), init="ones", keep_float32=True),
+                "norm": ParamSpec((self.inner,), init="ones", keep_float32=True),
+                "o_proj": ParamSpec((self.hidden, self.inner))}
+
+    def load(self, t: Dict[str, torch.Tensor]) -> None:
+        w, a, b = t["in_proj"], self.inner, self.inner + self.channels
+        self.w_in, spans = stack_rows([w[:a], w[a:b], w[b:]])       # each block of columns on a 16-byte boundary
+        self.spans = dict(zip(("z", "xbc", "step"), spans))
+        self.w_out = t["o_proj"].contiguous()
+        self.conv_w, self.conv_b, self.dt_bias = t["conv"].contiguous(), t["conv_bias"].contiguous(), t["dt_bias"].contiguous()
+        self.a_log, self.skip, self.norm_w = t["A_log"].contiguous(), t["D"].contiguous(), t["norm"].contiguous()
+
+    def cache_request(self) -> SlotState:
+        return SlotState((self.layout.total,), torch.float32)
+
+    def mixing_flops(self, q_len: int, ctx_before: int) -> float:
+        return 4.0 * self.h * self.n * self.vd * q_len
+
+    def mix(self, z: torch.Tensor, ctx, cache: SlotStateCache, y: torch.Tensor) -> None:
+        blk = lambda name: z[:, self.spans[name][0]:self.spans[name][1]]
+        conv, decay, step = rec_ops.delta_prepare(
+            blk("xbc"), self.conv_w, cache.state, self.layout.state_floats, ctx.req_of_token, ctx.q_start, ctx.slots,
+            a_raw=blk("step"), a_log=self.a_log, dt_bias=self.dt_bias, conv_bias=self.conv_b)
+        b, c = self.inner, self.inner + self.g * self.n
+        o = rec_ops.state_scan(conv[:, c:], conv[:, b:c], conv[:, :b], cache.state, self.layout, ctx.q_start, ctx.slots,
+                               kv_heads=self.g, decay=decay, beta=step, selective=True, skip=self.skip,
+                               max_q_len=ctx.host.max_q_len)
+        rec_ops.gate_norm(o, blk("z"), self.parts, self.norm_w, self.eps, ctx.req_of_token, y, out_scale=self.out_scale)
+
+
 class SumOfMixers(_ProjectedMixer):
     """Parameters: ``mixers``: name -> PartSpec of a ``Projected`` mixer (its ``out_scale`` is its factor in the sum).
     All read the same input.  Tensors of mixer ``name`` are named ``<name>.<its own name>``; what the mixers keep
-    is asked for and handed out as a dictionary by mixer name."""
+    is asked for and handed out as a dictionary by mixer name.
+
+    With ``norm_eps`` there are two mixers and each result is normed over the model's width before the sum, r / sqrt(
+    mean(r^2) + norm_eps) * w with a learned w (tensor ``<name>.out_norm``), and the sum is multiplied by ``factor``: the
+    mixers' output products then stay apart, and both norms, the sum and the factor are left to the pass that adds the
+    result to the stream (a ``NormedSum`` of two results)."""
 
     def __init__(self, spec: PartSpec, position: Optional[PositionEncoding] = None):
         super().__init__(spec, position)
@@ -271,19 +345,41 @@ class SumOfMixers(_ProjectedMixer):
         for name, m in self.subs.items():
             if not isinstance(m, Projected):
                 raise ValueError(f"sum_of_mixers: mixer {name!r} ({m.spec.kind}) cannot share its products")
+        self.norm_eps = float(spec.params["norm_eps"]) if spec.params.get("norm_eps") is not None else None
+        self.factor = float(spec.params.get("factor", 1.0))
+        if self.norm_eps is not None and len(self.subs) != 2:
+            raise ValueError(f"sum_of_mixers: two mixers are normed before their sum, not {len(self.subs)}")
+        if self.norm_eps is None and self.factor != 1.0:
+            raise ValueError("sum_of_mixers: without norms a mixer's factor is its own out_scale")
+        self.shares_projections = self.norm_eps is None
         self.hidden_width = sum(m.hidden_width for m in self.subs.values())
         self.in_spans: List[tuple] = []
+        self.out_weights: Dict[str, torch.Tensor] = {}
+        self.out_norms: Dict[str, torch.Tensor] = {}
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {f"{name}.{local}": ps for name, m in self.subs.items() for local, ps in m.param_specs().items()}
+        specs = {f"{name}.{local}": ps for name, m in self.subs.items() for local, ps in m.param_specs().items()}
+        if self.norm_eps is not None:
+            for name, m in self.subs.items():
+                specs[f"{name}.out_norm"] = ParamSpec((m.hidden,), init="ones", keep_float32=True)
+        return specs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         for name, m in self.subs.items():
             m.load({local: t[f"{name}.{local}"] for local in m.param_specs()})
         self.w_in, self.in_spans = stack_rows([m.in_weight() for m in self.subs.values()])
-        self.w_out = torch.cat([m.out_weight() for m in self.subs.values()], dim=1).contiguous()
+        if self.norm_eps is None:
+            self.w_out = torch.cat([m.out_weight() for m in self.subs.values()], dim=1).contiguous()
+        else:
+            self.out_weights = {name: m.out_weight() for name, m in self.subs.items()}
+            self.out_norms = {name: t[f"{name}.out_norm"].contiguous() for name in self.subs}
         for m in self.subs.values():
             m.release_projections()
+
+    def out_weight(self) -> torch.Tensor:
+        if self.norm_eps is not None:
+            raise ValueError("sum_of_mixers: normed results have an output product each")
+        return self.w_out
 
     def cache_request(self):
         req = {name: m.cache_request() for name, m in self.subs.items()}
@@ -308,8 +404,21 @@ class SumOfMixers(_ProjectedMixer):
             m.mix(z[:, a:b], ctx, (cache or {}).get(name), y[:, at:at + m.hidden_width])
             at += m.hidden_width
 
+    def forward(self, x: torch.Tensor, ctx, cache):
+        if self.norm_eps is None:
+            return super().forward(x, ctx, cache)
+        z = linear(x, self.w_in)
+        results = []
+        for (name, m), (a, b) in zip(self.subs.items(), self.in_spans):
+            y = torch.empty((x.shape[0], m.hidden_width), dtype=x.dtype, device=x.device)
+            m.mix(z[:, a:b], ctx, (cache or {}).get(name), y)
+            results.append((linear_partial(y, self.out_weights[name]), (self.out_norms[name], self.norm_eps)))
+        (first, norm), second = results
+        return NormedSum(first, norm=norm, second=second, factor=self.factor)
+
 
 register_part("mixer", "retention", Retention)
 register_part("mixer", "gated_delta", GatedDelta)
 register_part("mixer", "general_delta", GeneralDelta)
+register_part("mixer", "state_space", StateSpace)
 register_part("mixer", "sum_of_mixers", SumOfMixers)
