@@ -172,7 +172,7 @@ def short_convolution(x, w, b):
     """y_t = silu(b + sum_j w[., K-1-j] x_(t-j)) per channel, x before the start is zero."""
     K = w.shape[1]
     y = torch.zeros_like(x) + b
-    for j in range(K):
+    for j in range(min(K, x.shape[0])):
         y[j:] += x[:x.shape[0] - j] * w[:, K - 1 - j]
     return y * torch.sigmoid(y)
 

@@ -363,6 +363,85 @@ PRESETS["sazavik-1b"] = _sazavik_stack(2048, 32000, 4, 16, 8, 128, 2048, 1024, 4
 PRESETS["sazavik-3b"] = _sazavik_stack(3072, 32000, 6, 24, 8, 128, 2048, 1024, 6144, 64, 4, 1024, 3072)
 
 
+# ---- Ludelorn ------------------------------------------------------------------------------------------------------
+
+def _ld_heads(heads, kv_heads, dim, vdim, scale, window, pool=None, rot=None, yarn=None):
+    mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "mask": {"size": window}}
+    if pool is not None:
+        mixer["mask"]["pool"] = pool
+    if rot is not None:
+        mixer["rot"] = {"dims": rot[0], "base": rot[1]}
+        if yarn is not None:
+            mixer["rot"]["scaling"] = dict(zip(("factor", "original", "fast", "slow"), yarn))
+    return mixer
+
+
+def _ld_layer(kind, mixer, ff):
+    return {"type": kind, "mixer": mixer, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+
+
+def _ld_parallel(left, right, ff):
+    keys = ("heads", "vdim", "state", "groups", "norm_groups", "conv")
+    return _ld_layer("parallel", {"left": left, "right": dict(zip(keys, right))}, ff)
+
+
+def _ld_pooled(mixer, ff):
+    return _ld_layer("attention", mixer, ff)
+
+
+def _ld_biased(heads, kv_heads, dim, scale, window, buckets, bias_max, ff):
+    return _ld_layer("attention_2", {**_ld_heads(heads, kv_heads, dim, dim, scale, window), "bias_max": bias_max, "buckets": buckets}, ff)
+
+
+def _ludelorn(width, vocab, layers, scale=1.0, eps=1e-6) -> Dict[str, Any]:
+    return {"architecture": "Ludelorn", "embedding": {"scale": scale}, "layers": layers, "norm": {"eps": eps}, "vocab": vocab,
+            "width": width}
+
+
+def _ludelorn_stack(width, vocab, groups, heads, kv_heads, dim, ff) -> Dict[str, Any]:
+    """``groups`` times (parallel, pooled attention, parallel, attention with a distance bias): head size ``dim``
+    everywhere, a state space as wide as the model."""
+    sides = lambda: _ld_parallel(_ld_heads(heads, kv_heads, dim, dim, dim ** -0.5, 1024, rot=(dim, 500000.0), yarn=(8.0, 4096, 32.0, 1.0)),
+                                 (width // 64, 64, 128, kv_heads, kv_heads, 4), ff)
+    layers = []
+    for _ in range(groups):
+        layers += [sides(), _ld_pooled(_ld_heads(heads, kv_heads, dim, dim, dim ** -0.5, 512, pool=16, rot=(dim, 10000.0)), ff),
+                   sides(), _ld_biased(heads, kv_heads, dim, dim ** -0.5, 1024, 32, 512, ff)]
+    return _ludelorn(width, vocab, layers, scale=8.0)
+
+
+# Test shapes.  A: every mixer, partial rotations with and without YaRN, a pooled block longer than its window, a layer
+# without feed-forward, key and value sizes apart.  B: sizes that are multiples of nothing (no row on a 16-byte
+# boundary), one tap, one group, one part, windows and blocks of one position, two buckets.  C: the head sizes of the
+# tensor-core kernels, blocks of a page, a state of 128 rows.  D: many heads to a key head, windows that never bind, head
+# sizes that are multiples of 8 only, as many groups and parts as heads, six taps.
+PRESETS["ludelorn-tiny-A"] = _ludelorn(64, 96, [
+    _ld_parallel(_ld_heads(4, 2, 16, 24, 0.3, 9, rot=(8, 100.0), yarn=(4.0, 64, 6.0, 1.0)), (4, 12, 10, 2, 3, 3), 80),
+    _ld_pooled(_ld_heads(4, 2, 16, 8, 0.25, 5, pool=7, rot=(12, 50.0)), None),
+    _ld_biased(4, 2, 12, 0.3, 23, 8, 20, 48),
+    _ld_parallel(_ld_heads(2, 1, 20, 16, 0.2, 13, rot=(20, 30.0)), (3, 8, 6, 1, 2, 5), None),
+    _ld_pooled(_ld_heads(2, 2, 12, 20, 0.35, 11, pool=3, rot=(12, 1000.0), yarn=(2.0, 40, 4.0, 0.5)), 56)], scale=2.5)
+PRESETS["ludelorn-tiny-B"] = _ludelorn(37, 50, [
+    _ld_biased(3, 1, 7, 0.4, 4, 2, 3, 30),
+    _ld_parallel(_ld_heads(3, 3, 10, 5, 0.3, 6, rot=(10, 20.0), yarn=(3.0, 16, 2.0, 0.25)), (5, 3, 9, 1, 1, 1), 18),
+    _ld_pooled(_ld_heads(3, 1, 14, 9, 0.3, 1, pool=1, rot=(2, 7.0)), 26),
+    _ld_pooled(_ld_heads(2, 1, 6, 11, 0.4, 3, pool=4, rot=(6, 9.0)), None)], eps=1e-4)
+PRESETS["ludelorn-tiny-C"] = _ludelorn(128, 160, [
+    _ld_parallel(_ld_heads(4, 2, 64, 32, 0.125, 33, rot=(32, 10000.0), yarn=(4.0, 256, 16.0, 1.0)), (4, 32, 128, 2, 4, 4), 256),
+    _ld_pooled(_ld_heads(4, 4, 64, 64, 0.14, 40, pool=8, rot=(64, 1000.0)), 128),
+    _ld_biased(8, 2, 16, 0.25, 70, 16, 50, 256),
+    _ld_pooled(_ld_heads(2, 1, 128, 96, 0.09, 16, pool=16, rot=(64, 10000.0)), 256),
+    _ld_biased(2, 1, 128, 0.09, 20, 32, 64, 128)], scale=3.0)
+PRESETS["ludelorn-tiny-D"] = _ludelorn(96, 64, [
+    _ld_biased(20, 1, 24, 0.25, 4096, 10, 160, 72),
+    _ld_parallel(_ld_heads(16, 1, 40, 24, 0.2, 4096, rot=(40, 500.0)), (6, 16, 20, 6, 6, 6), 40),
+    _ld_pooled(_ld_heads(6, 2, 24, 40, 0.22, 19, pool=5, rot=(8, 77.0)), 88)], scale=0.7)
+# Sizes that resemble a real model's layers (random weights, for the benchmark): the widths, heads and feed-forwards of the
+# Tirezen benchmark models.
+PRESETS["ludelorn-1b"] = _ludelorn_stack(2048, 32000, 4, 16, 8, 128, 8192)
+PRESETS["ludelorn-3b"] = _ludelorn_stack(3072, 32000, 6, 24, 8, 128, 8192)
+
+
 def preset(name: str) -> Dict[str, Any]:
     """A fresh copy of the named configuration dictionary."""
     for key in (name, name.split("/")[-1], name.split("/")[-1].replace("Meta-", "")):
