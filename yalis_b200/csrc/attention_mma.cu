@@ -77,10 +77,11 @@ struct AttnParams {
   int hs, vs;                  // FORM 2: sizes of a key and a value (multiples of 8, at most HS)
   const float* rel;            // FORM 2: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
   int rel_len;
+  int rel_staged;              // the table of a block's heads fits the shared memory set aside for it
   int pool;                    // FORM 2: P > 0: pooled blocks of P positions before the window
   const __nv_bfloat16* pk_pool; const __nv_bfloat16* pv_pool;   // [pages, g, pool_page_size, HS / VS], an entry per block
   const int32_t* pool_table;
-  int pool_table_width, pool_page_size, pool_num_pages;
+  int pool_table_width, pool_page_size, pool_num_pages, pool_page_shift;
   int n_splits;
   float* part_o;               // [N, nh, n_splits, HS] (split mode)
   float* part_ml;              // [N, nh, n_splits, 2]
@@ -165,6 +166,7 @@ __device__ __forceinline__ void load_kv_tile_sized(__nv_bfloat16* k_dst, __nv_bf
   constexpr int CHUNKS = HS / 8, LD = HS + 8;
   const int width = pooled ? p.pool_table_width : p.table_width;
   const int32_t* bt = (pooled ? p.pool_table : p.block_table) + (size_t)req * width;
+  const int shift = pooled ? p.pool_page_shift : p.page_shift;
   const int ps = pooled ? p.pool_page_size : p.page_size, pages = pooled ? p.pool_num_pages : p.num_pages;
   const __nv_bfloat16* kp = pooled ? p.pk_pool : p.k_pool;
   const __nv_bfloat16* vp = pooled ? p.pv_pool : p.v_pool;
@@ -177,7 +179,7 @@ __device__ __forceinline__ void load_kv_tile_sized(__nv_bfloat16* k_dst, __nv_bf
     const int key = key0 + c / CHUNKS;
     at[i] = -1;
     if (key >= lo_key && key <= hi_key) {
-      const int pi = key / ps;
+      const int pi = shift >= 0 ? (key >> shift) : (key / ps);
       const int page = pi < width ? bt[pi] : -1;
       if (page >= 0 && page < pages) at[i] = ((long long)page * p.g + kvh) * ps + (key - pi * ps);
     }
@@ -259,6 +261,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [RB][LD]
   __nv_bfloat16* k_s = q_s + RB * LD;                                 // [NST][BN][LD]
   __nv_bfloat16* v_s = k_s + NST * BN * LD;                           // [NST][BN][LD]
+  float* rel_s = reinterpret_cast<float*>(v_s + NST * BN * LD);       // extended: [per][rel_len] in the exp2 domain
   pdl_launch_dependents();
   pdl_wait();
 
@@ -329,6 +332,10 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       }
     }
   }
+  if (EXT && p.rel && p.rel_staged) {
+    const float* src = p.rel + (size_t)kvh * p.per * p.rel_len;
+    for (int e = threadIdx.x; e < p.per * p.rel_len; e += NWARPS * 32) rel_s[e] = src[e] * 1.4426950408889634f;
+  }
   // Prologue: Q and the first tile form one group, then NST-2 further tiles one group each.
 #pragma unroll
   for (int t = 0; t < NST - 1; ++t) {
@@ -351,6 +358,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   float row_slope[2] = {0.f, 0.f};      // in the exp2 domain
   int row_blocks[2] = {0, 0};           // extended: pooled blocks the row sees
   const float* row_rel[2] = {nullptr, nullptr};
+  int row_head[2] = {0, 0};
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
     const int row = row0 + wrow + gid + i * 8;
@@ -360,6 +368,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     if (GEN && p.slopes && row_ok[i]) row_slope[i] = p.slopes[kvh * p.per + row % p.per] * 1.4426950408889634f;
     if (EXT && row_ok[i]) {
       row_blocks[i] = blocks_seen(p, row_pos[i]);
+      row_head[i] = row % p.per;
       if (p.rel) row_rel[i] = p.rel + (size_t)(kvh * p.per + row % p.per) * p.rel_len;
     }
   }
@@ -426,7 +435,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
               vis = key < row_blocks[i];
               off = 0.f;
             } else if (vis && p.rel) {
-              off -= __ldg(row_rel[i] + min(row_pos[i] - key, p.rel_len - 1)) * 1.4426950408889634f;
+              const int at = min(row_pos[i] - key, p.rel_len - 1);
+              off -= p.rel_staged ? rel_s[row_head[i] * p.rel_len + at] : row_rel[i][at] * 1.4426950408889634f;
             }
           }
           const float v = vis ? score_log2<GEN>(p, s[j][e], off) : -INFINITY;
@@ -663,14 +673,19 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 }
 
 template <int HS, bool DEC, int FORM>
-int launch_mode(const AttnParams& p, int n_requests, int max_rows, cudaStream_t stream) {
+int launch_mode(const AttnParams& args, int n_requests, int max_rows, cudaStream_t stream) {
   constexpr int LD = HS + 8;
   constexpr int RB = DEC ? 16 : BM, NST = DEC ? 3 : 2;
-  const size_t smem = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
+  constexpr size_t tiles = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
+  // what a staged table of biases may take without costing a resident block
+  constexpr int rel_room = FORM == 2 ? (DEC ? 1024 : 4096) : 0;
+  AttnParams p = args;
+  p.rel_staged = p.rel != nullptr && p.per * p.rel_len <= rel_room;
+  const size_t smem = tiles + (p.rel_staged ? (size_t)p.per * p.rel_len * sizeof(float) : 0);
   static bool configured = false;
   if (!configured) {
     if (cudaFuncSetAttribute(paged_attention_mma_kernel<HS, DEC, FORM>, cudaFuncAttributeMaxDynamicSharedMemorySize,
-                             (int)smem) != cudaSuccess)
+                             (int)(tiles + rel_room * sizeof(float))) != cudaSuccess)
       return YALIS_ERR_LAUNCH;
     configured = true;
   }
@@ -758,6 +773,9 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
   p.hs = hs; p.vs = vs; p.rel = rel; p.rel_len = rel_len; p.pool = pool;
   p.pk_pool = (const __nv_bfloat16*)pk_pool; p.pv_pool = (const __nv_bfloat16*)pv_pool; p.pool_table = pool_table;
   p.pool_table_width = pool_table_width; p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
+  p.pool_page_shift = -1;
+  for (int sh = 0; sh < 31; ++sh)
+    if ((1 << sh) == pool_page_size) p.pool_page_shift = sh;
   const bool extended = vs != hs || rel != nullptr || pool > 0 || !yalis_attention_mma_supports(hs);
   if (pool < 0 || (rel && rel_len < 1)) return YALIS_ERR_SHAPE;
   if (pool > 0) {

@@ -96,44 +96,81 @@ __global__ void store_block_means_kernel(const PrepParams p) {
 }
 
 // Sum over the block of the squares of `count` values (plus a bias) of a row.
-template <typename T>
+template <typename T, bool VEC>
 __device__ __forceinline__ float row_squares(const T* row, const T* bias, int count, float* scratch) {
   float ss = 0.f;
-  for (int c = threadIdx.x; c < count; c += blockDim.x) {
-    float x = to_f32<T>(row[c]);
-    if (bias) x += to_f32<T>(bias[c]);
-    ss = __fmaf_rn(x, x, ss);
+  if constexpr (VEC) {
+    for (int c = threadIdx.x * 4; c < count; c += blockDim.x * 4) {
+      float4 x = load4_f32(row + c);
+      if (bias) {
+        const float4 b = load4_f32(bias + c);
+        x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+      }
+      ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+    }
+  } else {
+    for (int c = threadIdx.x; c < count; c += blockDim.x) {
+      float x = to_f32<T>(row[c]);
+      if (bias) x += to_f32<T>(bias[c]);
+      ss = __fmaf_rn(x, x, ss);
+    }
   }
   return block_sum(ss, scratch);
 }
 
 // One warp per (token, head): heads [0, nq) are queries, [nq, nq + nk) keys, [nq + nk, nq + 2 nk) values.  A warp goes on
 // to further heads of its token where the grid has fewer warps than heads.
-template <typename T, typename TO>
+// TABLE: the block computes the token's sines and cosines once, in shared memory (steps of many tokens, where a block
+// walks all heads).  VEC: four consecutive values at a time (every row, size and offset a multiple of four, aligned).
+template <typename T, typename TO, bool TABLE, bool VEC>
 __global__ void qkv_prepare_kernel(const PrepParams p) {
-  extern __shared__ float xs_all[];           // a row of `width_max` floats per warp
+  extern __shared__ __align__(16) float xs_all[];   // a row of `row_floats` per warp, then (TABLE) cosines and sines
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
   const int n = blockIdx.x, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-  float* xs = xs_all + (size_t)(threadIdx.x >> 5) * (p.dim > p.vdim ? p.dim : p.vdim);
+  const int row_floats = ((p.dim > p.vdim ? p.dim : p.vdim) + 3) & ~3;
+  float* xs = xs_all + (size_t)(threadIdx.x >> 5) * row_floats;
   const int req = p.req_of_token[n];
   if (req < 0) return;
   const int pos = p.positions[n];
   const T* row = reinterpret_cast<const T*>(p.src) + (size_t)n * p.src_stride;
+  const int half = p.inv_freq ? p.rot_dims >> 1 : 0;
+  float* cos_s = xs_all + (size_t)warps * row_floats;
+  float* sin_s = cos_s + ((half + 3) & ~3);
+  if constexpr (TABLE) {
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      float sn, cs;
+      sincosf((float)pos * p.inv_freq[i], &sn, &cs);
+      cos_s[i] = cs * p.rot_scale;
+      sin_s[i] = sn * p.rot_scale;
+    }
+    __syncthreads();
+  }
   float all_q = 1.f, all_k = 1.f;             // norm over all heads: 1 / root mean square of the whole of q and of k
   if (p.norm_all) {
-    if (p.q_norm) all_q = 1.0f / sqrtf(row_squares(row + p.q_off, reinterpret_cast<const T*>(p.q_bias), p.nq * p.dim, scratch) /
+    if (p.q_norm) all_q = 1.0f / sqrtf(row_squares<T, VEC>(row + p.q_off, reinterpret_cast<const T*>(p.q_bias), p.nq * p.dim, scratch) /
                                            (float)(p.nq * p.dim) + p.norm_eps);
-    if (p.k_norm) all_k = 1.0f / sqrtf(row_squares(row + p.k_off, reinterpret_cast<const T*>(p.k_bias), p.nk * p.dim, scratch) /
+    if (p.k_norm) all_k = 1.0f / sqrtf(row_squares<T, VEC>(row + p.k_off, reinterpret_cast<const T*>(p.k_bias), p.nk * p.dim, scratch) /
                                            (float)(p.nk * p.dim) + p.norm_eps);
   }
+  auto turned = [&](int i, float& cs, float& sn) {
+    if constexpr (TABLE) {
+      cs = cos_s[i];
+      sn = sin_s[i];
+    } else {
+      sincosf((float)pos * p.inv_freq[i], &sn, &cs);
+      cs *= p.rot_scale;
+      sn *= p.rot_scale;
+    }
+  };
   for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < p.nq + 2 * p.nk; head += gridDim.y * warps) {
     const bool is_q = head < p.nq, is_v = head >= p.nq + p.nk;
     const int hh = is_q ? head : (is_v ? head - p.nq - p.nk : head - p.nq);
     const int width = is_v ? p.vdim : p.dim;
     const T* src = row + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + (size_t)hh * width;
     const T* bias = reinterpret_cast<const T*>(is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias));
+    if (bias) bias += (size_t)hh * width;
     TO* dst;
     if (is_q) {
       dst = reinterpret_cast<TO*>(p.q_out) + (size_t)n * p.q_out_stride + (size_t)hh * width;
@@ -150,45 +187,105 @@ __global__ void qkv_prepare_kernel(const PrepParams p) {
       dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
                  : reinterpret_cast<TO*>(p.k_out) + (size_t)n * p.k_out_stride + (size_t)hh * width;
     }
+    const float* nw = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
+    if (nw && p.norm_all) nw += (size_t)hh * width;
+    float factor = is_q ? p.q_scale : p.k_scale;
+    if (is_q && p.q_temp_every > 0) factor *= 1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1));
     __syncwarp();                                  // the warp is done with the row of its last head
     float ss = 0.f;
-    for (int d = lane; d < width; d += 32) {
-      float x = to_f32<T>(src[d]);
-      if (bias) x += to_f32<T>(bias[(size_t)hh * width + d]);
-      xs[d] = x;
-      ss = __fmaf_rn(x, x, ss);
-    }
-    if (is_v) {
-      for (int d = lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d]);
+    if constexpr (VEC) {
+      for (int d = lane * 4; d < width; d += 128) {
+        float4 x = load4_f32(src + d);
+        if (bias) {
+          const float4 b = load4_f32(bias + d);
+          x.x += b.x; x.y += b.y; x.z += b.z; x.w += b.w;
+        }
+        if (is_v) store4(dst + d, x);
+        else *reinterpret_cast<float4*>(xs + d) = x;
+        ss += (x.x * x.x + x.y * x.y) + (x.z * x.z + x.w * x.w);
+      }
     } else {
-      const float* nw = is_q ? p.q_norm : p.k_norm;
-      if (nw && p.norm_all) {
-        const float r = is_q ? all_q : all_k;
-        for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[(size_t)hh * width + d];
-      } else if (nw) {
-        ss = warp_sum(ss);
-        const float r = 1.0f / sqrtf(ss / (float)width + p.norm_eps);
-        for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[d];
+      for (int d = lane; d < width; d += 32) {
+        float x = to_f32<T>(src[d]);
+        if (bias) x += to_f32<T>(bias[d]);
+        if (is_v) dst[d] = from_f32<TO>(x);
+        else xs[d] = x;
+        ss = __fmaf_rn(x, x, ss);
+      }
+    }
+    if (!is_v) {
+      if (nw) {
+        const float r = p.norm_all ? (is_q ? all_q : all_k) : 1.0f / sqrtf(warp_sum(ss) / (float)width + p.norm_eps);
+        if constexpr (VEC) {
+          for (int d = lane * 4; d < width; d += 128) {
+            const float4 w = load4_f32(nw + d), x = *reinterpret_cast<const float4*>(xs + d);
+            *reinterpret_cast<float4*>(xs + d) = make_float4(x.x * r * w.x, x.y * r * w.y, x.z * r * w.z, x.w * r * w.w);
+          }
+        } else {
+          for (int d = lane; d < width; d += 32) xs[d] = xs[d] * r * nw[d];
+        }
       }
       __syncwarp();
-      float factor = is_q ? p.q_scale : p.k_scale;
-      if (is_q && p.q_temp_every > 0) factor *= 1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1));
-      const int half = p.inv_freq ? p.rot_dims >> 1 : 0;
-      for (int i = lane; i < half; i += 32) {
-        float sn, cs, o1, o2;
-        sincosf((float)pos * p.inv_freq[i], &sn, &cs);
-        const int a = p.rot_interleaved ? 2 * i : i, b = p.rot_interleaved ? 2 * i + 1 : i + half;
-        rotate_pair(xs[a], xs[b], cs * p.rot_scale, sn * p.rot_scale, o1, o2);
-        dst[a] = from_f32<TO>(o1 * factor);
-        dst[b] = from_f32<TO>(o2 * factor);
+      if constexpr (VEC) {
+        if (p.rot_interleaved) {
+          for (int d = lane * 4; d < 2 * half; d += 128) {
+            const float4 x = *reinterpret_cast<const float4*>(xs + d);
+            float4 o;
+            float cs, sn;
+            turned(d >> 1, cs, sn);
+            rotate_pair(x.x, x.y, cs, sn, o.x, o.y);
+            turned((d >> 1) + 1, cs, sn);
+            rotate_pair(x.z, x.w, cs, sn, o.z, o.w);
+            store4(dst + d, make_float4(o.x * factor, o.y * factor, o.z * factor, o.w * factor));
+          }
+        } else {
+          // two pairs a lane: a rotation of 64 sizes keeps the whole warp busy
+          for (int i = lane * 2; i < half; i += 64) {
+            const float2 a = *reinterpret_cast<const float2*>(xs + i), b = *reinterpret_cast<const float2*>(xs + i + half);
+            float2 oa, ob;
+            float cs, sn;
+            turned(i, cs, sn);
+            rotate_pair(a.x, b.x, cs, sn, oa.x, ob.x);
+            turned(i + 1, cs, sn);
+            rotate_pair(a.y, b.y, cs, sn, oa.y, ob.y);
+            store2(dst + i, make_float2(oa.x * factor, oa.y * factor));
+            store2(dst + i + half, make_float2(ob.x * factor, ob.y * factor));
+          }
+        }
+        for (int d = 2 * half + lane * 4; d < width; d += 128) {
+          const float4 x = *reinterpret_cast<const float4*>(xs + d);
+          store4(dst + d, make_float4(x.x * factor, x.y * factor, x.z * factor, x.w * factor));
+        }
+      } else {
+        for (int i = lane; i < half; i += 32) {
+          float sn, cs, o1, o2;
+          turned(i, cs, sn);
+          const int a = p.rot_interleaved ? 2 * i : i, b = p.rot_interleaved ? 2 * i + 1 : i + half;
+          rotate_pair(xs[a], xs[b], cs, sn, o1, o2);
+          dst[a] = from_f32<TO>(o1 * factor);
+          dst[b] = from_f32<TO>(o2 * factor);
+        }
+        for (int d = 2 * half + lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d] * factor);
       }
-      for (int d = 2 * half + lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d] * factor);
     }
     if (p.pool > 0 && !is_q && (pos + 1) % p.pool == 0) {
       __syncwarp();                                // the row that this warp has just stored ends a block
       store_block_mean<TO>(p, req, pos, hh, is_v, lane);
     }
   }
+}
+
+template <typename T, typename TO>
+int launch_qkv_prepare(const PrepParams& p, dim3 grid, int warps, bool table, bool vec, cudaStream_t stream) {
+  const int row_floats = ((p.dim > p.vdim ? p.dim : p.vdim) + 3) & ~3;
+  size_t smem = (size_t)warps * row_floats * sizeof(float);
+  if (table) smem += 2 * (size_t)((p.rot_dims / 2 + 3) & ~3) * sizeof(float);
+  if (smem > 48 * 1024) return YALIS_ERR_SHAPE;
+  const dim3 block(32 * warps);
+  if (table) return vec ? yalis_launch(qkv_prepare_kernel<T, TO, true, true>, grid, block, smem, stream, p)
+                        : yalis_launch(qkv_prepare_kernel<T, TO, true, false>, grid, block, smem, stream, p);
+  return vec ? yalis_launch(qkv_prepare_kernel<T, TO, false, true>, grid, block, smem, stream, p)
+             : yalis_launch(qkv_prepare_kernel<T, TO, false, false>, grid, block, smem, stream, p);
 }
 
 // ACT: 0 gelu with erf, 1 gelu with tanh, 2 silu, 3 the square of relu, 4 tanh.
@@ -351,18 +448,23 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   p.pool = single_tokens ? pool : 0;
   p.pk_pool = pk_pool; p.pv_pool = pv_pool; p.pool_table = pool_table; p.pool_table_width = pool_table_width;
   p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
-  const int warps = 4;
-  // a norm over all heads is summed by every block anew: with tokens enough to fill the GPU one block walks all heads
-  const int by = norm_all && n_tokens >= 2 * yalis_sm_count() ? 1 : (nq + 2 * nk + warps - 1) / warps;
-  const dim3 grid(n_tokens, by);
-  const size_t smem = (size_t)warps * (dim > vdim ? dim : vdim) * sizeof(float);
+  // Steps of many tokens: a block of eight warps walks all heads of its token, which shares the sines and cosines and
+  // the sums of a norm over all heads.  Few tokens: four heads a block, so that more blocks run at once.
+  const bool per_token = n_tokens >= 2 * yalis_sm_count() && dim <= 512 && vdim <= 512;
+  const int warps = per_token ? 8 : 4;
+  const dim3 grid(n_tokens, per_token ? 1 : (nq + 2 * nk + warps - 1) / warps);
+  const bool table = per_token && inv_freq != nullptr;
+  const uintptr_t ptrs = (uintptr_t)src | (uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)v_bias | (uintptr_t)q_norm |
+                         (uintptr_t)k_norm | (uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out | (uintptr_t)k_pool |
+                         (uintptr_t)v_pool;
+  const bool vec = ((dim | vdim | rot_dims | src_stride | q_off | k_off | v_off | q_out_stride | k_out_stride | v_out_stride) & 3) == 0 &&
+                   (ptrs & 15) == 0;
   int st;
-  if (dtype == YALIS_F32 && out_dtype == YALIS_F32)
-    st = yalis_launch(qkv_prepare_kernel<float, float>, grid, dim3(32 * warps), smem, stream, p);
+  if (dtype == YALIS_F32 && out_dtype == YALIS_F32) st = launch_qkv_prepare<float, float>(p, grid, warps, table, vec, stream);
   else if (dtype == YALIS_BF16 && out_dtype == YALIS_BF16)
-    st = yalis_launch(qkv_prepare_kernel<__nv_bfloat16, __nv_bfloat16>, grid, dim3(32 * warps), smem, stream, p);
+    st = launch_qkv_prepare<__nv_bfloat16, __nv_bfloat16>(p, grid, warps, table, vec, stream);
   else if (dtype == YALIS_BF16 && out_dtype == YALIS_F32)
-    st = yalis_launch(qkv_prepare_kernel<__nv_bfloat16, float>, grid, dim3(32 * warps), smem, stream, p);
+    st = launch_qkv_prepare<__nv_bfloat16, float>(p, grid, warps, table, vec, stream);
   else
     return YALIS_ERR_DTYPE;
   if (st != YALIS_OK || pool == 0 || single_tokens) return st;

@@ -40,56 +40,143 @@ __device__ __forceinline__ float sigmoid_f(float x) { return 1.0f / (1.0f + expf
 // g = exp(-exp(a_log[h]) * softplus(a_raw + dt_bias)) (per head, or per head and key channel) and the write
 // strength are computed beside it, in float32: beta = sigmoid(b_raw), or without b_raw (one column of a_raw per
 // head) the step size itself, beta = softplus(a_raw + dt_bias).  With conv_bias y_t[c] = silu(conv_bias[c] + ...).
+// A block takes a tile of consecutive tokens and a piece of the channels; a thread walks the tile with the last K-1
+// inputs of its channels in registers.  In steps of single tokens it also writes the new tail (`single`); otherwise
+// short_conv_tail_kernel does, once every block has read the old one.
 constexpr int kMaxTaps = 16;
 
-template <typename T>
-__global__ void delta_prepare_kernel(const T* __restrict__ x, int x_stride, const float* __restrict__ w,
-                                     const float* __restrict__ tail, size_t slot_stride,
-                                     const int32_t* __restrict__ req_of_token, const int32_t* __restrict__ q_start,
-                                     const int32_t* __restrict__ slots, float* __restrict__ out, int out_stride,
-                                     int channels, int taps, int kv_heads, int dim, float q_scale, float unit_eps,
-                                     const T* __restrict__ a_raw, int a_stride, int a_cols,
-                                     const float* __restrict__ a_log, const float* __restrict__ dt_bias,
-                                     const T* __restrict__ b_raw, int b_stride, int heads, float* __restrict__ g_out,
-                                     float* __restrict__ beta_out, const float* __restrict__ conv_bias) {
+struct DeltaPrepareParams {
+  const void* x; int x_stride;
+  const float* w; const float* conv_bias;
+  float* tail; size_t slot_stride;
+  const int32_t* req_of_token; const int32_t* q_start; const int32_t* slots;
+  float* out; int out_stride;
+  int n_tokens, channels, taps, tile, piece, single;
+  int kv_heads, dim; float q_scale, unit_eps;
+  const void* a_raw; int a_stride, a_cols; const float* a_log; const float* dt_bias;
+  const void* b_raw; int b_stride, heads;
+  float* g_out; float* beta_out;
+};
+
+// V neighbouring inputs as float32 (V = 2: one 4- or 8-byte load).
+template <typename T, int V>
+__device__ __forceinline__ void load_inputs(const T* p, float (&o)[V]) {
+  if constexpr (V == 2) {
+    if constexpr (sizeof(T) == 2) {
+      const float2 f = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p));
+      o[0] = f.x; o[1] = f.y;
+    } else {
+      const float2 f = *reinterpret_cast<const float2*>(p);
+      o[0] = f.x; o[1] = f.y;
+    }
+  } else {
+    o[0] = to_f32<T>(p[0]);
+  }
+}
+
+// KMAX: the most taps (a bound known at compile time keeps the history in registers); V: channels a thread takes.
+template <typename T, int KMAX, int V>
+__global__ void delta_prepare_kernel(const DeltaPrepareParams p) {
   pdl_launch_dependents();
   pdl_wait();
-  const int n = blockIdx.x;
-  const int req = req_of_token[n];
-  if (req < 0) return;
-  const int i = n - q_start[req];                 // index of the token in its request's portion
-  const float* tl = tail + (size_t)slots[req] * slot_stride;
-  float* row = out + (size_t)n * out_stride;
-  for (int c = threadIdx.x; c < channels; c += blockDim.x) {
-    float acc = 0.f;
-    for (int j = taps - 1; j >= 0; --j) {         // oldest input first: a fixed order of additions
-      float xv;
-      if (i - j >= 0) xv = to_f32<T>(x[(size_t)(n - j) * x_stride + c]);
-      else xv = tl[(size_t)c * (taps - 1) + (taps - 1 + i - j)];
-      acc = __fmaf_rn(w[(size_t)c * taps + (taps - 1 - j)], xv, acc);
+  const int n0 = blockIdx.x * p.tile, n1 = min(n0 + p.tile, p.n_tokens);
+  const int c_begin = blockIdx.y * p.piece, c_end = min(c_begin + p.piece, p.channels);
+  const int keep = p.taps - 1;
+  for (int c = c_begin + (int)threadIdx.x * V; c < c_end; c += (int)blockDim.x * V) {
+    float w[KMAX][V], bias[V], hist[KMAX][V];      // place m: the input KMAX - 1 - m tokens back (the last place is unused in hist)
+#pragma unroll
+    for (int v = 0; v < V; ++v) {
+      bias[v] = p.conv_bias ? p.conv_bias[c + v] : 0.f;
+#pragma unroll
+      for (int m = 0; m < KMAX; ++m) {
+        const int lag = KMAX - 1 - m;
+        w[m][v] = lag < p.taps ? p.w[(size_t)(c + v) * p.taps + (p.taps - 1 - lag)] : 0.f;
+        hist[m][v] = 0.f;
+      }
     }
-    row[c] = silu_exact(conv_bias ? acc + conv_bias[c] : acc);
-  }
-  if (a_raw != nullptr) {
-    const int per = a_cols / heads;               // 1, or dim
-    for (int c = threadIdx.x; c < a_cols; c += blockDim.x) {
-      const float step = softplus_f(to_f32<T>(a_raw[(size_t)n * a_stride + c]) + dt_bias[c]);
-      g_out[(size_t)n * a_cols + c] = expf(-expf(a_log[c / per]) * step);
-      if (b_raw == nullptr) beta_out[(size_t)n * heads + c] = step;
+    bool follows = false;                          // hist holds the inputs before token n
+    for (int n = n0; n < n1; ++n) {
+      const int req = p.req_of_token[n];
+      if (req < 0) {
+        follows = false;
+        continue;
+      }
+      const int i = n - p.q_start[req];            // index of the token in its request's portion
+      const T* xr = reinterpret_cast<const T*>(p.x) + (size_t)n * p.x_stride + c;
+      float* tl = p.tail + (size_t)p.slots[req] * p.slot_stride + (size_t)c * keep;
+      if (!follows || i == 0) {
+#pragma unroll
+        for (int m = 0; m < KMAX - 1; ++m) {
+          const int lag = KMAX - 1 - m;
+          if (lag <= keep) {
+            if (i >= lag) {
+              load_inputs<T, V>(xr - (size_t)lag * p.x_stride, hist[m]);
+            } else {
+#pragma unroll
+              for (int v = 0; v < V; ++v) hist[m][v] = tl[(size_t)v * keep + (keep + i - lag)];
+            }
+          }
+        }
+      }
+      load_inputs<T, V>(xr, hist[KMAX - 1]);
+      float y[V];
+#pragma unroll
+      for (int v = 0; v < V; ++v) {
+        float acc = 0.f;
+#pragma unroll
+        for (int m = 0; m < KMAX; ++m) acc = __fmaf_rn(w[m][v], hist[m][v], acc);     // oldest input first: a fixed order
+        y[v] = silu_exact(acc + bias[v]);
+      }
+      float* o = p.out + (size_t)n * p.out_stride + c;
+      if constexpr (V == 2) *reinterpret_cast<float2*>(o) = make_float2(y[0], y[1]);
+      else o[0] = y[0];
+#pragma unroll
+      for (int m = 0; m < KMAX - 1; ++m)
+#pragma unroll
+        for (int v = 0; v < V; ++v) hist[m][v] = hist[m + 1][v];
+      follows = true;
+      if (p.single) {
+#pragma unroll
+        for (int m = 0; m < KMAX - 1; ++m) {
+          const int lag = KMAX - 1 - m;            // after the shift: the input lag - 1 tokens back
+          if (lag <= keep)
+#pragma unroll
+            for (int v = 0; v < V; ++v) tl[(size_t)v * keep + (keep - lag)] = hist[m][v];
+        }
+      }
     }
-    for (int h = threadIdx.x; b_raw != nullptr && h < heads; h += blockDim.x)
-      beta_out[(size_t)n * heads + h] = sigmoid_f(to_f32<T>(b_raw[(size_t)n * b_stride + h]));
   }
-  if (kv_heads > 0) {
+  if (p.a_raw != nullptr) {
+    const T* a_raw = reinterpret_cast<const T*>(p.a_raw);
+    const T* b_raw = reinterpret_cast<const T*>(p.b_raw);
+    const int per = p.a_cols / p.heads;           // 1, or dim
+    const int first = blockIdx.y * blockDim.x + threadIdx.x, step = gridDim.y * blockDim.x;
+    for (int e = first; e < (n1 - n0) * p.a_cols; e += step) {
+      const int n = n0 + e / p.a_cols, c = e % p.a_cols;
+      if (p.req_of_token[n] < 0) continue;
+      const float s = softplus_f(to_f32<T>(a_raw[(size_t)n * p.a_stride + c]) + p.dt_bias[c]);
+      p.g_out[(size_t)n * p.a_cols + c] = expf(-expf(p.a_log[c / per]) * s);
+      if (b_raw == nullptr) p.beta_out[(size_t)n * p.heads + c] = s;
+    }
+    for (int e = first; b_raw != nullptr && e < (n1 - n0) * p.heads; e += step) {
+      const int n = n0 + e / p.heads, h = e % p.heads;
+      if (p.req_of_token[n] >= 0) p.beta_out[(size_t)n * p.heads + h] = sigmoid_f(to_f32<T>(b_raw[(size_t)n * p.b_stride + h]));
+    }
+  }
+  if (p.kv_heads > 0) {
     __syncthreads();                              // the block reads back what it wrote itself
     const int lane = threadIdx.x & 31, nw = blockDim.x >> 5;
-    for (int hh = threadIdx.x >> 5; hh < 2 * kv_heads; hh += nw) {     // q heads, then k heads
-      float* v = row + (size_t)hh * dim;
+    // the heads of q, then of k, that lie in this piece (a piece is a multiple of dim channels)
+    const int h0 = c_begin / p.dim, h1 = min(c_end, 2 * p.kv_heads * p.dim) / p.dim;
+    for (int e = threadIdx.x >> 5; e < (n1 - n0) * max(h1 - h0, 0); e += nw) {
+      const int n = n0 + e / (h1 - h0), hh = h0 + e % (h1 - h0);
+      if (p.req_of_token[n] < 0) continue;
+      float* v = p.out + (size_t)n * p.out_stride + (size_t)hh * p.dim;
       float ss = 0.f;
-      for (int d = lane; d < dim; d += 32) ss = __fmaf_rn(v[d], v[d], ss);
+      for (int d = lane; d < p.dim; d += 32) ss = __fmaf_rn(v[d], v[d], ss);
       ss = warp_sum(ss);
-      const float r = (hh < kv_heads ? q_scale : 1.0f) / sqrtf(ss + unit_eps);
-      for (int d = lane; d < dim; d += 32) v[d] *= r;
+      const float r = (hh < p.kv_heads ? p.q_scale : 1.0f) / sqrtf(ss + p.unit_eps);
+      for (int d = lane; d < p.dim; d += 32) v[d] *= r;
     }
   }
 }
@@ -497,6 +584,7 @@ YALIS_API int yalis_general_delta_prepare(const void* q, const void* k, const vo
 }
 
 // b_raw null (with a_raw [N, heads]): beta_out receives the step sizes softplus(a_raw + dt_bias).
+// single_tokens: no request brings more than one token (the tails are then written by the same kernel).
 // a_raw null: no decay and write strength are computed.  kv_heads 0: no head is brought to unit length.
 YALIS_API int yalis_delta_prepare(const void* x, int dtype, int x_stride, const float* w, float* tail,
                                   int64_t slot_stride, const int32_t* req_of_token, const int32_t* q_start,
@@ -504,20 +592,36 @@ YALIS_API int yalis_delta_prepare(const void* x, int dtype, int x_stride, const 
                                   int channels, int taps, int kv_heads, int dim, float q_scale, float unit_eps,
                                   const void* a_raw, int a_stride, int a_cols, const float* a_log, const float* dt_bias,
                                   const void* b_raw, int b_stride, int heads, float* g_out, float* beta_out,
-                                  const float* conv_bias, cudaStream_t stream) {
+                                  const float* conv_bias, int single_tokens, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
   if (taps < 1 || taps > kMaxTaps || channels <= 0 || kv_heads < 0 || 2 * kv_heads * dim > channels) return YALIS_ERR_SHAPE;
   if (a_raw && (heads <= 0 || a_cols % heads || !a_log || !dt_bias || (!b_raw && a_cols != heads) || !g_out || !beta_out)) return YALIS_ERR_SHAPE;
-  const int by = (channels + 127) / 128;
-  const int threads = channels >= 1024 ? 256 : 128;
+  DeltaPrepareParams p;
+  p.x = x; p.x_stride = x_stride; p.w = w; p.conv_bias = conv_bias; p.tail = tail; p.slot_stride = (size_t)slot_stride;
+  p.req_of_token = req_of_token; p.q_start = q_start; p.slots = slots; p.out = out; p.out_stride = out_stride;
+  p.n_tokens = n_tokens; p.channels = channels; p.taps = taps; p.single = single_tokens;
+  p.kv_heads = kv_heads; p.dim = dim; p.q_scale = q_scale; p.unit_eps = unit_eps;
+  p.a_raw = a_raw; p.a_stride = a_stride; p.a_cols = a_cols; p.a_log = a_log; p.dt_bias = dt_bias;
+  p.b_raw = b_raw; p.b_stride = b_stride; p.heads = heads; p.g_out = g_out; p.beta_out = beta_out;
+  const size_t element = dtype == YALIS_BF16 ? 2 : 4;
+  const bool pairs = channels % 2 == 0 && x_stride % 2 == 0 && out_stride % 2 == 0 && ((uintptr_t)x % (2 * element)) == 0 &&
+                     ((uintptr_t)out & 7) == 0 && (kv_heads == 0 || dim % 2 == 0);
+  const int v = pairs ? 2 : 1, threads = n_tokens >= 512 ? 256 : 128;
+  // a piece holds whole heads where heads are brought to unit length
+  p.piece = kv_heads > 0 ? (threads * v + dim - 1) / dim * dim : threads * v;
+  p.tile = n_tokens >= 1024 ? 8 : (n_tokens >= 256 ? 2 : 1);
+  const dim3 grid((n_tokens + p.tile - 1) / p.tile, (channels + p.piece - 1) / p.piece);
+  if (grid.y > 65535) return YALIS_ERR_SHAPE;
   YALIS_DISPATCH_DTYPE(dtype, T, {
-    int st = yalis_launch(delta_prepare_kernel<T>, dim3(n_tokens), dim3(threads), 0, stream, (const T*)x, x_stride, w,
-                          (const float*)tail, (size_t)slot_stride, req_of_token, q_start, slots, out, out_stride, channels,
-                          taps, kv_heads, dim, q_scale, unit_eps, (const T*)a_raw, a_stride, a_cols, a_log, dt_bias,
-                          (const T*)b_raw, b_stride, heads, g_out, beta_out, conv_bias);
-    if (st != YALIS_OK || taps == 1) return st;
-    return yalis_launch(short_conv_tail_kernel<T>, dim3(n_requests, by), dim3(128), 0, stream, (const T*)x, x_stride,
-                        tail, (size_t)slot_stride, q_start, slots, channels, taps);
+    int st;
+    if (taps <= 4)
+      st = pairs ? yalis_launch(delta_prepare_kernel<T, 4, 2>, grid, dim3(threads), 0, stream, p)
+                 : yalis_launch(delta_prepare_kernel<T, 4, 1>, grid, dim3(threads), 0, stream, p);
+    else
+      st = yalis_launch(delta_prepare_kernel<T, kMaxTaps, 1>, grid, dim3(threads), 0, stream, p);
+    if (st != YALIS_OK || taps == 1 || single_tokens) return st;
+    return yalis_launch(short_conv_tail_kernel<T>, dim3(n_requests, (channels + 127) / 128), dim3(128), 0, stream, (const T*)x,
+                        x_stride, tail, (size_t)slot_stride, q_start, slots, channels, taps);
   });
   return YALIS_OK;
 }

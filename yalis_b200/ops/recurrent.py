@@ -59,7 +59,8 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
                   req_of_token: torch.Tensor, q_start: torch.Tensor, slots: torch.Tensor, *, unit_heads: int = 0,
                   dim: int = 0, q_scale: float = 1.0, unit_eps: float = 1e-6, a_raw: Optional[torch.Tensor] = None,
                   a_log: Optional[torch.Tensor] = None, dt_bias: Optional[torch.Tensor] = None,
-                  b_raw: Optional[torch.Tensor] = None, conv_bias: Optional[torch.Tensor] = None):
+                  b_raw: Optional[torch.Tensor] = None, conv_bias: Optional[torch.Tensor] = None,
+                  single_tokens: bool = False):
     """What a delta rule reads, in one kernel: silu of a causal convolution over time, per channel, continuing each
     request from the tail its slot keeps; the heads of q and k brought to unit length; decay and write strength.
 
@@ -69,7 +70,8 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
     x / sqrt(sum x^2 + unit_eps), q times ``q_scale``.  With ``a_raw`` ([N, heads] or [N, heads * dim]), ``a_log``
     [heads], ``dt_bias`` (one per column of a_raw) and ``b_raw`` [N, heads]: g = exp(-exp(a_log) softplus(a_raw +
     dt_bias)) and beta = sigmoid(b_raw); without ``b_raw`` (``a_raw`` [N, heads]) beta is the step size softplus(a_raw +
-    dt_bias) itself.  ``conv_bias`` (float32 [C]) is added to the convolution before its silu.  Returns (float32 [N, C], g, beta), g and beta float32 or None; afterwards
+    dt_bias) itself.  ``conv_bias`` (float32 [C]) is added to the convolution before its silu.
+    ``single_tokens``: no request brings more than one token (one launch instead of two).  Returns (float32 [N, C], g, beta), g and beta float32 or None; afterwards
     the tails hold the last ``taps - 1`` inputs of every request."""
     name = "delta_prepare"
     need_cuda(name, x, weight, slot_rows, req_of_token, q_start, slots, a_raw, a_log, dt_bias, b_raw, conv_bias)
@@ -106,7 +108,7 @@ def delta_prepare(x: torch.Tensor, weight: torch.Tensor, slot_rows: torch.Tensor
         ptr(req_of_token), ptr(q_start), ptr(slots), ptr(out), i32(c), i32(n), i32(slots.numel()), i32(c), i32(taps),
         i32(unit_heads), i32(dim), f32(q_scale), f32(unit_eps), ptr(a_raw), i32(a_raw.stride(0) if a_raw is not None else 0),
         i32(a_cols), ptr(a_log), ptr(dt_bias), ptr(b_raw), i32(b_raw.stride(0) if b_raw is not None else 0), i32(heads),
-        ptr(g), ptr(beta), ptr(conv_bias), stream()), name)
+        ptr(g), ptr(beta), ptr(conv_bias), i32(int(single_tokens)), stream()), name)
     return out, g, beta
 
 

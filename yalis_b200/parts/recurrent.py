@@ -193,7 +193,8 @@ class GatedDelta(_ProjectedMixer):
         conv, decay, beta = rec_ops.delta_prepare(
             self._block(z, "qkv"), self.conv_w, cache.state, self.layout.state_floats, ctx.req_of_token, ctx.q_start, ctx.slots,
             unit_heads=self.g, dim=self.d, q_scale=self.d ** -0.5, unit_eps=self.UNIT_EPS, a_raw=a_raw, a_log=self.a_log,
-            dt_bias=self.dt_bias, b_raw=self._block(z, "b"))
+            dt_bias=self.dt_bias, b_raw=self._block(z, "b"),
+            single_tokens=ctx.host.max_q_len == 1)
         o = rec_ops.state_scan(conv[:, :gd], conv[:, gd:2 * gd], conv[:, 2 * gd:], cache.state, self.layout, ctx.q_start,
                                ctx.slots, kv_heads=self.g, decay=decay, beta=beta, max_q_len=ctx.host.max_q_len)
         if self.gate_kind == "silu":
@@ -321,7 +322,8 @@ class StateSpace(_ProjectedMixer):
         blk = lambda name: z[:, self.spans[name][0]:self.spans[name][1]]
         conv, decay, step = rec_ops.delta_prepare(
             blk("xbc"), self.conv_w, cache.state, self.layout.state_floats, ctx.req_of_token, ctx.q_start, ctx.slots,
-            a_raw=blk("step"), a_log=self.a_log, dt_bias=self.dt_bias, conv_bias=self.conv_b)
+            a_raw=blk("step"), a_log=self.a_log, dt_bias=self.dt_bias, conv_bias=self.conv_b,
+            single_tokens=ctx.host.max_q_len == 1)
         b, c = self.inner, self.inner + self.g * self.n
         o = rec_ops.state_scan(conv[:, c:], conv[:, b:c], conv[:, :b], cache.state, self.layout, ctx.q_start, ctx.slots,
                                kv_heads=self.g, decay=decay, beta=step, selective=True, skip=self.skip,
