@@ -34,7 +34,7 @@
 // P is split into its bfloat16 rounding and the bfloat16 rounding of the rest, and both
 // halves go through the tensor cores (the sum of the weights is float32 in either form).
 //
-// The extended form (FORM 2) is the general form with head sizes that are known at launch only
+// The extended form (FORM 2 and 3) is the general form with head sizes that are known at launch only
 // (keys and values may differ; both multiples of 8, padded to one of three tile widths), a
 // learned bias per head and distance added to the scaled score, and pooled blocks: beside the
 // keys of its window a row sees one key and value for every block of P positions that lies
@@ -74,11 +74,11 @@ struct AttnParams {
   const __nv_bfloat16* gate;   // GEN: [N, gate_stride] the result is multiplied by sigmoid(gate[t, head, :]) (null: not)
   int gate_stride;
   int gate_per_head;           // GEN: the gate is [N, nh], one number per head
-  int hs, vs;                  // FORM 2: sizes of a key and a value (multiples of 8, at most HS)
-  const float* rel;            // FORM 2: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
+  int hs, vs;                  // FORM 2, 3: sizes of a key and a value (multiples of 8, at most HS)
+  const float* rel;            // FORM 2, 3: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
   int rel_len;
   int rel_staged;              // the table of a block's heads fits the shared memory set aside for it
-  int pool;                    // FORM 2: P > 0: pooled blocks of P positions before the window
+  int pool;                    // FORM 2, 3: P > 0: pooled blocks of P positions before the window
   const __nv_bfloat16* pk_pool; const __nv_bfloat16* pv_pool;   // [pages, g, pool_page_size, HS / VS], an entry per block
   const int32_t* pool_table;
   int pool_table_width, pool_page_size, pool_num_pages, pool_page_shift;
@@ -91,6 +91,11 @@ struct AttnParams {
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
   const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16;\n" ::"r"(s), "l"(gmem));
+}
+// The same, or 16 zero bytes (nothing is read then, but `gmem` must be an address of the pool).
+__device__ __forceinline__ void cp_async16_or_zero(void* smem, const void* gmem, bool copy) {
+  const unsigned s = (unsigned)__cvta_generic_to_shared(smem);
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;\n" ::"r"(s), "l"(gmem), "r"(copy ? 16 : 0));
 }
 __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;\n" ::); }
 template <int N>
@@ -160,8 +165,8 @@ __device__ __forceinline__ void load_kv_tile(__nv_bfloat16* k_dst, __nv_bfloat16
 
 // The same for the extended form: keys and values of sizes known at launch, columns past them zero, from the token
 // pages or (`pooled`) from the pages of the pooled blocks.
-template <int HS>
-__device__ __forceinline__ void load_kv_tile_sized(__nv_bfloat16* k_dst, __nv_bfloat16* v_dst, const AttnParams& p, int req,
+template <int HS, bool SIZED>
+__device__ __forceinline__ void load_kv_tile_extended(__nv_bfloat16* k_dst, __nv_bfloat16* v_dst, const AttnParams& p, int req,
                                                    int kvh, int key0, int lo_key, int hi_key, bool pooled) {
   constexpr int CHUNKS = HS / 8, LD = HS + 8;
   const int width = pooled ? p.pool_table_width : p.table_width;
@@ -190,10 +195,12 @@ __device__ __forceinline__ void load_kv_tile_sized(__nv_bfloat16* k_dst, __nv_bf
     const int row = c / CHUNKS, ch = c - row * CHUNKS;
     __nv_bfloat16* kd = k_dst + row * LD + ch * 8;
     __nv_bfloat16* vd = v_dst + row * LD + ch * 8;
-    if (at[i] >= 0 && ch * 8 < p.hs) cp_async16(kd, kp + at[i] * p.hs + ch * 8);
-    else *reinterpret_cast<uint4*>(kd) = make_uint4(0u, 0u, 0u, 0u);
-    if (at[i] >= 0 && ch * 8 < p.vs) cp_async16(vd, vp + at[i] * p.vs + ch * 8);
-    else *reinterpret_cast<uint4*>(vd) = make_uint4(0u, 0u, 0u, 0u);
+    const bool row_ok = at[i] >= 0;
+    const long long r = row_ok ? at[i] : 0;
+    const int hs = SIZED ? p.hs : HS, vs = SIZED ? p.vs : HS;
+    const bool k_ok = row_ok && (!SIZED || ch * 8 < hs), v_ok = row_ok && (!SIZED || ch * 8 < vs);
+    cp_async16_or_zero(kd, kp + (k_ok ? r * hs + ch * 8 : 0), k_ok);
+    cp_async16_or_zero(vd, vp + (v_ok ? r * vs + ch * 8 : 0), v_ok);
   }
 }
 
@@ -245,11 +252,12 @@ __device__ __forceinline__ float finish_factor(const AttnParams& p, float m, flo
   return l > 0.f ? (GEN ? p.out_scale : 1.0f) / l : 0.f;
 }
 
-// FORM: 0 plain, 1 general, 2 extended (HS is then the padded size; p.hs and p.vs are the real ones).
+// FORM: 0 plain, 1 general, 2 extended, 3 extended with sizes known at launch (HS is then the padded size; p.hs and p.vs
+// are the real ones).
 template <int HS, bool DEC, int FORM>
 __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const AttnParams p) {
-  constexpr bool GEN = FORM >= 1, EXT = FORM == 2;
-  const int hs = EXT ? p.hs : HS, vs = EXT ? p.vs : HS;
+  constexpr bool GEN = FORM >= 1, EXT = FORM >= 2, SIZED = FORM == 3;
+  const int hs = SIZED ? p.hs : HS, vs = SIZED ? p.vs : HS;
   constexpr int LD = HS + 8;            // padded row: ldmatrix rows fall into distinct banks
   constexpr int KSTEPS = HS / 16;       // k-steps of Q K^T
   constexpr int DT = HS / 8;            // n8 tiles of the output along the head dimension
@@ -310,8 +318,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     __nv_bfloat16* kd = k_s + buf * BN * LD;
     __nv_bfloat16* vd = v_s + buf * BN * LD;
     if constexpr (EXT) {
-      if (tile < pool_tiles) load_kv_tile_sized<HS>(kd, vd, p, req, kvh, tile * BN, 0, nb_last - 1, true);
-      else load_kv_tile_sized<HS>(kd, vd, p, req, kvh, (first_key_tile + tile - pool_tiles) * BN, lo_key, hi_key, false);
+      if (tile < pool_tiles) load_kv_tile_extended<HS, SIZED>(kd, vd, p, req, kvh, tile * BN, 0, nb_last - 1, true);
+      else load_kv_tile_extended<HS, SIZED>(kd, vd, p, req, kvh, (first_key_tile + tile - pool_tiles) * BN, lo_key, hi_key, false);
     } else {
       load_kv_tile<HS>(kd, vd, bt, p, kvh, tile * BN, lo_key, hi_key);
     }
@@ -324,7 +332,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       const int r = c / CHUNKS, ch = c - r * CHUNKS;
       const int row = row0 + r;
       __nv_bfloat16* d = q_s + r * LD + ch * 8;
-      if (row < n_rows && (!EXT || ch * 8 < hs)) {
+      if (row < n_rows && (!SIZED || ch * 8 < hs)) {
         const int t = row / p.per, h = row - t * p.per;
         cp_async16(d, p.q + (size_t)(tok0 + t) * p.q_stride + (size_t)(kvh * p.per + h) * hs + ch * 8);
       } else {
@@ -395,7 +403,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     for (int j = 0; j < ST; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < KSTEPS; ++ks) {
-      if (EXT && ks * 16 >= hs) continue;
+      if (SIZED && ks * 16 >= hs) continue;
 #pragma unroll
       for (int j = 0; j < ST; j += 2) {
         unsigned kb[4];
@@ -480,7 +488,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       for (int kk = 0; kk < ST / 2; ++kk) {
 #pragma unroll
         for (int d = 0; d < DT; d += 2) {
-          if (EXT && d * 8 >= vs) continue;
+          if (SIZED && d * 8 >= vs) continue;
           unsigned vb[4];
           const int key = wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
           const int dim = d * 8 + (lane >> 4) * 8;
@@ -522,7 +530,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
         }
 #pragma unroll
         for (int d = 0; d < DT; d += 2) {
-          if (EXT && d * 8 >= vs) continue;
+          if (SIZED && d * 8 >= vs) continue;
           unsigned vb[4];
           const int key = wkey + kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8;
           const int dim = d * 8 + (lane >> 4) * 8;
@@ -660,7 +668,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     __nv_bfloat16* dst = p.out + (size_t)tok * p.out_stride + (size_t)head * vs;
 #pragma unroll
     for (int d = 0; d < DT; ++d) {
-      if (EXT && d * 8 >= vs) continue;
+      if (SIZED && d * 8 >= vs) continue;
       float v0 = o[d][i * 2] * inv, v1 = o[d][i * 2 + 1] * inv;
       if (GEN && p.gate) {
         v0 *= gate_factor(p, tok, head, vs, d * 8 + tig * 2);
@@ -678,7 +686,7 @@ int launch_mode(const AttnParams& args, int n_requests, int max_rows, cudaStream
   constexpr int RB = DEC ? 16 : BM, NST = DEC ? 3 : 2;
   constexpr size_t tiles = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
   // what a staged table of biases may take without costing a resident block
-  constexpr int rel_room = FORM == 2 ? (DEC ? 1024 : 4096) : 0;
+  constexpr int rel_room = FORM >= 2 ? (DEC ? 1024 : 4096) : 0;
   AttnParams p = args;
   p.rel_staged = p.rel != nullptr && p.per * p.rel_len <= rel_room;
   const size_t smem = tiles + (p.rel_staged ? (size_t)p.per * p.rel_len * sizeof(float) : 0);
@@ -706,8 +714,11 @@ int launch(const AttnParams& p, int n_requests, int max_rows, cudaStream_t strea
 
 template <int HS>
 int launch_extended(const AttnParams& p, int n_requests, int max_rows, cudaStream_t stream) {
-  return max_rows <= 16 ? launch_mode<HS, true, 2>(p, n_requests, max_rows, stream)
-                        : launch_mode<HS, false, 2>(p, n_requests, max_rows, stream);
+  if (p.hs == HS && p.vs == HS)
+    return max_rows <= 16 ? launch_mode<HS, true, 2>(p, n_requests, max_rows, stream)
+                          : launch_mode<HS, false, 2>(p, n_requests, max_rows, stream);
+  return max_rows <= 16 ? launch_mode<HS, true, 3>(p, n_requests, max_rows, stream)
+                        : launch_mode<HS, false, 3>(p, n_requests, max_rows, stream);
 }
 
 }  // namespace

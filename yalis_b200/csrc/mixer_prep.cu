@@ -123,7 +123,7 @@ __device__ __forceinline__ float row_squares(const T* row, const T* bias, int co
 // TABLE: the block computes the token's sines and cosines once, in shared memory (steps of many tokens, where a block
 // walks all heads).  VEC: four consecutive values at a time (every row, size and offset a multiple of four, aligned).
 template <typename T, typename TO, bool TABLE, bool VEC>
-__global__ void qkv_prepare_kernel(const PrepParams p) {
+__global__ void __launch_bounds__(256, 5) qkv_prepare_kernel(const PrepParams p) {
   extern __shared__ __align__(16) float xs_all[];   // a row of `row_floats` per warp, then (TABLE) cosines and sines
   __shared__ float scratch[32];
   pdl_launch_dependents();
@@ -164,6 +164,13 @@ __global__ void qkv_prepare_kernel(const PrepParams p) {
       sn *= p.rot_scale;
     }
   };
+  // what all heads of the token share: its cached row (of head 0), the query's factor, whether it ends a block
+  const long long row0 = p.k_pool != nullptr ? paged_row(p.block_table + (size_t)req * p.table_width, p.table_width, p.page_size,
+                                                         p.num_pages, p.nk, 0, pos)
+                                             : 0;
+  const float q_factor = p.q_temp_every > 0 ? p.q_scale * (1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1)))
+                                            : p.q_scale;
+  const bool ends_block = p.pool > 0 && (pos + 1) % p.pool == 0;
   for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < p.nq + 2 * p.nk; head += gridDim.y * warps) {
     const bool is_q = head < p.nq, is_v = head >= p.nq + p.nk;
     const int hh = is_q ? head : (is_v ? head - p.nq - p.nk : head - p.nq);
@@ -175,13 +182,11 @@ __global__ void qkv_prepare_kernel(const PrepParams p) {
     if (is_q) {
       dst = reinterpret_cast<TO*>(p.q_out) + (size_t)n * p.q_out_stride + (size_t)hh * width;
     } else if (p.k_pool != nullptr) {
-      const long long at = paged_row(p.block_table + (size_t)req * p.table_width, p.table_width, p.page_size, p.num_pages, p.nk,
-                                     hh, pos);
-      if (at < 0) {
+      if (row0 < 0) {
         if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
         continue;
       }
-      dst = reinterpret_cast<TO*>(is_v ? p.v_pool : p.k_pool) + at * width;
+      dst = reinterpret_cast<TO*>(is_v ? p.v_pool : p.k_pool) + (row0 + (long long)hh * p.page_size) * width;
     } else {
       if (p.k_out == nullptr) continue;            // nothing keeps this layer's keys and values: queries only
       dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
@@ -189,8 +194,7 @@ __global__ void qkv_prepare_kernel(const PrepParams p) {
     }
     const float* nw = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
     if (nw && p.norm_all) nw += (size_t)hh * width;
-    float factor = is_q ? p.q_scale : p.k_scale;
-    if (is_q && p.q_temp_every > 0) factor *= 1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1));
+    const float factor = is_q ? q_factor : p.k_scale;
     __syncwarp();                                  // the warp is done with the row of its last head
     float ss = 0.f;
     if constexpr (VEC) {
@@ -268,7 +272,7 @@ __global__ void qkv_prepare_kernel(const PrepParams p) {
         for (int d = 2 * half + lane; d < width; d += 32) dst[d] = from_f32<TO>(xs[d] * factor);
       }
     }
-    if (p.pool > 0 && !is_q && (pos + 1) % p.pool == 0) {
+    if (ends_block && !is_q) {
       __syncwarp();                                // the row that this warp has just stored ends a block
       store_block_mean<TO>(p, req, pos, hh, is_v, lane);
     }
