@@ -186,8 +186,10 @@ template <typename T>
 __global__ void short_conv_tail_kernel(const T* __restrict__ x, int x_stride, float* __restrict__ tail,
                                        size_t slot_stride, const int32_t* __restrict__ q_start,
                                        const int32_t* __restrict__ slots, int channels, int taps) {
-  pdl_launch_dependents();
+  // The recurrence that follows holds few blocks that run long: let in while delta_prepare still fills most SMs they
+  // would crowd onto the ones that come free first.
   pdl_wait();
+  pdl_launch_dependents();
   const int req = blockIdx.x;
   const int a = q_start[req], q_len = q_start[req + 1] - a;
   if (q_len <= 0) return;
