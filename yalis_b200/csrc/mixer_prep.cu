@@ -58,9 +58,34 @@ __device__ void store_block_mean(const PrepParams& p, int req, int pos, int head
     return;
   }
   T* dst = reinterpret_cast<T*>(is_v ? p.pv_pool : p.pk_pool) + entry * width;
+  const int first = pos - p.pool + 1, slot = first % p.page_size;
+  const float count = (float)p.pool;
+  if (slot + p.pool <= p.page_size && (width & 3) == 0 && (((uintptr_t)rows | (uintptr_t)p.pk_pool | (uintptr_t)p.pv_pool) & 15) == 0) {
+    // the block lies in one page: its rows follow one another, four values a lane, eight rows in flight
+    const long long row = paged_row(table, p.table_width, p.page_size, p.num_pages, p.nk, head, first);
+    if (row < 0) {
+      if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
+      return;
+    }
+    for (int d = lane * 4; d < width; d += 128) {
+      const T* src = rows + row * width + d;
+      float4 sum = make_float4(0.f, 0.f, 0.f, 0.f);
+      for (int j0 = 0; j0 < p.pool; j0 += 8) {
+        float4 x[8];
+#pragma unroll
+        for (int j = 0; j < 8; ++j) x[j] = j0 + j < p.pool ? load4_f32(src + (j0 + j) * width) : make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+        for (int j = 0; j < 8; ++j) {
+          sum.x += x[j].x; sum.y += x[j].y; sum.z += x[j].z; sum.w += x[j].w;
+        }
+      }
+      store4(dst + d, make_float4(sum.x / count, sum.y / count, sum.z / count, sum.w / count));
+    }
+    return;
+  }
   for (int d0 = 0; d0 < width; d0 += 128) {      // up to four sizes a lane at a time
     float sum[4] = {0.f, 0.f, 0.f, 0.f};
-    for (int at = pos - p.pool + 1; at <= pos; ++at) {
+    for (int at = first; at <= pos; ++at) {
       const long long row = paged_row(table, p.table_width, p.page_size, p.num_pages, p.nk, head, at);
       if (row < 0) {
         if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
@@ -75,24 +100,30 @@ __device__ void store_block_mean(const PrepParams& p, int req, int pos, int head
 #pragma unroll
     for (int i = 0; i < 4; ++i) {
       const int d = d0 + lane + 32 * i;
-      if (d < width) dst[d] = from_f32<T>(sum[i] / (float)p.pool);
+      if (d < width) dst[d] = from_f32<T>(sum[i] / count);
     }
   }
 }
 
-// For steps in which a request brings several tokens: after qkv_prepare has stored them, a warp per (token, key or value
-// head) stores the mean of the block that ends at the token, if one does.
+// For steps in which a request brings several tokens: after qkv_prepare has stored them, a warp per (tile of 32 or fewer
+// tokens, key or value head) looks for the tokens of its tile that end a block and stores those blocks' means.
 template <typename T>
-__global__ void store_block_means_kernel(const PrepParams p) {
+__global__ void store_block_means_kernel(const PrepParams p, int n_tokens, int tile) {
   pdl_launch_dependents();
   pdl_wait();
-  const int n = blockIdx.x, head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5);
+  const int head = blockIdx.y * (blockDim.x >> 5) + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (head >= 2 * p.nk) return;
-  const int req = p.req_of_token[n];
-  if (req < 0) return;
-  const int pos = p.positions[n];
-  if ((pos + 1) % p.pool) return;
-  store_block_mean<T>(p, req, pos, head >= p.nk ? head - p.nk : head, head >= p.nk, threadIdx.x & 31);
+  const int n = blockIdx.x * tile + lane;
+  const bool mine = lane < tile && n < n_tokens;
+  const int req = mine ? p.req_of_token[n] : -1;
+  const int pos = req >= 0 ? p.positions[n] : 0;
+  unsigned ends = __ballot_sync(0xffffffffu, req >= 0 && (pos + 1) % p.pool == 0);
+  while (ends) {
+    const int at = __ffs(ends) - 1;
+    ends &= ends - 1;
+    store_block_mean<T>(p, __shfl_sync(0xffffffffu, req, at), __shfl_sync(0xffffffffu, pos, at),
+                        head >= p.nk ? head - p.nk : head, head >= p.nk, lane);
+  }
 }
 
 // Sum over the block of the squares of `count` values (plus a bias) of a row.
@@ -473,8 +504,9 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
     return YALIS_ERR_DTYPE;
   if (st != YALIS_OK || pool == 0 || single_tokens) return st;
   p.pool = pool;
-  const dim3 means(n_tokens, (2 * nk + warps - 1) / warps);
-  YALIS_DISPATCH_DTYPE(dtype, T, return yalis_launch(store_block_means_kernel<T>, means, dim3(32 * warps), 0, stream, p));
+  const int tile = pool < 32 ? pool : 32;         // about one block's end per tile
+  const dim3 means((n_tokens + tile - 1) / tile, (2 * nk + 3) / 4);
+  YALIS_DISPATCH_DTYPE(dtype, T, return yalis_launch(store_block_means_kernel<T>, means, dim3(128), 0, stream, p, n_tokens, tile));
   return YALIS_OK;
 }
 
