@@ -57,13 +57,13 @@ def test_what_the_mixers_keep():
 
 
 def test_a_group_of_blocks_counts_in_blocks_of_tokens():
-    reqs = [{"tokens": PagedKV(2, 16, 40), "blocks": PagedKV(2, 16, None, pool=8)}, PagedKV(1, 8)]
+    reqs = [{"tokens": PagedKV(2, 16, 44), "blocks": PagedKV(2, 16, None, pool=8)}, PagedKV(1, 8)]
     groups = {g.name: g for g in plan_groups(reqs, 16, 50, 400, max_slots=3, step_tokens=64)}
     blocks = groups["kv_all_pool_8"]
     assert blocks.page_size == 128 and blocks.max_pages_per_request == 4 and blocks.num_pages == 7 + 3
     assert groups["kv_all"].num_pages == 50 and groups["kv_all"].page_size == 16
     size = group_page_bytes(reqs, [None, None], 16, 2)
-    assert size["kv_all_pool_8"] == 2 * 16 * 32 * 2 // 8 and size["kv_window_40"] == 2 * 16 * 32 * 2
+    assert size["kv_all_pool_8"] == 2 * 16 * 32 * 2 // 8 and size["kv_window_44"] == 2 * 16 * 32 * 2
     # the pool holds any requests that fit the tokens' pool: each takes ceil(length / 128) pages
     m = CacheManager(3, [blocks])
     lengths = [398, 370, 4]

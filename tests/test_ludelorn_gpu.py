@@ -97,7 +97,7 @@ def test_heads_are_normed_one_by_one_or_all_at_once_and_turned(dtype, n, nq, nk,
 def test_yarn_frequencies_in_the_rotary_part():
     from yalis_b200.config.spec import PartSpec
     from yalis_b200.parts.base import make_part
-    for dims, base, sc in ((16, 100.0, (4.0, 64, 6.0, 1.0)), (48, 5e5, (2.0, 1024, 32.0, 1.0)), (10, 20.0, (3.0, 16, 2.0, 0.25))):
+    for dims, base, sc in ((16, 100.0, (4.0, 64, 6.0, 1.0)), (40, 4e5, (2.0, 1024, 24.0, 1.0)), (10, 20.0, (3.0, 16, 2.0, 0.25))):
         keys = ("factor", "original", "fast", "slow")
         part = make_part("position", PartSpec("rotary", {"head_dim": dims, "theta": base, "exact_powers": True,
                                                          "scaling": {"kind": "yarn", **dict(zip(keys, sc))}}))
@@ -154,7 +154,7 @@ def attend_rows(q, keys, values, scale, W, **kw):
 CASES = [  # dtype, key size, value size, page, window, block size (None: none), buckets (None: none), heads, kv_heads
     (torch.float32, 12, 20, 16, 9, 4, None, 4, 2), (torch.float32, 8, 8, 8, 30, 30, None, 2, 2), (torch.float32, 10, 10, 4, 1, 1, None, 3, 1),
     (torch.float32, 12, 12, 16, 23, None, 8, 4, 2), (torch.float32, 7, 7, 8, 300, None, 6, 3, 1),
-    (torch.bfloat16, 64, 32, 16, 40, 8, None, 4, 2), (torch.bfloat16, 48, 48, 16, 17, 5, None, 6, 3), (torch.bfloat16, 128, 96, 8, 100, 3, None, 2, 1),
+    (torch.bfloat16, 64, 40, 16, 44, 6, None, 4, 2), (torch.bfloat16, 48, 48, 16, 17, 5, None, 6, 3), (torch.bfloat16, 128, 96, 8, 100, 3, None, 2, 1),
     (torch.bfloat16, 64, 64, 64, 64, 64, None, 4, 2), (torch.bfloat16, 40, 24, 16, 37, None, None, 8, 1), (torch.bfloat16, 24, 24, 16, 50, None, 10, 20, 1),
     (torch.bfloat16, 128, 128, 16, 70, None, 32, 4, 2), (torch.bfloat16, 16, 200, 16, 33, 2, None, 2, 2), (torch.bfloat16, 256, 8, 16, 20, 7, None, 2, 1)]
 

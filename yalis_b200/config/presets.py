@@ -428,7 +428,7 @@ PRESETS["ludelorn-tiny-B"] = _ludelorn(37, 50, [
     _ld_pooled(_ld_heads(2, 1, 6, 11, 0.4, 3, pool=4, rot=(6, 9.0)), None)], eps=1e-4)
 PRESETS["ludelorn-tiny-C"] = _ludelorn(128, 160, [
     _ld_parallel(_ld_heads(4, 2, 64, 32, 0.125, 33, rot=(32, 10000.0), yarn=(4.0, 256, 16.0, 1.0)), (4, 32, 128, 2, 4, 4), 256),
-    _ld_pooled(_ld_heads(4, 4, 64, 64, 0.14, 40, pool=8, rot=(64, 1000.0)), 128),
+    _ld_pooled(_ld_heads(4, 4, 64, 64, 0.14, 45, pool=10, rot=(64, 1000.0)), 128),
     _ld_biased(8, 2, 16, 0.25, 70, 16, 50, 256),
     _ld_pooled(_ld_heads(2, 1, 128, 96, 0.09, 16, pool=16, rot=(64, 10000.0)), 256),
     _ld_biased(2, 1, 128, 0.09, 20, 32, 64, 128)], scale=3.0)
