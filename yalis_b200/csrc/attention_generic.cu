@@ -19,6 +19,9 @@
 // block of P positions that lies wholly before it, blocks b < floor((pos - window + 1) / P); they come from pools of
 // their own (entry b of the request's block table over entries) and share the softmax with the window's keys.
 // Values may have a head size of their own (hsv).
+// Two maps (maps = 2): a query head has two queries and a key/value head two keys per position (each of size hs, side by
+// side in the query matrix and in a cached row of 2 hs), and one value; each map is a softmax of its own over the visible
+// keys.  With O1, O2 the maps' results  O = O1 - lambda * O2,  O <- O / sqrt(mean(O^2) + eps) * out_scale.
 // Mask by absolute position: yalis/attention/backend_impl/sdpa_and_flex.py:15-19, 301-307.
 // KV head of query head h: h / (nh / g)                                 (:59-67).
 #include "common.cuh"
@@ -42,11 +45,12 @@ struct GenericParams {
   int pool;                                      // P > 0: pooled blocks before the window
   const T* pk_pool; const T* pv_pool; const int32_t* pool_table;
   int pool_table_width, pool_page_size, pool_num_pages;   // in entries (one per block)
+  float lambda, diff_eps;                        // two maps
 };
 
-template <typename T>
+template <typename T, int MAPS>
 __global__ void paged_attention_generic_kernel(const GenericParams<T> p) {
-  extern __shared__ float smem[];  // [kWarps][hsv] accumulators, then m[kWarps], l[kWarps]
+  extern __shared__ float smem[];  // per map [kWarps][hsv] accumulators, then m[kWarps], l[kWarps]; two maps: [hsv] besides
   pdl_launch_dependents();
   pdl_wait();
   const int t = blockIdx.x, h = blockIdx.y;
@@ -57,15 +61,22 @@ __global__ void paged_attention_generic_kernel(const GenericParams<T> p) {
   const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
   const int per_lane = (p.hs + 31) >> 5, per_lane_v = (p.hsv + 31) >> 5;
 
-  float qr[kMaxPerLane], acc[kMaxPerLane];
-  const T* qp = p.q + (size_t)t * p.q_stride + (size_t)h * p.hs;
+  float qr[MAPS][kMaxPerLane], acc[MAPS][kMaxPerLane];
+  const T* qp = p.q + (size_t)t * p.q_stride + (size_t)h * (MAPS * p.hs);
 #pragma unroll
-  for (int i = 0; i < kMaxPerLane; ++i) {
-    const int d = lane + 32 * i;
-    qr[i] = (i < per_lane && d < p.hs) ? to_f32<T>(qp[d]) : 0.f;
-    acc[i] = 0.f;
+  for (int a = 0; a < MAPS; ++a)
+#pragma unroll
+    for (int i = 0; i < kMaxPerLane; ++i) {
+      const int d = lane + 32 * i;
+      qr[a][i] = (i < per_lane && d < p.hs) ? to_f32<T>(qp[a * p.hs + d]) : 0.f;
+      acc[a][i] = 0.f;
+    }
+  float m[MAPS], l[MAPS];
+#pragma unroll
+  for (int a = 0; a < MAPS; ++a) {
+    m[a] = -INFINITY;
+    l[a] = 0.f;
   }
-  float m = -INFINITY, l = 0.f;
   int lo = (p.window > 0 && pos - p.window + 1 > 0) ? pos - p.window + 1 : 0;
   if (p.chunk > 0) lo = max(lo, (pos / p.chunk) * p.chunk);
   const float slope = p.slopes ? p.slopes[h] : 0.f;
@@ -81,42 +92,85 @@ __global__ void paged_attention_generic_kernel(const GenericParams<T> p) {
     const int page = pi < (pooled ? p.pool_table_width : p.table_width) ? table[pi] : -1;
     if (page < 0 || page >= (pooled ? p.pool_num_pages : p.num_pages)) continue;  // unmapped: treated as masked
     const size_t row = ((size_t)page * p.g + kvh) * ps + (j - pi * ps);
-    const T* kp = (pooled ? p.pk_pool : p.k_pool) + row * p.hs;
+    const T* kp = (pooled ? p.pk_pool : p.k_pool) + row * (MAPS * p.hs);
     const T* vp = (pooled ? p.pv_pool : p.v_pool) + row * p.hsv;
-    float dot = 0.f;
+#pragma unroll
+    for (int a = 0; a < MAPS; ++a) {
+      float dot = 0.f;
+#pragma unroll
+      for (int i = 0; i < kMaxPerLane; ++i) {
+        const int d = lane + 32 * i;
+        if (i < per_lane && d < p.hs) dot += qr[a][i] * to_f32<T>(kp[a * p.hs + d]);
+      }
+      float s = warp_sum(dot) * p.scale;
+      if (p.slopes && !pooled) s -= slope * (float)(pos - j);
+      if (p.rel && !pooled) s += p.rel[(size_t)h * p.rel_len + min(pos - j, p.rel_len - 1)];
+      if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
+      const float m_new = fmaxf(m[a], s);
+      const float corr = expf(m[a] - m_new);
+      const float e = expf(s - m_new);
+      l[a] = l[a] * corr + e;
+#pragma unroll
+      for (int i = 0; i < kMaxPerLane; ++i) {
+        const int d = lane + 32 * i;
+        if (i < per_lane_v && d < p.hsv) acc[a][i] = acc[a][i] * corr + e * to_f32<T>(vp[d]);
+      }
+      m[a] = m_new;
+    }
+  }
+  const int map_floats = kWarps * p.hsv + 2 * kWarps;
+#pragma unroll
+  for (int a = 0; a < MAPS; ++a) {
+    float* acc_w = smem + a * map_floats + warp * p.hsv;
 #pragma unroll
     for (int i = 0; i < kMaxPerLane; ++i) {
       const int d = lane + 32 * i;
-      if (i < per_lane && d < p.hs) dot += qr[i] * to_f32<T>(kp[d]);
+      if (i < per_lane_v && d < p.hsv) acc_w[d] = acc[a][i];
     }
-    float s = warp_sum(dot) * p.scale;
-    if (p.slopes && !pooled) s -= slope * (float)(pos - j);
-    if (p.rel && !pooled) s += p.rel[(size_t)h * p.rel_len + min(pos - j, p.rel_len - 1)];
-    if (p.softcap > 0.f) s = p.softcap * tanhf(s / p.softcap);
-    const float m_new = fmaxf(m, s);
-    const float corr = expf(m - m_new);
-    const float e = expf(s - m_new);
-    l = l * corr + e;
-#pragma unroll
-    for (int i = 0; i < kMaxPerLane; ++i) {
-      const int d = lane + 32 * i;
-      if (i < per_lane_v && d < p.hsv) acc[i] = acc[i] * corr + e * to_f32<T>(vp[d]);
+    if (lane == 0) {
+      smem[a * map_floats + kWarps * p.hsv + warp] = m[a];
+      smem[a * map_floats + kWarps * p.hsv + kWarps + warp] = l[a];
     }
-    m = m_new;
-  }
-  float* acc_s = smem;
-  float* m_s = smem + kWarps * p.hsv;
-  float* l_s = m_s + kWarps;
-#pragma unroll
-  for (int i = 0; i < kMaxPerLane; ++i) {
-    const int d = lane + 32 * i;
-    if (i < per_lane_v && d < p.hsv) acc_s[warp * p.hsv + d] = acc[i];
-  }
-  if (lane == 0) {
-    m_s[warp] = m;
-    l_s[warp] = l;
   }
   __syncthreads();
+  if constexpr (MAPS == 2) {
+    __shared__ float scratch[32];
+    float* o_s = smem + 2 * map_floats;
+    float wgt[2][kWarps];
+#pragma unroll
+    for (int a = 0; a < 2; ++a) {
+      const float* ms = smem + a * map_floats + kWarps * p.hsv;
+      const float* ls = ms + kWarps;
+      float mm = -INFINITY, ll = 0.f;
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) mm = fmaxf(mm, ms[w]);
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) {
+        wgt[a][w] = ms[w] == -INFINITY ? 0.f : expf(ms[w] - mm);
+        ll += ls[w] * wgt[a][w];
+      }
+#pragma unroll
+      for (int w = 0; w < kWarps; ++w) wgt[a][w] = ll > 0.f ? wgt[a][w] / ll : 0.f;
+    }
+    float ss = 0.f;
+    for (int d = threadIdx.x; d < p.hsv; d += blockDim.x) {
+      float o[2] = {0.f, 0.f};
+#pragma unroll
+      for (int a = 0; a < 2; ++a)
+#pragma unroll
+        for (int w = 0; w < kWarps; ++w) o[a] += smem[a * map_floats + w * p.hsv + d] * wgt[a][w];
+      const float v = o[0] - p.lambda * o[1];
+      o_s[d] = v;
+      ss = __fmaf_rn(v, v, ss);
+    }
+    const float r = p.out_scale / sqrtf(block_sum(ss, scratch) / (float)p.hsv + p.diff_eps);
+    T* op = p.out + (size_t)t * p.out_stride + (size_t)h * p.hsv;
+    for (int d = threadIdx.x; d < p.hsv; d += blockDim.x) op[d] = from_f32<T>(o_s[d] * r);
+    return;
+  }
+  const float* acc_s = smem;
+  const float* m_s = smem + kWarps * p.hsv;
+  const float* l_s = m_s + kWarps;
   float mm = -INFINITY;
 #pragma unroll
   for (int w = 0; w < kWarps; ++w) mm = fmaxf(mm, m_s[w]);
@@ -145,6 +199,7 @@ __global__ void paged_attention_generic_kernel(const GenericParams<T> p) {
 
 }  // namespace
 
+// maps 2: two maps, hs the size of one map's queries and keys; no sink, gate or pooled blocks.
 // rel null: no bias per distance.  pool 0: no pooled blocks (the pool_* arguments are not read).
 YALIS_API int yalis_paged_attention_generic(const void* q, int q_stride, void* out, int out_stride,
                                             const void* k_pool, const void* v_pool, int dtype,
@@ -155,14 +210,15 @@ YALIS_API int yalis_paged_attention_generic(const void* q, int q_stride, void* o
                                             int chunk, const float* sink_logits, const float* slopes, const void* gate,
                                             int gate_stride, int gate_per_head, const float* rel, int rel_len, int pool,
                                             const void* pk_pool, const void* pv_pool, const int32_t* pool_table,
-                                            int pool_table_width, int pool_page_size, int pool_num_pages,
-                                            cudaStream_t stream) {
+                                            int pool_table_width, int pool_page_size, int pool_num_pages, int maps,
+                                            float lambda, float diff_eps, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
+  if (maps != 1 && (maps != 2 || sink || gate || pool > 0)) return YALIS_ERR_SHAPE;
   if (hs <= 0 || hs > 32 * kMaxPerLane || hsv <= 0 || hsv > 32 * kMaxPerLane || g <= 0 || nh % g != 0 || nh > 65535)
     return YALIS_ERR_SHAPE;
   if ((rel && rel_len < 1) || pool < 0 || (pool > 0 && (window <= 0 || chunk > 0 || !pk_pool || !pv_pool || !pool_table || pool_page_size < 1)))
     return YALIS_ERR_SHAPE;
-  const size_t smem = ((size_t)kWarps * hsv + 2 * kWarps) * sizeof(float);
+  const size_t smem = (maps * ((size_t)kWarps * hsv + 2 * kWarps) + (maps == 2 ? hsv : 0)) * sizeof(float);
   dim3 grid(n_tokens, nh);
   YALIS_DISPATCH_DTYPE(dtype, T, {
     GenericParams<T> p;
@@ -176,7 +232,9 @@ YALIS_API int yalis_paged_attention_generic(const void* q, int q_stride, void* o
     p.gate = (const T*)gate; p.gate_stride = gate_stride; p.gate_per_head = gate_per_head;
     p.pool = pool; p.pk_pool = (const T*)pk_pool; p.pv_pool = (const T*)pv_pool; p.pool_table = pool_table;
     p.pool_table_width = pool_table_width; p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
-    return yalis_launch(paged_attention_generic_kernel<T>, grid, dim3(kWarps * 32), smem, stream, p);
+    p.lambda = lambda; p.diff_eps = diff_eps;
+    return maps == 2 ? yalis_launch(paged_attention_generic_kernel<T, 2>, grid, dim3(kWarps * 32), smem, stream, p)
+                     : yalis_launch(paged_attention_generic_kernel<T, 1>, grid, dim3(kWarps * 32), smem, stream, p);
   });
   return YALIS_OK;
 }

@@ -40,6 +40,14 @@
 // keys of its window a row sees one key and value for every block of P positions that lies
 // wholly before the window.  The blocks have pools and a block table of their own; their tiles
 // come first, then those of the window, in one softmax.
+//
+// The form of two maps (FORM 4) has two queries per head and two keys per key/value head and position (side by side in a
+// cached row of 2 d sizes) over one value: each map is a softmax of its own, and the result is the first map's minus
+// lambda times the second's, divided by its root mean square, times a factor.  A row is then a (token, head, map): a
+// block takes half as many pairs (token, head) as it has rows, the first half of its rows for the first map and the second
+// half for the second, so a K tile of 2 d columns and its V tile are read once for both.  In prompts a warp's rows belong
+// to one map and it multiplies only that map's half of the columns; in decode steps the rows of both maps share a
+// warp and a row's query is zero in the other map's half.  The maps meet in shared memory, in float32, at the end.
 #include "common.cuh"
 
 namespace {
@@ -74,7 +82,9 @@ struct AttnParams {
   const __nv_bfloat16* gate;   // GEN: [N, gate_stride] the result is multiplied by sigmoid(gate[t, head, :]) (null: not)
   int gate_stride;
   int gate_per_head;           // GEN: the gate is [N, nh], one number per head
-  int hs, vs;                  // FORM 2, 3: sizes of a key and a value (multiples of 8, at most HS)
+  int map_dim;                 // FORM 4: d, the size of one map's query and key (hs = 2 d, a multiple of 32)
+  float lambda, diff_eps;      // FORM 4
+  int hs, vs;                  // FORM 2, 3, 4: sizes of a key and a value (multiples of 8, at most HS)
   const float* rel;            // FORM 2, 3: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
   int rel_len;
   int rel_staged;              // the table of a block's heads fits the shared memory set aside for it
@@ -83,9 +93,9 @@ struct AttnParams {
   const int32_t* pool_table;
   int pool_table_width, pool_page_size, pool_num_pages, pool_page_shift;
   int n_splits;
-  float* part_o;               // [N, nh, n_splits, HS] (split mode)
-  float* part_ml;              // [N, nh, n_splits, 2]
-  int32_t* tickets;            // [R * g] zero before the launch and zero again after it (split mode)
+  float* part_o;               // [N, nh, n_splits, HS] (split mode); FORM 4: [N, nh, 2, n_splits, HS]
+  float* part_ml;              // the same places, 2 floats each
+  int32_t* tickets;            // one per block of a split: zero before the launch and zero again after it (split mode)
 };
 
 __device__ __forceinline__ void cp_async16(void* smem, const void* gmem) {
@@ -253,10 +263,10 @@ __device__ __forceinline__ float finish_factor(const AttnParams& p, float m, flo
 }
 
 // FORM: 0 plain, 1 general, 2 extended, 3 extended with sizes known at launch (HS is then the padded size; p.hs and p.vs
-// are the real ones).
+// are the real ones), 4 two maps (sizes known at launch too; p.hs is that of both maps' keys together).
 template <int HS, bool DEC, int FORM>
 __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const AttnParams p) {
-  constexpr bool GEN = FORM >= 1, EXT = FORM >= 2, SIZED = FORM == 3;
+  constexpr bool GEN = FORM >= 1, EXT = FORM >= 2, SIZED = FORM >= 3, MAPS = FORM == 4;
   const int hs = SIZED ? p.hs : HS, vs = SIZED ? p.vs : HS;
   constexpr int LD = HS + 8;            // padded row: ldmatrix rows fall into distinct banks
   constexpr int KSTEPS = HS / 16;       // k-steps of Q K^T
@@ -264,6 +274,9 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   constexpr int WKEYS = DEC ? BN / NWARPS : BN;   // keys of a tile that one warp handles
   constexpr int ST = WKEYS / 8;         // n8 tiles of S along this warp's keys
   constexpr int RB = DEC ? 16 : BM;     // rows per block
+  constexpr int PB = MAPS ? RB / 2 : RB;            // pairs (token, head) per block: rows r and r + PB are the maps of one
+  constexpr bool HALF = MAPS && !DEC;               // a warp multiplies one map's half of the columns
+  constexpr int QSTEPS = HALF ? KSTEPS / 2 : KSTEPS;
   constexpr int NST = DEC ? 3 : 2;      // K/V tiles in flight: decode blocks are latency bound
   extern __shared__ __align__(16) unsigned char smem_raw[];
   __nv_bfloat16* q_s = reinterpret_cast<__nv_bfloat16*>(smem_raw);   // [RB][LD]
@@ -275,19 +288,21 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 
   const int req = blockIdx.y / p.g, kvh = blockIdx.y - req * p.g;
   const int tok0 = p.q_start[req], q_len = p.q_start[req + 1] - tok0;
-  const int n_rows = q_len * p.per;
-  const int row0 = blockIdx.x * RB;
+  const int n_rows = q_len * p.per;              // (two maps: pairs)
+  const int row0 = blockIdx.x * PB;
   if (row0 >= n_rows) return;
   const int split = blockIdx.z;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int gid = lane >> 2, tig = lane & 3;
   const int wrow = DEC ? 0 : warp * 16;           // first row of this warp within the block's tile
   const int wkey = DEC ? warp * WKEYS : 0;        // first key of this warp within a key tile
+  const int wcol = HALF ? (wrow / PB) * p.map_dim : 0;         // first column of this warp's queries and keys
+  const int wcols = HALF ? p.map_dim : hs;
   const int32_t* bt = p.block_table + (size_t)req * p.table_width;
 
   // Positions of the tile's first and last token bound the keys this block needs.
   const int first_tok = row0 / p.per;
-  const int last_row = min(row0 + RB, n_rows) - 1;
+  const int last_row = min(row0 + PB, n_rows) - 1;
   const int last_tok = last_row / p.per;
   const int pos_first = p.positions[tok0 + first_tok];
   const int pos_last = p.positions[tok0 + last_tok];
@@ -330,9 +345,11 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     constexpr int CHUNKS = HS / 8;
     for (int c = threadIdx.x; c < RB * CHUNKS; c += NWARPS * 32) {
       const int r = c / CHUNKS, ch = c - r * CHUNKS;
-      const int row = row0 + r;
+      const int row = row0 + r % PB;
       __nv_bfloat16* d = q_s + r * LD + ch * 8;
-      if (row < n_rows && (!SIZED || ch * 8 < hs)) {
+      bool mine = !SIZED || ch * 8 < hs;
+      if (MAPS) mine = mine && (ch * 8 >= p.map_dim) == (r >= PB);    // the other map's half of the row stays zero
+      if (row < n_rows && mine) {
         const int t = row / p.per, h = row - t * p.per;
         cp_async16(d, p.q + (size_t)(tok0 + t) * p.q_stride + (size_t)(kvh * p.per + h) * hs + ch * 8);
       } else {
@@ -353,11 +370,11 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   cp_async_wait<NST - 2>();     // the group with Q and tile 0 has landed
   __syncthreads();
 
-  unsigned qf[KSTEPS][4];
+  unsigned qf[QSTEPS][4];
 #pragma unroll
-  for (int ks = 0; ks < KSTEPS; ++ks) {
+  for (int ks = 0; ks < QSTEPS; ++ks) {
     const int r = wrow + (lane & 7) + ((lane >> 3) & 1) * 8;
-    const int c = ks * 16 + (lane >> 4) * 8;
+    const int c = wcol + ks * 16 + (lane >> 4) * 8;
     ldmatrix_x4(qf[ks], q_s + r * LD + c);
   }
   // Rows of this thread: gid and gid + 8 of the warp's 16.
@@ -369,7 +386,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   int row_head[2] = {0, 0};
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
-    const int row = row0 + wrow + gid + i * 8;
+    const int row = row0 + (wrow + gid + i * 8) % PB;
     row_ok[i] = row < n_rows;
     row_pos[i] = row_ok[i] ? p.positions[tok0 + row / p.per] : -1;
     row_lo[i] = row_ok[i] ? first_visible<GEN>(p, row_pos[i]) : 0;
@@ -402,13 +419,13 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 #pragma unroll
     for (int j = 0; j < ST; ++j) s[j][0] = s[j][1] = s[j][2] = s[j][3] = 0.f;
 #pragma unroll
-    for (int ks = 0; ks < KSTEPS; ++ks) {
-      if (SIZED && ks * 16 >= hs) continue;
+    for (int ks = 0; ks < QSTEPS; ++ks) {
+      if (SIZED && ks * 16 >= wcols) continue;
 #pragma unroll
       for (int j = 0; j < ST; j += 2) {
         unsigned kb[4];
         const int key = wkey + j * 8 + (lane & 7) + (lane >> 4) * 8;
-        const int dim = ks * 16 + ((lane >> 3) & 1) * 8;
+        const int dim = wcol + ks * 16 + ((lane >> 3) & 1) * 8;
         ldmatrix_x4(kb, kt + key * LD + dim);
         mma_bf16(s[j], qf[ks], kb[0], kb[1]);
         mma_bf16(s[j + 1], qf[ks], kb[2], kb[3]);
@@ -417,8 +434,8 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
     // ---- mask, online softmax (exp2 domain) -----------------------------------------
     float m_new[2] = {m_run[0], m_run[1]};
     // A tile strictly inside every row's visible range needs no mask (the common case in decode).
-    const bool inner = pooled ? key0 + BN <= nb_first && row0 + RB <= n_rows
-                              : key0 + BN - 1 <= pos_first && key0 >= lo_last && row0 + RB <= n_rows &&
+    const bool inner = pooled ? key0 + BN <= nb_first && row0 + PB <= n_rows
+                              : key0 + BN - 1 <= pos_first && key0 >= lo_last && row0 + PB <= n_rows &&
                                     !(GEN && p.slopes) && !(EXT && p.rel);
     if (inner) {
 #pragma unroll
@@ -570,6 +587,89 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
       }
     }
     __syncthreads();
+    if constexpr (MAPS) {
+      float* os = mo + NWARPS * 16 * HS;              // [PB][vs]: the difference of the maps
+      const int pairs = min(PB, n_rows - row0);
+      // what the four warps have for a row and column: (maximum, sum of weights, weighted values)
+      auto merged = [&](int r, int d) {
+        float mm = -INFINITY, ll = 0.f, acc = 0.f;
+#pragma unroll
+        for (int w = 0; w < NWARPS; ++w) mm = fmaxf(mm, mml[(w * 16 + r) * 2]);
+#pragma unroll
+        for (int w = 0; w < NWARPS; ++w) {
+          const float m = mml[(w * 16 + r) * 2];
+          const float f = (m == -INFINITY) ? 0.f : exp2f(m - mm);
+          ll += mml[(w * 16 + r) * 2 + 1] * f;
+          acc += mo[((size_t)w * 16 + r) * HS + d] * f;
+        }
+        return make_float3(mm, ll, acc);
+      };
+      // the norm of every pair's difference and the store: a warp per pair
+      auto store_pairs = [&]() {
+        __syncthreads();
+        for (int u = warp; u < pairs; u += NWARPS) {
+          const int row = row0 + u, t = row / p.per, h = row - t * p.per;
+          float ss = 0.f;
+          for (int d = lane; d < vs; d += 32) ss = __fmaf_rn(os[u * vs + d], os[u * vs + d], ss);
+          const float r = p.out_scale / sqrtf(warp_sum(ss) / (float)vs + p.diff_eps);
+          __nv_bfloat16* dst = p.out + (size_t)(tok0 + t) * p.out_stride + (size_t)(kvh * p.per + h) * vs;
+          for (int d = lane; d < vs; d += 32) dst[d] = __float2bfloat16_rn(os[u * vs + d] * r);
+        }
+      };
+      if (p.n_splits == 1) {
+        for (int e = threadIdx.x; e < pairs * vs; e += NWARPS * 32) {
+          const int u = e / vs, d = e - u * vs;
+          const float3 a = merged(u, d), b = merged(u + PB, d);
+          os[e] = a.z / a.y - p.lambda * (b.z / b.y);
+        }
+        store_pairs();
+        return;
+      }
+      for (int e = threadIdx.x; e < 2 * pairs * vs; e += NWARPS * 32) {
+        const int ru = e / vs, d = e - ru * vs;
+        const int map = ru >= pairs, u = ru - map * pairs;
+        const int row = row0 + u, t = row / p.per, h = row - t * p.per;
+        const size_t slot = (((size_t)(tok0 + t) * p.nh + kvh * p.per + h) * 2 + map) * p.n_splits + split;
+        const float3 a = merged(u + map * PB, d);
+        p.part_o[slot * vs + d] = a.z;
+        if (d == 0) {
+          p.part_ml[slot * 2] = a.x;
+          p.part_ml[slot * 2 + 1] = a.y;
+        }
+      }
+      __shared__ int s_done;
+      int32_t* ticket = p.tickets + (size_t)blockIdx.y * gridDim.x + blockIdx.x;
+      __threadfence();
+      __syncthreads();
+      if (threadIdx.x == 0) s_done = (atomicAdd(ticket, 1) == p.n_splits - 1) ? 1 : 0;
+      __syncthreads();
+      if (!s_done) return;
+      __threadfence();
+      for (int e = threadIdx.x; e < pairs * vs; e += NWARPS * 32) {
+        const int u = e / vs, d = e - u * vs;
+        const int row = row0 + u, t = row / p.per, h = row - t * p.per;
+        const volatile float* ml = p.part_ml;
+        const volatile float* po = p.part_o;
+        float res[2];
+#pragma unroll
+        for (int map = 0; map < 2; ++map) {
+          const size_t base = (((size_t)(tok0 + t) * p.nh + kvh * p.per + h) * 2 + map) * p.n_splits;
+          float mm = -INFINITY, ll = 0.f, acc = 0.f;
+          for (int sp = 0; sp < p.n_splits; ++sp) mm = fmaxf(mm, ml[(base + sp) * 2]);
+          for (int sp = 0; sp < p.n_splits; ++sp) {
+            const float m = ml[(base + sp) * 2];
+            const float f = (m == -INFINITY) ? 0.f : exp2f(m - mm);
+            ll += ml[(base + sp) * 2 + 1] * f;
+            acc += po[(base + sp) * vs + d] * f;
+          }
+          res[map] = acc / ll;
+        }
+        os[e] = res[0] - p.lambda * res[1];
+      }
+      store_pairs();
+      if (threadIdx.x == 0) *ticket = 0;
+      return;
+    }
     const int rows_here = min(16, n_rows - row0);
     for (int e = threadIdx.x; e < rows_here * vs; e += NWARPS * 32) {
       const int r = e / vs, d = e - r * vs;
@@ -649,6 +749,50 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
         if (threadIdx.x == 0) p.tickets[blockIdx.y] = 0;
       }
     }
+  } else if constexpr (MAPS) {
+    // The second map's warps leave their results in shared memory; the first map's warps take lambda times them off.
+    constexpr int OLD = HS + 8;
+    float* other = reinterpret_cast<float*>(k_s);     // [PB][OLD] (fits the two K tiles)
+    static_assert(PB * OLD * sizeof(float) <= NST * BN * LD * sizeof(__nv_bfloat16), "the second map's results must fit");
+    __syncthreads();                                  // every warp is done with the K tiles
+    if (wrow >= PB) {
+#pragma unroll
+      for (int i = 0; i < 2; ++i) {
+        const float inv = l_run[i] > 0.f ? 1.0f / l_run[i] : 0.f;
+        float* dst = other + (wrow - PB + gid + i * 8) * OLD;
+#pragma unroll
+        for (int d = 0; d < DT; ++d)
+          if (d * 8 < vs) *reinterpret_cast<float2*>(dst + d * 8 + tig * 2) = make_float2(o[d][i * 2] * inv, o[d][i * 2 + 1] * inv);
+      }
+    }
+    __syncthreads();
+    if (wrow >= PB) return;
+#pragma unroll
+    for (int i = 0; i < 2; ++i) {
+      const float inv = l_run[i] > 0.f ? 1.0f / l_run[i] : 0.f;
+      const float* src = other + (wrow + gid + i * 8) * OLD;
+      float ss = 0.f;
+#pragma unroll
+      for (int d = 0; d < DT; ++d) {
+        if (d * 8 >= vs) continue;
+        const float2 b = *reinterpret_cast<const float2*>(src + d * 8 + tig * 2);
+        o[d][i * 2] = o[d][i * 2] * inv - p.lambda * b.x;
+        o[d][i * 2 + 1] = o[d][i * 2 + 1] * inv - p.lambda * b.y;
+        ss = __fmaf_rn(o[d][i * 2], o[d][i * 2], ss);
+        ss = __fmaf_rn(o[d][i * 2 + 1], o[d][i * 2 + 1], ss);
+      }
+      ss += __shfl_xor_sync(0xffffffffu, ss, 1);      // the four lanes of a row
+      ss += __shfl_xor_sync(0xffffffffu, ss, 2);
+      if (!row_ok[i]) continue;
+      const float r = p.out_scale / sqrtf(ss / (float)vs + p.diff_eps);
+      const int row = row0 + wrow + gid + i * 8;
+      const int t = row / p.per, h = row - t * p.per;
+      __nv_bfloat16* dst = p.out + (size_t)(tok0 + t) * p.out_stride + (size_t)(kvh * p.per + h) * vs;
+#pragma unroll
+      for (int d = 0; d < DT; ++d)
+        if (d * 8 < vs)
+          *reinterpret_cast<__nv_bfloat162*>(dst + d * 8 + tig * 2) = __floats2bfloat162_rn(o[d][i * 2] * r, o[d][i * 2 + 1] * r);
+    }
   } else {
 #pragma unroll
   for (int i = 0; i < 2; ++i) {
@@ -683,10 +827,10 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 template <int HS, bool DEC, int FORM>
 int launch_mode(const AttnParams& args, int n_requests, int max_rows, cudaStream_t stream) {
   constexpr int LD = HS + 8;
-  constexpr int RB = DEC ? 16 : BM, NST = DEC ? 3 : 2;
+  constexpr int RB = DEC ? 16 : BM, PB = FORM == 4 ? RB / 2 : RB, NST = DEC ? 3 : 2;
   constexpr size_t tiles = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
   // what a staged table of biases may take without costing a resident block
-  constexpr int rel_room = FORM >= 2 ? (DEC ? 1024 : 4096) : 0;
+  constexpr int rel_room = FORM == 2 || FORM == 3 ? (DEC ? 1024 : 4096) : 0;
   AttnParams p = args;
   p.rel_staged = p.rel != nullptr && p.per * p.rel_len <= rel_room;
   const size_t smem = tiles + (p.rel_staged ? (size_t)p.per * p.rel_len * sizeof(float) : 0);
@@ -697,7 +841,7 @@ int launch_mode(const AttnParams& args, int n_requests, int max_rows, cudaStream
       return YALIS_ERR_LAUNCH;
     configured = true;
   }
-  dim3 grid((max_rows + RB - 1) / RB, n_requests * p.g, p.n_splits);
+  dim3 grid((max_rows + PB - 1) / PB, n_requests * p.g, p.n_splits);
   if (grid.y > 65535 || grid.z > 65535) return YALIS_ERR_SHAPE;
   return yalis_launch(paged_attention_mma_kernel<HS, DEC, FORM>, grid, dim3(NWARPS * 32), smem, stream, p);
 }
@@ -721,6 +865,12 @@ int launch_extended(const AttnParams& p, int n_requests, int max_rows, cudaStrea
                         : launch_mode<HS, false, 3>(p, n_requests, max_rows, stream);
 }
 
+template <int HS>
+int launch_maps(const AttnParams& p, int n_requests, int max_pairs, cudaStream_t stream) {
+  return max_pairs <= 16 ? launch_mode<HS, true, 4>(p, n_requests, max_pairs, stream)
+                         : launch_mode<HS, false, 4>(p, n_requests, max_pairs, stream);
+}
+
 }  // namespace
 
 // Head sizes this kernel is built for.
@@ -738,6 +888,11 @@ YALIS_API int yalis_attention_mma_extended_supports(int hs, int vs) {
   return hs >= 8 && vs >= 8 && hs <= 256 && vs <= 256 && hs % 8 == 0 && vs % 8 == 0;
 }
 
+// Whether the form of two maps takes queries and keys of size d per map and values of size vs.
+YALIS_API int yalis_attention_mma_maps_supports(int d, int vs) {
+  return d >= 16 && d <= 128 && d % 16 == 0 && vs >= 8 && vs <= 256 && vs % 8 == 0;
+}
+
 // Scratch floats (hs: the size of a value) needed for n_splits > 1: part_o then part_ml.  Besides, `tickets` needs
 // n_requests * g int32 that are zero before the first launch (each launch leaves them zero).
 YALIS_API long long yalis_attention_mma_scratch_floats(int n_tokens, int nh, int hs, int n_splits) {
@@ -746,7 +901,9 @@ YALIS_API long long yalis_attention_mma_scratch_floats(int n_tokens, int nh, int
 
 // softcap 0: none.  With a cap, a sink, a factor other than 1 or exact_weights the general form of the kernel runs;
 // with vs != hs, a bias per distance (rel), pooled blocks (pool > 0) or a head size that has no kernel of its own the
-// extended form.
+// extended form.  maps 2: the form of two maps, hs the size of both maps' keys together and nh heads of two queries each
+// (no soft cap, sink, chunk, slopes, gate, rel or pooled blocks); a step may be split while its pairs (token, head) of a
+// request and key/value head are at most 16, with two partial results per head and a ticket per 8 pairs.
 YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, void* out, int out_stride, const void* k_pool,
                                                 const void* v_pool, const int32_t* positions, const int32_t* q_start,
                                                 const int32_t* req_of_token, const int32_t* block_table, int table_width,
@@ -757,10 +914,13 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
                                                 const float* slopes, const void* gate, int gate_stride,
                                                 int gate_per_head, int vs, const float* rel, int rel_len, int pool,
                                                 const void* pk_pool, const void* pv_pool, const int32_t* pool_table,
-                                                int pool_table_width, int pool_page_size, int pool_num_pages,
-                                                cudaStream_t stream) {
+                                                int pool_table_width, int pool_page_size, int pool_num_pages, int maps,
+                                                float lambda, float diff_eps, cudaStream_t stream) {
   if (n_tokens <= 0 || n_requests <= 0) return YALIS_OK;
   if (softcap < 0.f) return YALIS_ERR_SHAPE;
+  if (maps != 1 && (maps != 2 || hs % 2 || !yalis_attention_mma_maps_supports(hs / 2, vs) || softcap > 0.f || sink || chunk > 0 ||
+                    slopes || gate || rel || pool > 0))
+    return YALIS_ERR_SHAPE;
   if (g <= 0 || nh % g != 0 || n_splits < 1 || max_q_len < 1) return YALIS_ERR_SHAPE;
   if (((uintptr_t)q | (uintptr_t)k_pool | (uintptr_t)v_pool | (uintptr_t)out) & 15) return YALIS_ERR_ALIGN;
   if ((q_stride % 8) || (out_stride % 2)) return YALIS_ERR_ALIGN;
@@ -787,6 +947,7 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
   p.pool_page_shift = -1;
   for (int sh = 0; sh < 31; ++sh)
     if ((1 << sh) == pool_page_size) p.pool_page_shift = sh;
+  p.map_dim = hs / 2; p.lambda = lambda; p.diff_eps = diff_eps;
   const bool extended = vs != hs || rel != nullptr || pool > 0 || !yalis_attention_mma_supports(hs);
   if (pool < 0 || (rel && rel_len < 1)) return YALIS_ERR_SHAPE;
   if (pool > 0) {
@@ -799,10 +960,16 @@ YALIS_API int yalis_paged_attention_mma_general(const void* q, int q_stride, voi
   if (n_splits > 1) {
     if (scratch == nullptr || tickets == nullptr || max_q_len * p.per > 16) return YALIS_ERR_SHAPE;
     p.part_o = scratch;
-    p.part_ml = scratch + (size_t)n_tokens * nh * n_splits * vs;
+    p.part_ml = scratch + (size_t)n_tokens * nh * maps * n_splits * vs;
   }
   const int max_rows = max_q_len * p.per;
   int st;
+  if (maps == 2) {
+    const int widest = hs > vs ? hs : vs;
+    if (widest <= 64) return launch_maps<64>(p, n_requests, max_rows, stream);
+    if (widest <= 128) return launch_maps<128>(p, n_requests, max_rows, stream);
+    return launch_maps<256>(p, n_requests, max_rows, stream);
+  }
   if (extended) {
     const int widest = hs > vs ? hs : vs;
     if (widest <= 64) return launch_extended<64>(p, n_requests, max_rows, stream);
@@ -870,7 +1037,7 @@ YALIS_API int yalis_paged_attention_mma(const void* q, int q_stride, void* out, 
   return yalis_paged_attention_mma_general(q, q_stride, out, out_stride, k_pool, v_pool, positions, q_start, req_of_token,
                                            block_table, table_width, page_size, num_pages, n_tokens, n_requests, max_q_len,
                                            nh, g, hs, scale, window, n_splits, scratch, tickets, 0.f, 0, 1.0f, 0, 0, nullptr, nullptr,
-                                           nullptr, 0, 0, hs, nullptr, 0, 0, nullptr, nullptr, nullptr, 0, 0, 0, stream);
+                                           nullptr, 0, 0, hs, nullptr, 0, 0, nullptr, nullptr, nullptr, 0, 0, 0, 1, 0.f, 0.f, stream);
 }
 
 YALIS_API long long yalis_paged_attention_mma_noalloc_needed(int n_tokens, int n_requests, int nh, int g, int hs,

@@ -135,6 +135,113 @@ __device__ __forceinline__ void choose_experts(F logit, int E, int top, float ep
   }
 }
 
+// What a router may have beyond scores and a choice of the largest.
+struct ChoiceRules {
+  const float* correction;   // [E] added to the scores for the choice alone (null: nothing)
+  int groups, keep;          // groups > 0: E forms so many equal groups of neighbours, and only members of the `keep`
+                             // groups with the largest choice scores can be chosen
+  int real;                  // outputs [real, E) are identity experts: the sum of their chosen weights goes to `identity`
+  float* identity;           // [n_tokens] or null
+};
+
+// The choice of one token by one warp under such rules.  z [E] (shared memory): the token's logits, overwritten by the
+// choice scores; gs [groups] (shared memory): space for the groups' scores.  Scores are softmax over all outputs, or
+// sigmoid of each; ties go to the smaller index, among groups too.  kPer: outputs a lane holds (32 kPer >= E).
+template <int kPer>
+__device__ __forceinline__ void choose_experts_by_rules(float* z, float* gs, const ChoiceRules& rules, int E, int top, float eps,
+                                                        float factor, int lane, int32_t* __restrict__ ids,
+                                                        float* __restrict__ weights, float* __restrict__ identity, int sigmoid) {
+  float s[kPer], c[kPer];                // scores and choice scores
+  if (sigmoid) {
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) s[i] = lane + 32 * i < E ? 1.0f / (1.0f + expf(-z[lane + 32 * i])) : 0.f;
+  } else {
+    float m = -INFINITY, sum = 0.f;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      s[i] = lane + 32 * i < E ? z[lane + 32 * i] : -INFINITY;
+      m = fmaxf(m, s[i]);
+    }
+    m = warp_max(m);
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      s[i] = lane + 32 * i < E ? expf(s[i] - m) : 0.f;
+      sum += s[i];
+    }
+    sum = warp_sum(sum);
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) s[i] = s[i] / sum;
+  }
+#pragma unroll
+  for (int i = 0; i < kPer; ++i) {
+    const int e = lane + 32 * i;
+    c[i] = e < E ? s[i] + (rules.correction ? rules.correction[e] : 0.f) : -INFINITY;
+    if (e < E) z[e] = c[i];
+  }
+  if (rules.groups > 0) {
+    const int size = E / rules.groups;
+    __syncwarp();
+    for (int g = lane; g < rules.groups; g += 32) {
+      float best = -INFINITY;
+      for (int e = g * size; e < (g + 1) * size; ++e) best = fmaxf(best, z[e]);
+      gs[g] = best;
+    }
+    __syncwarp();
+#pragma unroll
+    for (int i = 0; i < kPer; ++i) {
+      const int e = lane + 32 * i;
+      if (e >= E) continue;
+      const int g = e / size;
+      const float mine = gs[g];
+      int before = 0;                    // groups that come before this one
+      for (int o = 0; o < rules.groups; ++o) before += gs[o] > mine || (gs[o] == mine && o < g);
+      if (before >= rules.keep) c[i] = -INFINITY;
+    }
+  }
+  float chosen_w = 0.f, total = 0.f, same = 0.f;     // lane j keeps the j-th choice
+  int chosen_e = -1;
+  for (int j = 0; j < top; ++j) {
+    float best = -INFINITY, score = 0.f;
+    int best_e = 0x7fffffff;
+#pragma unroll
+    for (int i = 0; i < kPer; ++i)
+      if (c[i] > best) {                 // ascending e within a lane: the first maximum is the smallest index
+        best = c[i];
+        best_e = lane + 32 * i;
+        score = s[i];
+      }
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) {
+      const float ob = __shfl_xor_sync(0xffffffffu, best, o), os = __shfl_xor_sync(0xffffffffu, score, o);
+      const int oe = __shfl_xor_sync(0xffffffffu, best_e, o);
+      if (ob > best || (ob == best && oe < best_e)) {
+        best = ob;
+        best_e = oe;
+        score = os;
+      }
+    }
+    if ((best_e & 31) == lane) {
+#pragma unroll
+      for (int i = 0; i < kPer; ++i)
+        if (lane + 32 * i == best_e) c[i] = -INFINITY;
+    }
+    if (lane == j) {
+      chosen_w = score;
+      chosen_e = best_e < E ? best_e : -1;           // (fewer candidates than `top`, or scores that are no numbers)
+    }
+    if (best_e < E) {
+      total += score;
+      if (best_e >= rules.real) same += score;
+    }
+  }
+  const float scale = eps < 0.f ? factor : factor / (total + eps);
+  if (lane < top) {
+    ids[lane] = chosen_e;
+    weights[lane] = chosen_e < 0 ? 0.f : chosen_w * scale;
+  }
+  if (identity && lane == 0) *identity = same * scale;
+}
+
 // From given logits: one warp per token.
 __global__ void route_topk_kernel(const float* __restrict__ logits, int E, int top, float eps, float factor,
                                   const int32_t* __restrict__ req_of_token, int32_t* __restrict__ ids,
@@ -170,12 +277,13 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float& a, float& b
 // the choice.  A block takes TOK tokens: their rows wait in shared memory in their own dtype, the warps share out
 // the experts, and a row of the router read once serves all TOK tokens (each token's sum has the same order whatever
 // TOK is); then warp t chooses for token t.
-template <typename T, int TOK>
+template <typename T, int TOK, bool RULES>
 __global__ void route_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ w, int E, int K, int top,
                              float eps, float factor, const int32_t* __restrict__ req_of_token, int32_t* __restrict__ ids,
                              float* __restrict__ weights, int n_tokens, int sigmoid, const float* __restrict__ side,
-                             float* __restrict__ side_out) {
-  extern __shared__ __align__(16) unsigned char route_smem[];   // [TOK][K] rows (T), then [TOK][E] logits (float)
+                             float* __restrict__ side_out, const ChoiceRules rules) {
+  // [TOK][K] rows (T), then [TOK][E] logits and [TOK][groups] group scores (float)
+  extern __shared__ __align__(16) unsigned char route_smem[];
   T* xs = reinterpret_cast<T*>(route_smem);
   float* z = reinterpret_cast<float*>(route_smem + (((size_t)TOK * K * sizeof(T) + 15) & ~(size_t)15));
   pdl_launch_dependents();
@@ -246,27 +354,38 @@ __global__ void route_kernel(const T* __restrict__ x, long x_stride, const float
         ids[(size_t)n * top + j] = -1;
         weights[(size_t)n * top + j] = 0.f;
       }
+      if (rules.identity && lane == 0) rules.identity[n] = 0.f;
       continue;
     }
-    const float* zt = z + t * E;
+    float* zt = z + t * E;
+    if constexpr (RULES) {
+      float* gs = z + TOK * E + t * rules.groups;
+      float* same = rules.identity ? rules.identity + n : nullptr;
+      int32_t* id = ids + (size_t)n * top;
+      float* wt = weights + (size_t)n * top;
+      if (E <= 32) choose_experts_by_rules<1>(zt, gs, rules, E, top, eps, factor, lane, id, wt, same, sigmoid);
+      else if (E <= 128) choose_experts_by_rules<4>(zt, gs, rules, E, top, eps, factor, lane, id, wt, same, sigmoid);
+      else choose_experts_by_rules<kMaxExperts / 32>(zt, gs, rules, E, top, eps, factor, lane, id, wt, same, sigmoid);
+      continue;
+    }
     choose_experts([&](int e) { return zt[e]; }, E, top, eps, factor, lane, ids + (size_t)n * top, weights + (size_t)n * top, sigmoid);
   }
 }
 
-template <typename T, int TOK>
+template <typename T, int TOK, bool RULES>
 int launch_route(const void* x, long x_stride, const float* w, int n_tokens, int E, int K, int top, float eps, float factor,
                  const int32_t* req_of_token, int32_t* ids, float* weights, int sigmoid, const float* side, float* side_out,
-                 cudaStream_t stream) {
-  const size_t smem = (((size_t)TOK * K * sizeof(T) + 15) & ~(size_t)15) + (size_t)TOK * E * sizeof(float);
+                 const ChoiceRules& rules, cudaStream_t stream) {
+  const size_t smem = (((size_t)TOK * K * sizeof(T) + 15) & ~(size_t)15) + (size_t)TOK * (E + rules.groups) * sizeof(float);
   if (smem > 200 * 1024) return YALIS_ERR_SHAPE;
   static size_t configured = 0;
   if (smem > 48 * 1024 && smem > configured) {
-    if (cudaFuncSetAttribute(route_kernel<T, TOK>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
+    if (cudaFuncSetAttribute(route_kernel<T, TOK, RULES>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess)
       return YALIS_ERR_LAUNCH;
     configured = smem;
   }
-  return yalis_launch(route_kernel<T, TOK>, dim3((n_tokens + TOK - 1) / TOK), dim3(256), smem, stream, (const T*)x, x_stride, w, E, K,
-                      top, eps, factor, req_of_token, ids, weights, n_tokens, sigmoid, side, side_out);
+  return yalis_launch(route_kernel<T, TOK, RULES>, dim3((n_tokens + TOK - 1) / TOK), dim3(256), smem, stream, (const T*)x, x_stride, w, E, K,
+                      top, eps, factor, req_of_token, ids, weights, n_tokens, sigmoid, side, side_out, rules);
 }
 
 // One block.  entries = n_tokens * top.  tiles: (expert, first slot) per row tile of `bm` slots, ended by n_tiles.
@@ -637,18 +756,26 @@ YALIS_API int yalis_route_topk(const float* logits, int n_tokens, int E, int top
 
 // The router and the choice in one launch.  x: [n_tokens, K] float32 or bfloat16; w: float32 [E, K].  Steps of a
 // thousand tokens and more take eight to a block where their rows fit shared memory (fewer tokens would leave SMs
-// without a block: 64 tokens in 8 blocks took 48 us, in 64 blocks 13).
+// without a block: 64 tokens in 8 blocks took 48 us, in 64 blocks 13).  correction, groups and keep, real and identity:
+// see ChoiceRules (null, 0, E and null: none).
 YALIS_API int yalis_route(const void* x, int x_dtype, long x_stride, const float* w, int n_tokens, int E, int K, int top, float eps, float factor,
                           const int32_t* req_of_token, int32_t* ids, float* weights, int sigmoid, const float* side,
-                          float* side_out, cudaStream_t stream) {
+                          float* side_out, const float* correction, int groups, int keep, int real, float* identity,
+                          cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
   if (E <= 0 || E > kMaxExperts || top <= 0 || top > kMaxTop || top > E || K <= 0) return YALIS_ERR_SHAPE;
   if ((side == nullptr) != (side_out == nullptr)) return YALIS_ERR_SHAPE;
+  if (groups < 0 || (groups > 0 && (E % groups || keep < 1 || keep > groups || keep * (E / groups) < top))) return YALIS_ERR_SHAPE;
+  if (real < 0 || real > E || (real < E && !identity)) return YALIS_ERR_SHAPE;
+  const ChoiceRules rules = {correction, groups, keep, real, identity};
   const size_t elt = x_dtype == YALIS_BF16 ? 2 : 4;
-  const bool many = n_tokens >= 1024 && 8 * ((size_t)K * elt + (size_t)E * 4) + 16 <= 96 * 1024;
-  YALIS_DISPATCH_DTYPE(x_dtype, T,
-                       return many ? launch_route<T, 8>(x, x_stride, w, n_tokens, E, K, top, eps, factor, req_of_token, ids, weights, sigmoid, side, side_out, stream)
-                                   : launch_route<T, 1>(x, x_stride, w, n_tokens, E, K, top, eps, factor, req_of_token, ids, weights, sigmoid, side, side_out, stream));
+  const bool many = n_tokens >= 1024 && 8 * ((size_t)K * elt + (size_t)(E + groups) * 4) + 16 <= 96 * 1024;
+  const bool ruled = correction || groups > 0 || real < E;
+  YALIS_DISPATCH_DTYPE(x_dtype, T, {
+    auto launch = many ? (ruled ? launch_route<T, 8, true> : launch_route<T, 8, false>)
+                       : (ruled ? launch_route<T, 1, true> : launch_route<T, 1, false>);
+    return launch(x, x_stride, w, n_tokens, E, K, top, eps, factor, req_of_token, ids, weights, sigmoid, side, side_out, rules, stream);
+  });
   return YALIS_OK;
 }
 

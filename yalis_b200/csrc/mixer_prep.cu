@@ -30,6 +30,7 @@ struct PrepParams {
   const int32_t* block_table; int table_width, page_size, num_pages;
   const int32_t* positions; const int32_t* req_of_token;
   int nq, nk, dim, vdim;
+  int maps;                                  // keys per key/value head, side by side in its cached row [maps * dim] (1: the usual)
   int32_t* bad_page;
   int pool;                                  // P > 0: the warp that stores the last row of a block of P positions stores their mean
   void* pk_pool; void* pv_pool;              // [pages, nk, pool_page_size, dim] and [..., vdim], an entry per block
@@ -149,7 +150,7 @@ __device__ __forceinline__ float row_squares(const T* row, const T* bias, int co
   return block_sum(ss, scratch);
 }
 
-// One warp per (token, head): heads [0, nq) are queries, [nq, nq + nk) keys, [nq + nk, nq + 2 nk) values.  A warp goes on
+// One warp per (token, head): heads [0, nq) are queries, then nk * maps keys, then nk values.  A warp goes on
 // to further heads of its token where the grid has fewer warps than heads.
 // TABLE: the block computes the token's sines and cosines once, in shared memory (steps of many tokens, where a block
 // walks all heads).  VEC: four consecutive values at a time (every row, size and offset a multiple of four, aligned).
@@ -182,8 +183,8 @@ __global__ void __launch_bounds__(256, 5) qkv_prepare_kernel(const PrepParams p)
   if (p.norm_all) {
     if (p.q_norm) all_q = 1.0f / sqrtf(row_squares<T, VEC>(row + p.q_off, reinterpret_cast<const T*>(p.q_bias), p.nq * p.dim, scratch) /
                                            (float)(p.nq * p.dim) + p.norm_eps);
-    if (p.k_norm) all_k = 1.0f / sqrtf(row_squares<T, VEC>(row + p.k_off, reinterpret_cast<const T*>(p.k_bias), p.nk * p.dim, scratch) /
-                                           (float)(p.nk * p.dim) + p.norm_eps);
+    if (p.k_norm) all_k = 1.0f / sqrtf(row_squares<T, VEC>(row + p.k_off, reinterpret_cast<const T*>(p.k_bias), p.nk * p.maps * p.dim, scratch) /
+                                           (float)(p.nk * p.maps * p.dim) + p.norm_eps);
   }
   auto turned = [&](int i, float& cs, float& sn) {
     if constexpr (TABLE) {
@@ -202,9 +203,10 @@ __global__ void __launch_bounds__(256, 5) qkv_prepare_kernel(const PrepParams p)
   const float q_factor = p.q_temp_every > 0 ? p.q_scale * (1.0f + p.q_temp_coef * logf((float)((pos + 1) / p.q_temp_every + 1)))
                                             : p.q_scale;
   const bool ends_block = p.pool > 0 && (pos + 1) % p.pool == 0;
-  for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < p.nq + 2 * p.nk; head += gridDim.y * warps) {
-    const bool is_q = head < p.nq, is_v = head >= p.nq + p.nk;
-    const int hh = is_q ? head : (is_v ? head - p.nq - p.nk : head - p.nq);
+  const int keys = p.nk * p.maps;
+  for (int head = blockIdx.y * warps + (threadIdx.x >> 5); head < p.nq + keys + p.nk; head += gridDim.y * warps) {
+    const bool is_q = head < p.nq, is_v = head >= p.nq + keys;
+    const int hh = is_q ? head : (is_v ? head - p.nq - keys : head - p.nq);
     const int width = is_v ? p.vdim : p.dim;
     const T* src = row + (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + (size_t)hh * width;
     const T* bias = reinterpret_cast<const T*>(is_q ? p.q_bias : (is_v ? p.v_bias : p.k_bias));
@@ -217,7 +219,8 @@ __global__ void __launch_bounds__(256, 5) qkv_prepare_kernel(const PrepParams p)
         if (lane == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
         continue;
       }
-      dst = reinterpret_cast<TO*>(is_v ? p.v_pool : p.k_pool) + (row0 + (long long)hh * p.page_size) * width;
+      if (is_v) dst = reinterpret_cast<TO*>(p.v_pool) + (row0 + (long long)hh * p.page_size) * width;
+      else dst = reinterpret_cast<TO*>(p.k_pool) + (row0 + (long long)(hh / p.maps) * p.page_size) * (p.maps * width) + hh % p.maps * width;
     } else {
       if (p.k_out == nullptr) continue;            // nothing keeps this layer's keys and values: queries only
       dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
@@ -324,9 +327,9 @@ int launch_qkv_prepare(const PrepParams& p, dim3 grid, int warps, bool table, bo
 }
 
 // ACT: 0 gelu with erf, 1 gelu with tanh, 2 silu, 3 the square of relu, 4 tanh.
-// With `bias` (float32, one per column) it is added to x first.
-template <typename T>
-__global__ void activation_kernel(const T* __restrict__ x, int x_stride, T* __restrict__ y, int y_stride, int rows,
+// With `bias` (float32, one per column) it is added to x first.  TO: the result's type (T, or float32).
+template <typename T, typename TO>
+__global__ void activation_kernel(const T* __restrict__ x, int x_stride, TO* __restrict__ y, int y_stride, int rows,
                                   int cols, int act, const float* __restrict__ bias) {
   pdl_launch_dependents();
   pdl_wait();
@@ -341,7 +344,7 @@ __global__ void activation_kernel(const T* __restrict__ x, int x_stride, T* __re
     else if (act == 2) o = silu_exact(z);
     else if (act == 4) o = tanhf(z);
     else o = fmaxf(z, 0.f) * fmaxf(z, 0.f);
-    y[r * y_stride + c] = from_f32<T>(o);
+    y[r * y_stride + c] = from_f32<TO>(o);
   }
 }
 
@@ -375,6 +378,28 @@ __global__ void activation_bf16x8_kernel(const __nv_bfloat16* __restrict__ x, in
     h[i] = __floats2bfloat162_rn(act_value(z.x, act), act_value(z.y, act));
   }
   *reinterpret_cast<uint4*>(y + r * y_stride + c) = raw;
+}
+
+// Four elements a thread with float32 results (bfloat16 rows on 8-byte boundaries, float32 rows on 16-byte ones).  Its
+// reader may be a kernel of few, long blocks (a recurrence over the rows it makes): those are let in only once this one
+// has begun, so that they do not crowd onto the SMs that come free first.
+template <typename T>
+__global__ void activation_f32x4_kernel(const T* __restrict__ x, int x_stride, float* __restrict__ y, int y_stride, int rows,
+                                        int cols, int act, const float* __restrict__ bias) {
+  pdl_wait();
+  pdl_launch_dependents();
+  const int quads = cols >> 2;
+  const size_t total = (size_t)rows * quads;
+  for (size_t e = (size_t)blockIdx.x * blockDim.x + threadIdx.x; e < total; e += (size_t)gridDim.x * blockDim.x) {
+    const size_t r = e / quads;
+    const int c = (int)(e - r * quads) << 2;
+    float4 z = load4_f32(x + r * x_stride + c);
+    if (bias) {
+      const float4 b = load4_f32(bias + c);
+      z.x += b.x; z.y += b.y; z.z += b.z; z.w += b.w;
+    }
+    store4(y + r * y_stride + c, make_float4(act_value(z.x, act), act_value(z.y, act), act_value(z.z, act), act_value(z.w, act)));
+  }
 }
 
 // A gated activation over rows that hold a gate part and an up part (at column offsets of one matrix):
@@ -452,6 +477,8 @@ __global__ void add_rows_vector_kernel(float* __restrict__ x, const float* __res
 // pool > 0: the means of blocks of `pool` keys and values go to pk_pool / pv_pool.  With single_tokens (no request brings
 // more than one token) the warp that stores a block's last row does it; otherwise a second kernel does, once all rows of
 // the step are stored.
+// maps > 1 (without pooled blocks): every key/value head has `maps` keys of size dim, which lie side by side in src and in a
+// cached row; nk counts the key/value heads.
 // out_dtype: the dtype of q_out and of the plain k_out / v_out (pools always have the model dtype `dtype`).
 YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int q_off, int k_off, int v_off,
                                 const void* q_bias, const void* k_bias, const void* v_bias, const float* q_norm,
@@ -463,10 +490,11 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
                                 const int32_t* positions, const int32_t* req_of_token, int n_tokens, int nq, int nk,
                                 int dim, int vdim, int32_t* bad_page, int pool, void* pk_pool, void* pv_pool,
                                 const int32_t* pool_table, int pool_table_width, int pool_page_size, int pool_num_pages,
-                                int single_tokens, cudaStream_t stream) {
+                                int single_tokens, int maps, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
   if (pool < 0 || (pool > 0 && (!k_pool || !pk_pool || !pv_pool || !pool_table || pool_page_size < 1))) return YALIS_ERR_SHAPE;
-  if (dim <= 0 || dim > kMaxHeadDim || vdim <= 0 || vdim > kMaxHeadDim || nq <= 0 || nk <= 0 || nq + 2 * nk > 65535)
+  if (dim <= 0 || dim > kMaxHeadDim || vdim <= 0 || vdim > kMaxHeadDim || nq <= 0 || nk <= 0 || maps < 1 ||
+      nq + (maps + 1) * nk > 65535 || (maps > 1 && pool > 0))
     return YALIS_ERR_SHAPE;
   if (inv_freq && (rot_dims <= 0 || (rot_dims & 1) || rot_dims > dim)) return YALIS_ERR_SHAPE;
   if (k_pool && out_dtype != dtype) return YALIS_ERR_DTYPE;
@@ -479,7 +507,7 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   p.q_out = q_out; p.q_out_stride = q_out_stride; p.k_out = k_out; p.k_out_stride = k_out_stride;
   p.v_out = v_out; p.v_out_stride = v_out_stride; p.k_pool = k_pool; p.v_pool = v_pool; p.block_table = block_table;
   p.table_width = table_width; p.page_size = page_size; p.num_pages = num_pages; p.positions = positions;
-  p.req_of_token = req_of_token; p.nq = nq; p.nk = nk; p.dim = dim; p.vdim = vdim; p.bad_page = bad_page;
+  p.req_of_token = req_of_token; p.nq = nq; p.nk = nk; p.dim = dim; p.vdim = vdim; p.maps = maps; p.bad_page = bad_page;
   p.pool = single_tokens ? pool : 0;
   p.pk_pool = pk_pool; p.pv_pool = pv_pool; p.pool_table = pool_table; p.pool_table_width = pool_table_width;
   p.pool_page_size = pool_page_size; p.pool_num_pages = pool_num_pages;
@@ -487,7 +515,7 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   // the sums of a norm over all heads.  Few tokens: four heads a block, so that more blocks run at once.
   const bool per_token = n_tokens >= 2 * yalis_sm_count() && dim <= 512 && vdim <= 512;
   const int warps = per_token ? 8 : 4;
-  const dim3 grid(n_tokens, per_token ? 1 : (nq + 2 * nk + warps - 1) / warps);
+  const dim3 grid(n_tokens, per_token ? 1 : (nq + (maps + 1) * nk + warps - 1) / warps);
   const bool table = per_token && inv_freq != nullptr;
   const uintptr_t ptrs = (uintptr_t)src | (uintptr_t)q_bias | (uintptr_t)k_bias | (uintptr_t)v_bias | (uintptr_t)q_norm |
                          (uintptr_t)k_norm | (uintptr_t)q_out | (uintptr_t)k_out | (uintptr_t)v_out | (uintptr_t)k_pool |
@@ -510,18 +538,29 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   return YALIS_OK;
 }
 
-YALIS_API int yalis_activation(const void* x, int x_stride, void* y, int y_stride, int dtype, int rows, int cols,
+// y_f32: the result is float32 whatever the input's type.
+YALIS_API int yalis_activation(const void* x, int x_stride, void* y, int y_stride, int dtype, int y_f32, int rows, int cols,
                                int act, const float* bias, cudaStream_t stream) {
   if (rows <= 0 || cols <= 0) return YALIS_OK;
   if (act < 0 || act > 4) return YALIS_ERR_SHAPE;
   const size_t total = (size_t)rows * cols;
   const int blocks = (int)((total + 255) / 256 < 148 * 16 ? (total + 255) / 256 : 148 * 16);
+  if (y_f32 && cols % 4 == 0 && x_stride % 4 == 0 && y_stride % 4 == 0 && !((uintptr_t)x & (dtype == YALIS_BF16 ? 7 : 15)) &&
+      !(((uintptr_t)y | (uintptr_t)bias) & 15)) {
+    const size_t quads = (total / 4 + 255) / 256;
+    const dim3 grid((unsigned)(quads < 148 * 16 ? quads : 148 * 16));
+    YALIS_DISPATCH_DTYPE(dtype, T, return yalis_launch(activation_f32x4_kernel<T>, grid, dim3(256), 0, stream, (const T*)x,
+                                                       x_stride, (float*)y, y_stride, rows, cols, act, bias));
+  }
+  if (y_f32 && dtype == YALIS_BF16)
+    return yalis_launch(activation_kernel<__nv_bfloat16, float>, dim3(blocks), dim3(256), 0, stream, (const __nv_bfloat16*)x,
+                        x_stride, (float*)y, y_stride, rows, cols, act, bias);
   if (dtype == YALIS_BF16 && cols % 8 == 0 && x_stride % 8 == 0 && y_stride % 8 == 0 && !((uintptr_t)x & 15) &&
       !((uintptr_t)y & 15) && !((uintptr_t)bias & 7) && rows <= 65535)
     return yalis_launch(activation_bf16x8_kernel, dim3((cols / 8 + 127) / 128, rows), dim3(128), 0, stream,
                         (const __nv_bfloat16*)x, x_stride, (__nv_bfloat16*)y, y_stride, cols, act, bias);
   YALIS_DISPATCH_DTYPE(dtype, T,
-                       return yalis_launch(activation_kernel<T>, dim3(blocks), dim3(256), 0, stream, (const T*)x, x_stride,
+                       return yalis_launch((activation_kernel<T, T>), dim3(blocks), dim3(256), 0, stream, (const T*)x, x_stride,
                                            (T*)y, y_stride, rows, cols, act, bias));
   return YALIS_OK;
 }

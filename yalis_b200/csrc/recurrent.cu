@@ -499,14 +499,19 @@ __global__ void head_norm_gate_kernel(const float* __restrict__ o, int o_stride,
   }
 }
 
-// ---- gate, then norm in equal parts -----------------------------------------------------------------------------
-//   y = o * silu(z);   y[part] <- y / sqrt(mean(y^2 over the part) + eps) * weight * out_scale
-// A block per (token, part); a part waits in shared memory between the two passes.
-template <typename T>
+// ---- gate and norm in equal parts -------------------------------------------------------------------------------
+//   y = o * act(z);   y[part] <- y / sqrt(mean(y^2 over the part) + eps) * weight * out_scale           (after = 0)
+//   y = o / sqrt(mean(o^2 over the part) + eps) * weight * act(z) * out_scale                            (after = 1)
+// GATE: 1 silu, 2 sigmoid.  A block per (token, part); a part waits in shared memory between the two passes.  VEC: four
+// values at a time (all rows and parts on 16-byte boundaries of float32, 8-byte ones of bfloat16).
+__device__ __forceinline__ float gate_value(float z, int kind) { return kind == 1 ? silu_exact(z) : sigmoid_f(z); }
+
+template <typename T, bool VEC>
 __global__ void gate_norm_kernel(const float* __restrict__ o, int o_stride, const T* __restrict__ z, int z_stride,
                                  const float* __restrict__ weight, T* __restrict__ y, int y_stride,
-                                 const int32_t* __restrict__ req_of_token, int width, float eps, float out_scale) {
-  extern __shared__ float part_s[];               // [width]
+                                 const int32_t* __restrict__ req_of_token, int width, float eps, float out_scale, int kind,
+                                 int after) {
+  extern __shared__ __align__(16) float part_s[];  // [width]
   __shared__ float scratch[32];
   pdl_launch_dependents();
   pdl_wait();
@@ -514,15 +519,42 @@ __global__ void gate_norm_kernel(const float* __restrict__ o, int o_stride, cons
   if (req_of_token[n] < 0) return;
   const float* op = o + (size_t)n * o_stride + c0;
   const T* zp = z + (size_t)n * z_stride + c0;
-  float ss = 0.f;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) {
-    const float v = op[c] * silu_exact(to_f32<T>(zp[c]));
-    part_s[c] = v;
-    ss = __fmaf_rn(v, v, ss);
-  }
-  const float r = 1.0f / sqrtf(block_sum(ss, scratch) / (float)width + eps);
   T* yp = y + (size_t)n * y_stride + c0;
-  for (int c = threadIdx.x; c < width; c += blockDim.x) yp[c] = from_f32<T>(part_s[c] * r * weight[c0 + c] * out_scale);
+  const float* wp = weight + c0;
+  float ss = 0.f;
+  if constexpr (VEC) {
+    for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
+      float4 v = load4_f32(op + c);
+      if (!after) {
+        const float4 g = load4_f32(zp + c);
+        v.x *= gate_value(g.x, kind); v.y *= gate_value(g.y, kind); v.z *= gate_value(g.z, kind); v.w *= gate_value(g.w, kind);
+      }
+      *reinterpret_cast<float4*>(part_s + c) = v;
+      ss = __fmaf_rn(v.x, v.x, ss); ss = __fmaf_rn(v.y, v.y, ss); ss = __fmaf_rn(v.z, v.z, ss); ss = __fmaf_rn(v.w, v.w, ss);
+    }
+    const float r = out_scale / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    for (int c = threadIdx.x * 4; c < width; c += blockDim.x * 4) {
+      float4 v = *reinterpret_cast<const float4*>(part_s + c);
+      const float4 w = load4_f32(wp + c);
+      v.x *= r * w.x; v.y *= r * w.y; v.z *= r * w.z; v.w *= r * w.w;
+      if (after) {
+        const float4 g = load4_f32(zp + c);
+        v.x *= gate_value(g.x, kind); v.y *= gate_value(g.y, kind); v.z *= gate_value(g.z, kind); v.w *= gate_value(g.w, kind);
+      }
+      store4(yp + c, v);
+    }
+  } else {
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = after ? op[c] : op[c] * gate_value(to_f32<T>(zp[c]), kind);
+      part_s[c] = v;
+      ss = __fmaf_rn(v, v, ss);
+    }
+    const float r = out_scale / sqrtf(block_sum(ss, scratch) / (float)width + eps);
+    for (int c = threadIdx.x; c < width; c += blockDim.x) {
+      const float v = part_s[c] * r * wp[c];
+      yp[c] = from_f32<T>(after ? v * gate_value(to_f32<T>(zp[c]), kind) : v);
+    }
+  }
 }
 
 // ---- what the generalized delta rule reads ------------------------------------------------------------
@@ -725,20 +757,24 @@ YALIS_API int yalis_head_norm_gate(const float* o, int o_stride, const float* we
 }
 
 // o float32 [N, parts * width]; z (model dtype) the gate's input; weight float32 [parts * width]; y in the model dtype.
+// gate_kind 1: silu, 2: sigmoid; after: the gate stands behind the norm.
 YALIS_API int yalis_gate_norm(const float* o, int o_stride, const void* z, int z_stride, const float* weight, void* y,
                               int y_stride, int dtype, const int32_t* req_of_token, int n_tokens, int parts, int width,
-                              float eps, float out_scale, cudaStream_t stream) {
+                              float eps, float out_scale, int gate_kind, int after, cudaStream_t stream) {
   if (n_tokens <= 0) return YALIS_OK;
-  if (parts <= 0 || parts > 65535 || width <= 0) return YALIS_ERR_SHAPE;
+  if (parts <= 0 || parts > 65535 || width <= 0 || gate_kind < 1 || gate_kind > 2) return YALIS_ERR_SHAPE;
   const int threads = width >= 1024 ? 256 : (width >= 256 ? 128 : 64);
   const size_t smem = (size_t)width * sizeof(float);
   if (smem > 200 * 1024) return YALIS_ERR_SHAPE;
+  const uintptr_t narrow = dtype == YALIS_BF16 ? 7 : 15;
+  const bool vec = ((width | o_stride | z_stride | y_stride) & 3) == 0 && !(((uintptr_t)o | (uintptr_t)weight) & 15) &&
+                   !(((uintptr_t)z | (uintptr_t)y) & narrow);
   YALIS_DISPATCH_DTYPE(dtype, T, {
-    if (smem > 48 * 1024 &&
-        cudaFuncSetAttribute(gate_norm_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
+    auto kernel = vec ? gate_norm_kernel<T, true> : gate_norm_kernel<T, false>;
+    if (smem > 48 * 1024 && cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess)
       return YALIS_ERR_LAUNCH;
-    return yalis_launch(gate_norm_kernel<T>, dim3(n_tokens, parts), dim3(threads), smem, stream, o, o_stride, (const T*)z, z_stride,
-                        weight, (T*)y, y_stride, req_of_token, width, eps, out_scale);
+    return yalis_launch(kernel, dim3(n_tokens, parts), dim3(threads), smem, stream, o, o_stride, (const T*)z, z_stride,
+                        weight, (T*)y, y_stride, req_of_token, width, eps, out_scale, gate_kind, after);
   });
   return YALIS_OK;
 }

@@ -7,9 +7,12 @@
 //                      x_t <- sum_s mix[s][t] x_s + out[t] * y          (all copies from the old ones)
 //   read  (optional)   u  = sum_s in[s] x_s                             (in absent: the plain sum)
 //                      h  = tanh(alpha * u) * w[c] + b[c]               (norm absent: h = u)
+//                or    h  = u / sqrt(mean_c(u^2) + eps) * rms_w[c]
 //
-// Nothing here needs a sum over a row, so a thread owns a few columns of one row and the copies stay in registers
-// between the write of one sub-layer and the read of the next.  With S = 1, mix = out = in = 1 this is the plain
+// A thread owns a few columns of one row and the copies stay in registers between the write of one sub-layer and the
+// read of the next.  Only the root-mean-square norm needs a sum over a row: its form of the kernel gives a block the
+// whole row and keeps u in registers (or in shared memory, for rows longer than a block's threads can hold) until the
+// sum is known.  With S = 1, mix = out = in = 1 this is the plain
 // "x += y; h = norm(x)" of a pre-norm layer, so the same kernel serves a model with one copy.  All arithmetic is
 // float32; y, gate and h are in the model's dtype (the partial results of a split product are float32).
 //
@@ -31,6 +34,7 @@ struct StreamStep {
   const float* mix; const float* out_w;         // [copies, copies] (from, to) and [copies]; both null: x_t += y
   const float* in_w;                            // [copies] or null (the plain sum)
   const float* alpha; const float* norm_w; const float* norm_b;              // norm: all three or none
+  const float* rms_w; float rms_eps;            // the other norm: root mean square (null: none)
   const int32_t* rows; int n_rows;              // rows null: every row, the result of the write is stored
   void* h; long h_stride; int h_f32;            // [n_rows, width] or null
   int store;
@@ -57,16 +61,10 @@ __device__ __forceinline__ void load_values(const void* base, bool f32, size_t a
   }
 }
 
+// Columns [c0, c0 + V) of row n: the write, the copies stored, and u of the read (unless nothing is read).
 // SC: the number of copies when the launcher knows a kernel for it (1 to 4), else 0: read from the arguments.
 template <int V, int SC>
-__global__ void __launch_bounds__(256) stream_step_kernel(const StreamStep a) {
-  pdl_launch_dependents();
-  pdl_wait();
-  const int r = blockIdx.y;
-  const int n = a.rows ? a.rows[r] : r;
-  if (n < 0) return;
-  const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * V;
-  if (c0 >= a.width) return;
+__device__ __forceinline__ void stream_columns(const StreamStep& a, int n, int c0, float (&u)[V]) {
   const int S = SC ? SC : a.copies, D = a.width;
   float* xr = a.x + (size_t)n * S * D + c0;
   float xs[kMaxCopies][V];
@@ -169,7 +167,6 @@ __global__ void __launch_bounds__(256) stream_step_kernel(const StreamStep a) {
       }
   }
   if (a.h == nullptr) return;
-  float u[V];
 #pragma unroll
   for (int j = 0; j < V; ++j) u[j] = 0.f;
 #pragma unroll
@@ -179,14 +176,11 @@ __global__ void __launch_bounds__(256) stream_step_kernel(const StreamStep a) {
 #pragma unroll
       for (int j = 0; j < V; ++j) u[j] = a.in_w ? __fmaf_rn(w, xs[s][j], u[j]) : u[j] + xs[s][j];
     }
-  if (a.alpha != nullptr) {
-    const float al = a.alpha[0];
-    float nw[V], nb[V];
-    load_values<V>(a.norm_w, true, c0, a.vec, nw);
-    load_values<V>(a.norm_b, true, c0, a.vec, nb);
-#pragma unroll
-    for (int j = 0; j < V; ++j) u[j] = __fmaf_rn(tanhf(al * u[j]), nw[j], nb[j]);
-  }
+}
+
+// h[r, c0 ..] = u.
+template <int V>
+__device__ __forceinline__ void store_read(const StreamStep& a, int r, int c0, const float (&u)[V]) {
   if (V == 4 && a.vec) {
     if (a.h_f32) {
       *reinterpret_cast<float4*>(reinterpret_cast<float*>(a.h) + (size_t)r * a.h_stride + c0) =
@@ -205,6 +199,70 @@ __global__ void __launch_bounds__(256) stream_step_kernel(const StreamStep a) {
     if (a.h_f32) reinterpret_cast<float*>(a.h)[(size_t)r * a.h_stride + c0 + j] = u[j];
     else reinterpret_cast<__nv_bfloat16*>(a.h)[(size_t)r * a.h_stride + c0 + j] = __float2bfloat16_rn(u[j]);
   }
+}
+
+template <int V, int SC>
+__global__ void __launch_bounds__(256) stream_step_kernel(const StreamStep a) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.y;
+  const int n = a.rows ? a.rows[r] : r;
+  if (n < 0) return;
+  const int c0 = (blockIdx.x * blockDim.x + threadIdx.x) * V;
+  if (c0 >= a.width) return;
+  float u[V];
+  stream_columns<V, SC>(a, n, c0, u);
+  if (a.h == nullptr) return;
+  if (a.alpha != nullptr) {
+    const float al = a.alpha[0];
+    float nw[V], nb[V];
+    load_values<V>(a.norm_w, true, c0, a.vec, nw);
+    load_values<V>(a.norm_b, true, c0, a.vec, nb);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = __fmaf_rn(tanhf(al * u[j]), nw[j], nb[j]);
+  }
+  store_read<V>(a, r, c0, u);
+}
+
+// With the root-mean-square norm: a block per row.  ONE: a thread has at most one group of V columns, which waits in
+// registers for the row's sum; otherwise u waits in shared memory.
+template <int V, int SC, bool ONE>
+__global__ void __launch_bounds__(V == 4 && SC == 0 ? 512 : 1024) stream_rms_kernel(const StreamStep a) {
+  extern __shared__ __align__(16) float u_s[];   // [width] unless ONE
+  __shared__ float scratch[32];
+  pdl_launch_dependents();
+  pdl_wait();
+  const int r = blockIdx.x;
+  const int n = a.rows ? a.rows[r] : r;
+  if (n < 0) return;
+  const int D = a.width, first = threadIdx.x * V, step = blockDim.x * V;
+  float u[V], ss = 0.f;
+  for (int c0 = first; c0 < D; c0 += step) {
+    stream_columns<V, SC>(a, n, c0, u);
+#pragma unroll
+    for (int j = 0; j < V; ++j) {
+      ss = __fmaf_rn(u[j], u[j], ss);
+      if (!ONE) u_s[c0 + j] = u[j];
+    }
+  }
+  const float k = 1.0f / sqrtf(block_sum(ss, scratch) / (float)D + a.rms_eps);
+  for (int c0 = first; c0 < D; c0 += step) {
+    float w[V];
+    load_values<V>(a.rms_w, true, c0, a.vec, w);
+#pragma unroll
+    for (int j = 0; j < V; ++j) u[j] = (ONE ? u[j] : u_s[c0 + j]) * k * w[j];
+    store_read<V>(a, r, c0, u);
+  }
+}
+
+template <int V, int SC>
+int launch_rms(const StreamStep& a, int count, cudaStream_t stream) {
+  const int groups = (a.width + V - 1) / V, most = V == 4 && SC == 0 ? 512 : 1024;
+  const int threads = groups < most ? (groups + 31) / 32 * 32 : most;
+  if (groups <= threads) return yalis_launch(stream_rms_kernel<V, SC, true>, dim3(count), dim3(threads), 0, stream, a);
+  const size_t smem = (size_t)a.width * sizeof(float);
+  if (smem > 48 * 1024) return YALIS_ERR_SHAPE;
+  return yalis_launch(stream_rms_kernel<V, SC, false>, dim3(count), dim3(512), smem, stream, a);
 }
 
 // x[n, :] += table[row(n), :] for every token of a request (float32 stream of one copy).
@@ -260,18 +318,19 @@ YALIS_API int yalis_stream_step(float* x, int n_tokens, int copies, int width, c
                                 int gate_f32, const float* layer_scale, const float* mix, const float* out_w,
                                 const float* in_w, const float* alpha, const float* norm_w, const float* norm_b,
                                 const int32_t* rows, int n_rows, void* h, long h_stride, int h_f32, const float* src,
-                                cudaStream_t stream) {
+                                const float* rms_w, float rms_eps, cudaStream_t stream) {
   if (copies < 1 || copies > kMaxCopies || width <= 0) return YALIS_ERR_SHAPE;
   if ((mix == nullptr) != (out_w == nullptr)) return YALIS_ERR_SHAPE;
   if ((alpha == nullptr) != (norm_w == nullptr) || (alpha == nullptr) != (norm_b == nullptr)) return YALIS_ERR_SHAPE;
   if (y != nullptr && !y_f32 && y_parts != 1) return YALIS_ERR_SHAPE;
+  if (rms_w != nullptr && (alpha != nullptr || h == nullptr)) return YALIS_ERR_SHAPE;
   const int count = rows ? n_rows : n_tokens;
   if (count <= 0) return YALIS_OK;
   StreamStep a;
   a.x = x; a.src = src; a.copies = copies; a.width = width; a.y = y; a.y_parts = y_parts; a.y_part_stride = y_part_stride;
   a.y_stride = y_stride; a.y_f32 = y_f32; a.gate = gate; a.gate_stride = gate_stride; a.gate_bias = gate_bias;
   a.gate_f32 = gate_f32; a.layer_scale = layer_scale; a.mix = mix; a.out_w = out_w; a.in_w = in_w; a.alpha = alpha;
-  a.norm_w = norm_w; a.norm_b = norm_b; a.rows = rows; a.n_rows = n_rows; a.h = h; a.h_stride = h_stride; a.h_f32 = h_f32;
+  a.norm_w = norm_w; a.norm_b = norm_b; a.rms_w = rms_w; a.rms_eps = rms_eps; a.rows = rows; a.n_rows = n_rows; a.h = h; a.h_stride = h_stride; a.h_f32 = h_f32;
   a.store = rows == nullptr ? 1 : 0;
   const bool wide = width % 4 == 0 && !((uintptr_t)x & 15) && !((uintptr_t)src & 15);
   // 8- and 16-byte accesses to everything beside x: every base and row stride must allow them
@@ -280,7 +339,18 @@ YALIS_API int yalis_stream_step(float* x, int n_tokens, int copies, int width, c
   };
   a.vec = wide && fits(y, y_f32, y_stride) && (y == nullptr || y_part_stride % 4 == 0) && fits(gate, gate_f32, gate_stride) &&
           fits(gate_bias, true, 0) && fits(layer_scale, true, 0) && fits(norm_w, true, 0) && fits(norm_b, true, 0) &&
+          fits(rms_w, true, 0) &&
           fits(h, h_f32, h_stride);
+  if (rms_w != nullptr) {
+    if (!wide) return launch_rms<1, 0>(a, count, stream);
+    switch (copies) {
+      case 1: return launch_rms<4, 1>(a, count, stream);
+      case 2: return launch_rms<4, 2>(a, count, stream);
+      case 3: return launch_rms<4, 3>(a, count, stream);
+      case 4: return launch_rms<4, 4>(a, count, stream);
+      default: return launch_rms<4, 0>(a, count, stream);
+    }
+  }
   const int per = wide ? 4 : 1;
   const int threads = 256;
   const dim3 grid((width + threads * per - 1) / (threads * per), count);

@@ -44,7 +44,8 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
                             out_scale: float = 1.0, chunk: Optional[int] = None,
                             sink_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
                             gate: Optional[torch.Tensor] = None, rel: Optional[torch.Tensor] = None,
-                            pool: Optional["PooledBlocks"] = None) -> torch.Tensor:
+                            pool: Optional["PooledBlocks"] = None,
+                            difference: Optional["MapDifference"] = None) -> torch.Tensor:
     """Exact attention of every token over the cached keys of its request.
 
     ``q`` may be the fused qkv matrix (only its first heads*head_dim columns are
@@ -55,14 +56,18 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
     [heads], 0 without them); ``gate`` [N, heads * v_head_dim], or [N, heads] for one number per head, multiplies the
     result by its sigmoid; ``rel`` (float32 [heads, L]) adds rel[h, min(p - j, L - 1)] to the scaled score; ``pool``
     (with a window) lets p see, beside its window, the pooled blocks that lie wholly before it (``PooledBlocks``);
-    ``v_head_dim`` is the head size of the values when it is not the keys'.  The result,
+    ``v_head_dim`` is the head size of the values when it is not the keys'; with ``difference`` every head has two maps
+    (``MapDifference``): ``head_dim`` is the size of one map's query, a head's two queries lie side by side in ``q``, and
+    the keys' pool holds [pages, kv_heads, page_size, 2 * head_dim].  The result,
     times ``out_scale``, is [N, heads*v_head_dim] in q's dtype (``out`` may be a
     column block of a wider matrix).
     """
     name = "paged_attention_generic"
     LAUNCHED["generic"] += 1
     vd = head_dim if v_head_dim is None else int(v_head_dim)
-    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads, head_dim, vd)
+    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads,
+                  _key_size(head_dim, difference), vd)
+    _check_difference(name, difference, sink, gate, pool)
     need(head_dim <= 256 and vd <= 256, name, f"head sizes {head_dim}, {vd} must be at most 256")
     n = q.shape[0]
     if out is None:
@@ -79,8 +84,32 @@ def paged_attention_generic(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch
         i32(k_pool.shape[0]), i32(n), i32(num_heads), i32(num_kv_heads), i32(head_dim), i32(vd), f32(scale),
         i32(window or 0), f32(softcap or 0.0), i32(int(sink)), f32(out_scale), i32(chunk or 0), ptr(sink_logits), ptr(slopes),
         ptr(gate), i32(gate.stride(0) if gate is not None else 0), i32(_per_head(gate, num_heads, vd)), ptr(rel),
-        i32(rel.shape[1] if rel is not None else 0), *pooled, stream()), name)
+        i32(rel.shape[1] if rel is not None else 0), *pooled, *_difference_arguments(difference), stream()), name)
     return out
+
+
+@dataclass(frozen=True)
+class MapDifference:
+    """Two attention maps per head over one value: with a1 and a2 the maps' results (each a softmax of its own), a head's
+    result is o / sqrt(mean(o^2) + eps) for o = a1 - balance * a2."""
+
+    balance: float
+    eps: float
+
+
+def _key_size(head_dim: int, difference: Optional[MapDifference]) -> int:
+    return head_dim if difference is None else 2 * head_dim
+
+
+def _check_difference(name, difference, *others) -> None:
+    need(difference is None or not any(o is not None and o is not False for o in others), name,
+         "two maps go without sinks, gates, biases, caps, chunks and pooled blocks")
+
+
+def _difference_arguments(difference: Optional[MapDifference]):
+    if difference is None:
+        return i32(1), f32(0.0), f32(0.0)
+    return i32(2), f32(difference.balance), f32(difference.eps)
 
 
 @dataclass(frozen=True)
@@ -169,6 +198,12 @@ def mma_extended_supports(head_dim: int, v_head_dim: int) -> bool:
     return bool(lib().yalis_attention_mma_extended_supports(i32(head_dim), i32(v_head_dim)))
 
 
+def mma_maps_supports(head_dim: int, v_head_dim: int) -> bool:
+    """Whether the tensor-core kernel's form of two maps takes these sizes: queries and keys of multiples of 16 up to 128
+    per map, values of multiples of 8 up to 256."""
+    return bool(lib().yalis_attention_mma_maps_supports(i32(head_dim), i32(v_head_dim)))
+
+
 def decode_splits(n_requests: int, num_kv_heads: int) -> int:
     """How many blocks share the keys of one (request, KV head) in a decode step, so that
     few requests still fill the GPU: as many as fit in ONE wave of two blocks per SM (a second,
@@ -233,7 +268,8 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
                         out_scale: float = 1.0, exact_weights: bool = False, chunk: Optional[int] = None,
                         sink_logits: Optional[torch.Tensor] = None, slopes: Optional[torch.Tensor] = None,
                         gate: Optional[torch.Tensor] = None, v_head_dim: Optional[int] = None,
-                        rel: Optional[torch.Tensor] = None, pool: Optional[PooledBlocks] = None) -> torch.Tensor:
+                        rel: Optional[torch.Tensor] = None, pool: Optional[PooledBlocks] = None,
+                        difference: Optional[MapDifference] = None) -> torch.Tensor:
     """Tensor-core attention (bfloat16) of the step's tokens over the cache; the same
     semantics as ``paged_attention_generic``.  ``q_start`` int32 [R+1] gives each request's
     token range; ``max_q_len`` bounds the launch grid.  ``n_splits`` > 1 divides the keys of
@@ -242,16 +278,20 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
     ``paged_attention_generic``; with any of them, or with
     ``exact_weights``, the softmax weights meet the values with 16 bits of mantissa (in two bfloat16 halves)
     instead of 8.  ``v_head_dim``, ``rel`` and ``pool`` as there too; they, and head sizes the other forms are not built
-    for, take the kernel's extended form.  ``out`` may be a column block of a wider matrix if it starts on a 16-byte
-    boundary.
+    for, take the kernel's extended form; ``difference`` (as there) the form of two maps.  ``out`` may be a column block
+    of a wider matrix if it starts on a 16-byte boundary.
     """
     name = "paged_attention_mma"
     LAUNCHED["mma"] += 1
     vd = head_dim if v_head_dim is None else int(v_head_dim)
     extended = vd != head_dim or rel is not None or pool is not None or not mma_supports(head_dim)
-    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads, head_dim, vd)
+    key_size, maps = _key_size(head_dim, difference), 1 if difference is None else 2
+    _check_common(name, q, k_pool, v_pool, positions, req_of_token, block_table, num_heads, num_kv_heads, key_size, vd)
+    _check_difference(name, difference, sink, gate, pool, softcap, chunk, slopes, rel)
     need(q.dtype == torch.bfloat16, name, "bfloat16 only (float32 goes to the generic kernel)")
-    need(mma_extended_supports(head_dim, vd) if extended else mma_supports(head_dim), name,
+    need(difference is None or mma_maps_supports(head_dim, vd), name,
+         f"head sizes {head_dim} (per map), {vd} are not built (multiples of 16 to 128, values of 8 to 256)")
+    need(difference is not None or (mma_extended_supports(head_dim, vd) if extended else mma_supports(head_dim)), name,
          f"head sizes {head_dim}, {vd} are not built (equal: multiples of 16 to 128, of 32 to 256; extended form: of 8 to 256)")
     n, r = q.shape[0], q_start.numel() - 1
     need(q_start.dtype == torch.int32 and q_start.is_contiguous() and q_start.is_cuda, name, "q_start must be int32 [R+1]")
@@ -270,17 +310,17 @@ def paged_attention_mma(q: torch.Tensor, k_pool: torch.Tensor, v_pool: torch.Ten
         need(max_q_len * (num_heads // num_kv_heads) <= 16, name, "splitting the keys is for decode steps only")
         floats = lib().yalis_attention_mma_scratch_floats
         floats.restype = ctypes.c_longlong
-        scratch = torch.empty(int(floats(i32(n), i32(num_heads), i32(vd), i32(n_splits))), dtype=torch.float32,
+        scratch = torch.empty(int(floats(i32(n), i32(maps * num_heads), i32(vd), i32(n_splits))), dtype=torch.float32,
                               device=q.device)
-        tickets = _tickets(q.device, r * num_kv_heads)
+        tickets = _tickets(q.device, r * num_kv_heads * maps)       # (two maps: up to two blocks of pairs each)
     check(lib().yalis_paged_attention_mma_general(
         ptr(q), i32(q.stride(0)), ptr(out), i32(out.stride(0)), ptr(k_pool), ptr(v_pool), ptr(positions), ptr(q_start),
         ptr(req_of_token), ptr(block_table), i32(block_table.shape[1]), i32(k_pool.shape[2]), i32(k_pool.shape[0]),
-        i32(n), i32(r), i32(max_q_len), i32(num_heads), i32(num_kv_heads), i32(head_dim), f32(scale), i32(window or 0),
+        i32(n), i32(r), i32(max_q_len), i32(num_heads), i32(num_kv_heads), i32(key_size), f32(scale), i32(window or 0),
         i32(n_splits), ptr(scratch), ptr(tickets), f32(softcap or 0.0), i32(int(sink)), f32(out_scale),
         i32(int(exact_weights)), i32(chunk or 0), ptr(sink_logits), ptr(slopes), ptr(gate),
         i32(gate.stride(0) if gate is not None else 0), i32(_per_head(gate, num_heads, vd)), i32(vd), ptr(rel),
-        i32(rel.shape[1] if rel is not None else 0), *pooled, stream()), name)
+        i32(rel.shape[1] if rel is not None else 0), *pooled, *_difference_arguments(difference), stream()), name)
     return out
 
 

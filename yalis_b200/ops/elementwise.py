@@ -252,22 +252,22 @@ ACTIVATIONS = {"gelu": ACT_GELU_ERF, "gelu_erf": ACT_GELU_ERF, "gelu_tanh": ACT_
 
 
 def activation(x: torch.Tensor, kind: str, out: Optional[torch.Tensor] = None,
-               bias: Optional[torch.Tensor] = None) -> torch.Tensor:
+               bias: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
     """act(x), or act(x + bias) with ``bias`` float32 [C], element by element in float32: ``gelu_erf`` 0.5 z (1 + erf(z / sqrt 2)), ``gelu_tanh``
     0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))), ``silu``, ``relu2`` (max(z, 0)^2) or ``tanh``.  ``x`` and ``out`` are [N, C] with unit inner
-    stride (column blocks of wider matrices are fine)."""
+    stride (column blocks of wider matrices are fine).  The result has the dtype of x, or is float32 (``out_dtype``)."""
     name = "activation"
     need_cuda(name, x, out)
     need(kind in ACTIVATIONS, name, f"unknown activation {kind!r} (one of {', '.join(ACTIVATIONS)})")
     need(x.dim() == 2 and x.stride(1) == 1, name, "x must be [N, C] with unit inner stride")
     if out is None:
-        out = torch.empty(x.shape, dtype=x.dtype, device=x.device)
-    need(out.shape == x.shape and out.dtype == x.dtype and out.stride(1) == 1, name, "bad out tensor")
+        out = torch.empty(x.shape, dtype=out_dtype or x.dtype, device=x.device)
+    need(out.shape == x.shape and out.dtype in (x.dtype, torch.float32) and out.stride(1) == 1, name, "bad out tensor")
     need_cuda(name, bias)
     need(bias is None or (bias.dtype == torch.float32 and bias.shape == (x.shape[1],) and bias.is_contiguous()), name,
          "the bias must be float32 [C]")
     check(lib().yalis_activation(ptr(x), i32(x.stride(0)), ptr(out), i32(out.stride(0)), i32(dtype_code(x.dtype)),
-                                 i32(x.shape[0]), i32(x.shape[1]), i32(ACTIVATIONS[kind]), ptr(bias), stream()), name)
+                                 i32(int(out.dtype == torch.float32)), i32(x.shape[0]), i32(x.shape[1]), i32(ACTIVATIONS[kind]), ptr(bias), stream()), name)
     return out
 
 
@@ -292,7 +292,7 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
                 bad_flag: Optional[torch.Tensor] = None, interleaved: bool = False, q_temperature=None,
                 rot_scale: float = 1.0, norm_all: bool = False, pool: int = 0, pooled_k: Optional[torch.Tensor] = None,
                 pooled_v: Optional[torch.Tensor] = None, pooled_table: Optional[torch.Tensor] = None,
-                single_tokens: bool = False):
+                single_tokens: bool = False, maps: int = 1):
     """Prepares the heads of a mixer from its input projection ``src`` [N, ...] (model dtype), whose query,
     key and value heads start at the columns ``offsets`` = (q, k, v):
 
@@ -303,6 +303,9 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
         times ``rot_scale``;
         q <- q * q_scale, k <- k * k_scale;  with ``q_temperature`` = (coef, every) also
         q <- q * (1 + coef * ln(floor((position + 1) / every) + 1)).
+
+    ``maps`` M > 1: a key/value head has M keys of size ``dim``, side by side in ``src`` and in a row of the pool
+    [pages, nk, page_size, M * dim]; ``nk`` counts key/value heads, ``nq`` every query of size ``dim``.
 
     With pools, keys [pages, nk, page_size, dim] and values [pages, nk, page_size, vdim] are written to the pages
     of ``block_table`` (not at all when ``store`` is False) and the queries [N, nq * dim] are returned.  With ``pool``
@@ -315,13 +318,13 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
     need(src.dim() == 2 and src.stride(1) == 1, name, "src must be [N, ...] with unit inner stride")
     n = src.shape[0]
     q_off, k_off, v_off = (int(o) for o in offsets)
-    need(max(q_off + nq * dim, k_off + nk * dim, v_off + nk * vdim) <= src.shape[1], name, "head columns lie outside src")
+    need(max(q_off + nq * dim, k_off + nk * maps * dim, v_off + nk * vdim) <= src.shape[1], name, "head columns lie outside src")
     for t in (positions, req_of_token):
         need(t.dtype == torch.int32 and t.shape == (n,) and t.is_contiguous(), name, "positions/req_of_token: int32 [N]")
-    for b, width in zip(biases, (nq * dim, nk * dim, nk * vdim)):
+    for b, width in zip(biases, (nq * dim, nk * maps * dim, nk * vdim)):
         need(b is None or (b.dtype == src.dtype and b.shape == (width,) and b.is_contiguous()), name,
              "a bias must be a contiguous vector over its heads in the dtype of src")
-    for w, heads in ((q_norm, nq), (k_norm, nk)):
+    for w, heads in ((q_norm, nq), (k_norm, nk * maps)):
         need(w is None or (w.dtype == torch.float32 and w.shape == ((heads * dim if norm_all else dim),) and w.is_contiguous()),
              name, "a norm scale must be float32 [dim], or [heads * dim] when the norm is over all heads")
     rot_dims = 0
@@ -338,19 +341,19 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
         need(out_dtype == src.dtype, name, "with pools the queries keep the dtype of src")
         need(v_pool is not None and block_table is not None and k_pool.dtype == v_pool.dtype == src.dtype
              and k_pool.dim() == 4 and v_pool.dim() == 4 and k_pool.shape[:3] == v_pool.shape[:3]
-             and k_pool.shape[1] == nk and k_pool.shape[3] == dim and v_pool.shape[3] == vdim
+             and k_pool.shape[1] == nk and k_pool.shape[3] == maps * dim and v_pool.shape[3] == vdim
              and k_pool.is_contiguous() and v_pool.is_contiguous(), name,
              "pools must be contiguous [pages, kv_heads, page_size, dim] and [..., vdim] in the dtype of src")
         need(block_table.dtype == torch.int32 and block_table.dim() == 2 and block_table.is_contiguous(), name,
              "block_table must be contiguous int32 [R, width]")
         num_pages, page_size, table_width = k_pool.shape[0], k_pool.shape[2], block_table.shape[1]
     else:
-        k_out = torch.empty((n, nk * dim), dtype=out_dtype, device=src.device)
+        k_out = torch.empty((n, nk * maps * dim), dtype=out_dtype, device=src.device)
         v_out = torch.empty((n, nk * vdim), dtype=out_dtype, device=src.device)
     pooled_width = pooled_page = pooled_pages = 0
     if pool:
         need_cuda(name, pooled_k, pooled_v, pooled_table)
-        need(paged and store and pool > 0, name, "pooled blocks need pages to store to")
+        need(paged and store and pool > 0 and maps == 1, name, "pooled blocks need pages to store to, and one key per head")
         need(pooled_k is not None and pooled_v is not None and pooled_k.shape[:3] == pooled_v.shape[:3]
              and pooled_k.dim() == 4 and pooled_k.shape[1] == nk and pooled_k.shape[3] == dim and pooled_v.shape[3] == vdim
              and pooled_k.dtype == pooled_v.dtype == src.dtype and pooled_k.is_contiguous() and pooled_v.is_contiguous(), name,
@@ -371,5 +374,5 @@ def qkv_prepare(src: torch.Tensor, offsets, nq: int, nk: int, dim: int, vdim: in
         i32(table_width), i32(page_size), i32(num_pages), ptr(positions), ptr(req_of_token), i32(n), i32(nq), i32(nk),
         i32(dim), i32(vdim), ptr(bad_flag), i32(pool), ptr(pooled_k if pool else None), ptr(pooled_v if pool else None),
         ptr(pooled_table if pool else None), i32(pooled_width), i32(pooled_page), i32(pooled_pages), i32(int(single_tokens)),
-        stream()), name)
+        i32(maps), stream()), name)
     return q_out if paged else (q_out, k_out, v_out)

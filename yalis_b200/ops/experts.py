@@ -39,13 +39,20 @@ def _score_code(name: str, score: str) -> int:
 
 
 def route(x: torch.Tensor, router: torch.Tensor, top: int, eps: Optional[float] = 1e-20, req_of_token: Optional[torch.Tensor] = None,
-          factor: float = 1.0, score: str = "softmax", side: Optional[torch.Tensor] = None):
+          factor: float = 1.0, score: str = "softmax", side: Optional[torch.Tensor] = None,
+          correction: Optional[torch.Tensor] = None, groups=None, identity: int = 0):
     """``route_topk`` of the logits ``x router^T`` in one launch: ``x`` [N, K] (float32 or bfloat16, unit inner stride),
     ``router`` float32 [E, K].  The logits are float32 sums in a fixed order per (token, expert).  With ``side``
-    (float32 [K]) a third result is returned: float32 [N], sigmoid(x . side), a gate per token from the same rows."""
+    (float32 [K]) a third result is returned: float32 [N], sigmoid(x . side), a gate per token from the same rows.
+
+    ``correction`` (float32 [E]) is added to the scores for the choice alone: the weights are the scores without it.
+    ``groups`` = (count, keep): the E outputs form ``count`` equal groups of neighbours, a group's score is the largest
+    choice score in it, and only members of the ``keep`` best groups can be chosen.  With ``identity`` I > 0 the last I
+    outputs stand for experts that return their input: their ids appear like any others, and one more result is
+    returned: float32 [N], the sum of a token's weights of such experts."""
     name = "route"
-    need_cuda(name, x, router, req_of_token, side)
-    side_out = None
+    need_cuda(name, x, router, req_of_token, side, correction)
+    side_out = identity_out = None
     if side is not None:
         need(side.dtype == torch.float32 and side.shape == (x.shape[1],) and side.is_contiguous(), name, "side must be float32 [K]")
         side_out = torch.zeros(x.shape[0], dtype=torch.float32, device=x.device)
@@ -53,12 +60,21 @@ def route(x: torch.Tensor, router: torch.Tensor, top: int, eps: Optional[float] 
          and router.shape[1] == x.shape[1], name, "x [N, K], router contiguous float32 [E, K]")
     n, e = x.shape[0], router.shape[0]
     need(0 < top <= min(e, MAX_TOP) and e <= MAX_EXPERTS, name, f"needs top <= min(E, {MAX_TOP}) and E <= {MAX_EXPERTS}")
+    need(correction is None or (correction.dtype == torch.float32 and correction.shape == (e,) and correction.is_contiguous()), name,
+         "the correction must be float32 [E]")
+    count, keep = (0, 0) if groups is None else (int(v) for v in groups)
+    need(groups is None or (count > 0 and e % count == 0 and 0 < keep <= count and keep * (e // count) >= top), name,
+         f"groups {groups} do not divide {e} outputs or leave fewer than {top} to choose from")
+    need(0 <= identity <= e, name, "at most all outputs are identity experts")
+    if identity:
+        identity_out = torch.empty(n, dtype=torch.float32, device=x.device)
     ids = torch.empty((n, top), dtype=torch.int32, device=x.device)
     weights = torch.empty((n, top), dtype=torch.float32, device=x.device)
     check(lib().yalis_route(ptr(x), i32(dtype_code(x.dtype)), i64(x.stride(0)), ptr(router), i32(n), i32(e), i32(x.shape[1]), i32(top),
                             f32(-1.0 if eps is None else eps), f32(factor), ptr(req_of_token), ptr(ids), ptr(weights),
-                            i32(_score_code(name, score)), ptr(side), ptr(side_out), stream()), name)
-    return (ids, weights) if side is None else (ids, weights, side_out)
+                            i32(_score_code(name, score)), ptr(side), ptr(side_out), ptr(correction), i32(count), i32(keep), i32(e - identity),
+                            ptr(identity_out), stream()), name)
+    return (ids, weights) + tuple(t for t in (side_out, identity_out) if t is not None)
 
 
 @dataclass
@@ -79,6 +95,7 @@ class ExpertPlan:
 
 
 def expert_plan(ids: torch.Tensor, n_experts: int, bm: int) -> ExpertPlan:
+    """Entries whose id is negative or at least ``n_experts`` (no request's, an identity expert's) take no slot."""
     name = "expert_plan"
     need_cuda(name, ids)
     need(ids.dtype == torch.int32 and ids.dim() == 2 and ids.is_contiguous(), name, "ids must be contiguous int32 [N, top]")

@@ -231,9 +231,10 @@ def general_delta_prepare(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, a_r
 
 
 def gate_norm(o: torch.Tensor, z: torch.Tensor, parts: int, weight: torch.Tensor, eps: float, req_of_token: torch.Tensor,
-              out: torch.Tensor, out_scale: float = 1.0) -> torch.Tensor:
-    """y = o * silu(z), then each of ``parts`` equal column ranges divided by its own root mean square
-    (sqrt(mean(y^2) + eps)), times ``weight`` and ``out_scale``.  ``o`` float32 [N, C]; ``z`` [N, C] in the dtype of
+              out: torch.Tensor, out_scale: float = 1.0, gate_kind: int = GATE_SILU, after: bool = False) -> torch.Tensor:
+    """y = o * act(z), then each of ``parts`` equal column ranges divided by its own root mean square
+    (sqrt(mean(y^2) + eps)), times ``weight`` and ``out_scale``; with ``after`` the norm and the weight come first, on o,
+    and then act(z).  act: silu or sigmoid (``gate_kind``).  ``o`` float32 [N, C]; ``z`` [N, C] in the dtype of
     ``out``; ``weight`` float32 [C]; ``out`` [N, C] (column blocks of wider matrices are fine)."""
     name = "gate_norm"
     need_cuda(name, o, z, weight, req_of_token, out)
@@ -241,11 +242,12 @@ def gate_norm(o: torch.Tensor, z: torch.Tensor, parts: int, weight: torch.Tensor
     need(o.dtype == torch.float32 and o.stride(1) == 1, name, "o must be float32 [N, C] with unit inner stride")
     need(z.shape == (n, c) and z.stride(1) == 1 and z.dtype == out.dtype, name, "z must be [N, C] in the output's dtype")
     need(out.shape == (n, c) and out.stride(1) == 1, name, "out must be [N, C] with unit inner stride")
+    need(gate_kind in (GATE_SILU, GATE_SIGMOID), name, "the gate is silu or sigmoid")
     need(parts > 0 and c % parts == 0, name, f"{c} columns do not divide into {parts} parts")
     need(weight.dtype == torch.float32 and weight.shape == (c,) and weight.is_contiguous(), name, "weight must be float32 [C]")
     need(req_of_token.dtype == torch.int32 and req_of_token.shape == (n,) and req_of_token.is_contiguous(), name,
          "req_of_token must be int32 [N]")
     check(lib().yalis_gate_norm(ptr(o), i32(o.stride(0)), ptr(z), i32(z.stride(0)), ptr(weight), ptr(out), i32(out.stride(0)),
                                 i32(dtype_code(out.dtype)), ptr(req_of_token), i32(n), i32(parts), i32(c // parts), f32(eps),
-                                f32(out_scale), stream()), name)
+                                f32(out_scale), i32(gate_kind), i32(int(after)), stream()), name)
     return out

@@ -7,7 +7,7 @@ from typing import Optional, Tuple
 
 import torch
 
-from ._lib import check, dtype_code, i32, i64, lib, need, need_cuda, ptr, stream
+from ._lib import check, dtype_code, f32, i32, i64, lib, need, need_cuda, ptr, stream
 
 MAX_COPIES = 8
 
@@ -18,14 +18,16 @@ def stream_step(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, gate: Opti
                 in_weights: Optional[torch.Tensor] = None,
                 norm: Optional[Tuple[torch.Tensor, torch.Tensor, torch.Tensor]] = None,
                 rows: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None,
-                read: bool = True, source: Optional[torch.Tensor] = None) -> Optional[torch.Tensor]:
+                read: bool = True, source: Optional[torch.Tensor] = None,
+                rms: Optional[Tuple[torch.Tensor, float]] = None) -> Optional[torch.Tensor]:
     """One pass over the stream ``x`` float32 [N, S, D] (S copies; [N, D] counts as one copy).
 
     Write, when ``y`` is given ([N, D] in float32 or bfloat16, or float32 partial sums [P, N, D] added in order):
     y <- y * layer_scale * sigmoid(gate + gate_bias) (each factor optional; ``gate`` [N, D] float32 or bfloat16), then
     x_t <- sum_s mix[s, t] x_s + out_weights[t] y for all copies from the old ones (without ``mix``: x_t += y).
     Read, when ``read``: u = sum_s in_weights[s] x_s (without ``in_weights``: the sum), h = tanh(alpha u) w + b with
-    ``norm`` = (alpha [1], w [D], b [D]), else h = u; returned as [N, D] in ``out_dtype``.
+    ``norm`` = (alpha [1], w [D], b [D]), h = u / sqrt(mean(u^2) + eps) w with ``rms`` = (w [D], eps), else h = u; returned
+    as [N, D] in ``out_dtype``.
 
     With ``rows`` (int32 row indices, -1: skip) only those rows are read, into [len(rows), D], and the written copies are
     not stored: the stream stays as it was.
@@ -63,6 +65,11 @@ def stream_step(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, gate: Opti
         need(alpha.dtype == torch.float32 and alpha.numel() == 1 and w.dtype == b.dtype == torch.float32
              and w.shape == b.shape == (d,) and w.is_contiguous() and b.is_contiguous(), name,
              "norm must be (alpha float32 [1], w float32 [D], b float32 [D])")
+    rms_w, rms_eps = (None, 0.0) if rms is None else rms
+    if rms_w is not None:
+        need_cuda(name, rms_w)
+        need(norm is None and read and rms_w.dtype == torch.float32 and rms_w.shape == (d,) and rms_w.is_contiguous(), name,
+             "rms must be (w float32 [D], eps), belongs to a read and excludes norm")
     if rows is not None:
         need(rows.dtype == torch.int32 and rows.dim() == 1 and rows.is_contiguous(), name, "rows must be int32 [R]")
     count = n if rows is None else rows.numel()
@@ -78,7 +85,8 @@ def stream_step(x: torch.Tensor, *, y: Optional[torch.Tensor] = None, gate: Opti
         i32(int(y is not None and y.dtype == torch.float32)), ptr(gate), i64(gate.stride(0) if gate is not None else 0),
         ptr(gate_bias), i32(int(gate is not None and gate.dtype == torch.float32)), ptr(layer_scale), ptr(mix), ptr(out_weights),
         ptr(in_weights), ptr(alpha), ptr(w), ptr(b), ptr(rows), i32(0 if rows is None else rows.numel()), ptr(h),
-        i64(h.stride(0) if h is not None else 0), i32(int(h is not None and h.dtype == torch.float32)), ptr(source), stream()), name)
+        i64(h.stride(0) if h is not None else 0), i32(int(h is not None and h.dtype == torch.float32)), ptr(source),
+        ptr(rms_w), f32(rms_eps), stream()), name)
     return h
 
 

@@ -146,7 +146,12 @@ class GeneralAttention(Mixer, Projected):
     before the window: the means of the block's keys and values as the cache holds them; tokens and blocks share one
     softmax), ``q_temperature`` ({"coef", "every"}: the query at position p is multiplied by
     1 + coef ln(floor((p + 1) / every) + 1)), ``gate`` (the heads' results are multiplied by sigmoid(W_g x), one more
-    matrix over the mixer's input; ``"head"``: one number per head instead of one per element), ``out_bias`` (a bias on the output product), ``own_kv`` (False: the mixer has no
+    matrix over the mixer's input; ``"head"``: one number per head instead of one per element), ``difference`` ({"offset":
+    d, "eps"}: two maps per head over the same values: q and k have two parts of ``head_dim`` sizes per head, side by side,
+    each with the norm and rotation of a head of its own; each pair of parts is an attention of its own, and of the maps'
+    results a1 and a2 the head's is (1 - d) o / sqrt(mean(o^2) + eps) with o = a1 - b a2 and b = exp(lq1 . lk1) -
+    exp(lq2 . lk2) + d, one number for the layer from the learned vectors ``lq1`` ... ``lk2`` [head_dim]),
+    ``out_bias`` (a bias on the output product), ``own_kv`` (False: the mixer has no
     key and value projections and reads the cache of the schedule entry it is pointed at; default True),
     ``cache_window`` (how many positions back the keys are kept, when that is not the mixer's own ``window`` or
     ``chunk``: the widest reach among this mixer and the mixers that read its cache), ``out_scale``.  Scores, weights
@@ -185,6 +190,14 @@ class GeneralAttention(Mixer, Projected):
         if p.get("cache_window") is None and self.window is not None and self.chunk is not None:
             self.cache_window = min(self.window, self.chunk)
         self.out_scale = float(p.get("out_scale", 1.0))
+        df = p.get("difference")
+        self.difference = (float(df["offset"]), float(df["eps"])) if df is not None else None
+        self.maps = 1 if df is None else 2
+        self.combine: Optional[attn_ops.MapDifference] = None
+        if df is not None and (self.sink or self.softcap is not None or self.chunk is not None or self.slopes_host is not None
+                               or self.distance_bias is not None or self.pool is not None or self.gated or self.values_from_keys
+                               or self.norm_all or not self.own_kv or self.out_scale != 1.0):
+            raise ValueError("two maps per head go with a window, a norm per head and a rotation only")
         if self.slopes_host is not None and len(self.slopes_host) != self.nh:
             raise ValueError(f"{len(self.slopes_host)} distance slopes for {self.nh} heads")
         if self.chunk is not None and self.chunk <= 0 or self.q_temperature is not None and self.q_temperature[1] <= 0:
@@ -213,15 +226,16 @@ class GeneralAttention(Mixer, Projected):
         self.spans = {}
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        specs = {"q_proj": ParamSpec((self.nh * self.hs, self.hidden)), "o_proj": ParamSpec((self.hidden, self.nh * self.vd))}
+        qd, kd = self._query_rows(), self._key_rows()
+        specs = {"q_proj": ParamSpec((qd, self.hidden)), "o_proj": ParamSpec((self.hidden, self.nh * self.vd))}
         if self.own_kv:
-            specs["k_proj"] = ParamSpec((self.g * self.hs, self.hidden))
+            specs["k_proj"] = ParamSpec((kd, self.hidden))
             if not self.values_from_keys:
                 specs["v_proj"] = ParamSpec((self.g * self.vd, self.hidden))
         if self.bias:
-            specs["q_bias"] = ParamSpec((self.nh * self.hs,), init="zeros")
+            specs["q_bias"] = ParamSpec((qd,), init="zeros")
             if self.own_kv:
-                specs.update({"k_bias": ParamSpec((self.g * self.hs,), init="zeros"), "v_bias": ParamSpec((self.g * self.vd,), init="zeros")})
+                specs.update({"k_bias": ParamSpec((kd,), init="zeros"), "v_bias": ParamSpec((self.g * self.vd,), init="zeros")})
         if self.norm_eps is not None and self.norm_weight:
             specs["q_norm"] = ParamSpec((self.nh * self.hs if self.norm_all else self.hs,), init="ones", keep_float32=True)
             if self.own_kv:
@@ -234,7 +248,15 @@ class GeneralAttention(Mixer, Projected):
             specs["g_proj"] = ParamSpec((self.nh if self.gate_per_head else self.nh * self.vd, self.hidden))
         if self.out_bias:
             specs["o_bias"] = ParamSpec((self.hidden,), init="zeros", keep_float32=True)
+        if self.difference is not None:
+            specs.update({n: ParamSpec((self.hs,), keep_float32=True) for n in ("lq1", "lk1", "lq2", "lk2")})
         return specs
+
+    def _query_rows(self) -> int:
+        return self.nh * self.maps * self.hs
+
+    def _key_rows(self) -> int:
+        return self.g * self.maps * self.hs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         # the input matrices stacked, each block of the product's columns on a 16-byte boundary
@@ -243,7 +265,7 @@ class GeneralAttention(Mixer, Projected):
         plain = not self.gated and self.own_kv and not self.values_from_keys
         if plain:
             self.w_in = torch.cat([t[n] for n in names], dim=0).contiguous()
-            qd, kd = self.nh * self.hs, self.g * self.hs
+            qd, kd = self._query_rows(), self._key_rows()
             spans = [(0, qd), (qd, qd + kd), (qd + kd, qd + kd + self.g * self.vd)]
         else:
             from .base import stack_rows
@@ -269,6 +291,10 @@ class GeneralAttention(Mixer, Projected):
             self.slopes = torch.tensor(self.slopes_host, dtype=torch.float32, device=self.w_in.device)
         if self.out_bias:
             self.o_bias = t["o_bias"].float().contiguous()
+        if self.difference is not None:
+            dot = lambda a, b: float((t[a].double() * t[b].double()).sum())
+            offset, eps = self.difference
+            self.combine = attn_ops.MapDifference(math.exp(dot("lq1", "lk1")) - math.exp(dot("lq2", "lk2")) + offset, eps)
 
     def in_weight(self) -> torch.Tensor:
         return self.w_in
@@ -283,6 +309,8 @@ class GeneralAttention(Mixer, Projected):
 
     def cache_request(self):
         vd = None if self.vd == self.hs else self.vd
+        if self.difference is not None:
+            return PagedKV(self.g, self.maps * self.hs, self.cache_window, v_head_dim=self.vd)
         tokens = PagedKV(self.g, self.hs, self.cache_window, v_head_dim=vd)
         if self.pool is None:
             return tokens
@@ -294,6 +322,8 @@ class GeneralAttention(Mixer, Projected):
         kernel."""
         if dtype != torch.bfloat16:
             return False
+        if self.difference is not None:
+            return attn_ops.mma_maps_supports(self.hs, self.vd)
         plain = self.vd == self.hs and self.distance_bias is None and self.pool is None and attn_ops.mma_supports(self.hs)
         return plain or attn_ops.mma_extended_supports(self.hs, self.vd)
 
@@ -301,7 +331,8 @@ class GeneralAttention(Mixer, Projected):
         """(longest portion, key splits): a step in which a request's rows fill at most one tile of 16 (single
         tokens of up to 16 heads per group) may divide each request's keys among blocks."""
         rows = host.max_q_len * (self.nh // self.g)
-        return host.max_q_len, (attn_ops.decode_splits(len(host.slots), self.g) if rows <= 16 else 1)
+        blocks = self.g * (2 if self.difference is not None and rows > 8 else 1)      # two maps: eight rows of each a block
+        return host.max_q_len, (attn_ops.decode_splits(len(host.slots), blocks) if rows <= 16 else 1)
 
     def capture_key(self, host):
         # the exact kernel launches the same for every step; the tensor-core one by the longest portion
@@ -321,7 +352,7 @@ class GeneralAttention(Mixer, Projected):
     def mixing_flops(self, q_len: int, ctx_before: int) -> float:
         keys = sum(self.keys_seen(ctx_before + t) + self.blocks_seen(ctx_before + t) for t in range(q_len)) if self.window or self.chunk \
             else q_len * ctx_before + q_len * (q_len + 1) / 2
-        return 2.0 * self.nh * (self.hs + self.vd) * keys
+        return 2.0 * self.nh * self.maps * (self.hs + self.vd) * keys
 
     def mix(self, z: torch.Tensor, ctx, cache, y: torch.Tensor) -> None:
         if self.position is None:
@@ -342,30 +373,32 @@ class GeneralAttention(Mixer, Projected):
         v_at = self.spans["v_proj"][0] if "v_proj" in self.spans else k_at
         pooling = {} if blocks is None else dict(pool=blocks.size, pooled_k=blocks.k, pooled_v=blocks.v, pooled_table=blocks.table,
                                                  single_tokens=ctx.host.max_q_len == 1)
-        q = qkv_prepare(z, (q_at, k_at, v_at), self.nh, self.g, self.hs, self.vd, ctx.positions, ctx.req_of_token,
+        q = qkv_prepare(z, (q_at, k_at, v_at), self.nh * self.maps, self.g, self.hs, self.vd, ctx.positions, ctx.req_of_token,
                         out_dtype=z.dtype, biases=self.biases, q_norm=self.q_norm, k_norm=self.k_norm,
                         norm_eps=self.norm_eps or 0.0, inv_freq=freq, k_pool=cache.k, v_pool=cache.v, block_table=table,
                         store=cache.writable, bad_flag=ctx.error_flag, interleaved=interleaved,
-                        q_temperature=self.q_temperature, rot_scale=magnitude, norm_all=self.norm_all, **pooling)
+                        q_temperature=self.q_temperature, rot_scale=magnitude, norm_all=self.norm_all,
+                        maps=self.maps, **pooling)
         gate = None
         if self.gated:
             a, b = self.spans["g_proj"]
             gate = z[:, a:b]
         extras = dict(chunk=self.chunk, sink_logits=self.sink_logits, slopes=self.slopes, gate=gate, rel=self.rel, pool=blocks,
                       v_head_dim=self.vd)
+        scale_out = self.out_scale if self.difference is None else 1.0 - self.difference[0]
         if self._tensor_core_form(z.dtype):
             longest, splits = self._launch_shape(ctx.host)
             direct = y.data_ptr() % 16 == 0 and y.stride(0) % 2 == 0
             out = attn_ops.paged_attention_mma(q, cache.k, cache.v, ctx.positions, ctx.q_start, ctx.req_of_token, table, longest,
                                                self.nh, self.g, self.hs, scale=self.scale, window=self.window, n_splits=splits,
                                                out=y if direct else None, softcap=self.softcap, sink=self.sink,
-                                               out_scale=self.out_scale, exact_weights=True, **extras)
+                                               out_scale=scale_out, exact_weights=True, difference=self.combine, **extras)
             if not direct:
                 y.copy_(out)
             return
         attn_ops.paged_attention_generic(q, cache.k, cache.v, ctx.positions, ctx.req_of_token, table, self.nh, self.g, self.hs,
                                          scale=self.scale, window=self.window, out=y,
-                                         softcap=self.softcap, sink=self.sink, out_scale=self.out_scale, **extras)
+                                         softcap=self.softcap, sink=self.sink, out_scale=scale_out, difference=self.combine, **extras)
 
     def forward(self, x: torch.Tensor, ctx, cache: PagedKVCache):
         out = self.project_and_mix(x, ctx, cache)

@@ -5,8 +5,8 @@ all copies at once, x_t <- sum_s mix[s, t] x_s + out_t y.  Before the write y ma
 by a learned vector (``layer_scale``) and by a gate sigmoid(W_g h + b_g) computed from what the sub-layer read
 (``gate``).  With one copy and no mixing this is the plain residual sum with those two factors.
 
-``scaled_sum`` (category ``connection``): the plain residual sum of a stream of one copy with a learned vector on the
-sub-layer's result, x += y * scale; the vector rides along with the result into the pass that adds it.
+``scaled_sum`` (category ``connection``): the plain residual sum of a stream of one copy with a learned vector and a
+constant on the sub-layer's result, x += y * scale * factor; both ride along with the result into the pass that adds it.
 
 ``pre_norm_connected`` (category ``block``): x <- write_1(mixer(norm_1(read_1 x))), then the same with the
 feed-forward, if the layer has one.  The norm reads the copies, applies the pending write of the sub-layer before
@@ -28,7 +28,8 @@ from .base import Block, Connection, NormedSum, ParamSpec, PendingWrite, Residua
 
 class HyperConnection(Connection):
     """Parameters: ``hidden_size``, ``copies`` (of the stream), ``mixing`` (bool: learned read weights, write weights
-    and a matrix that mixes the copies; False: the plain sum), ``layer_scale`` (bool), ``gate`` (bool)."""
+    and a matrix that mixes the copies; False: the plain sum), ``layer_scale`` (bool), ``gate`` (bool), ``factor`` (a
+    constant on the result, which joins the write weights; it needs them; default 1)."""
 
     def __init__(self, spec: PartSpec):
         super().__init__(spec)
@@ -38,6 +39,9 @@ class HyperConnection(Connection):
         self.has_scale, self.has_gate = bool(p.get("layer_scale", False)), bool(p.get("gate", False))
         if not 1 <= self.copies <= MAX_COPIES:
             raise ValueError(f"a stream has 1 to {MAX_COPIES} copies, not {self.copies}")
+        self.factor = float(p.get("factor", 1.0))
+        if self.factor != 1.0 and not self.mixing:
+            raise ValueError("a constant on the result needs the write weights that carry it")
         if self.copies > 1 and not self.mixing:
             raise ValueError("a stream of several copies needs the mixing weights")
         self.w_in = self.w_out = self.mix = self.scale = self.gate_w = self.gate_b = None
@@ -57,7 +61,7 @@ class HyperConnection(Connection):
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
         if self.mixing:
-            self.w_in, self.w_out, self.mix = t["in"].contiguous(), t["out"].contiguous(), t["mix"].contiguous()
+            self.w_in, self.w_out, self.mix = t["in"].contiguous(), (t["out"] * self.factor).contiguous(), t["mix"].contiguous()
         if self.has_scale:
             self.scale = t["scale"].contiguous()
         if self.has_gate:
@@ -78,24 +82,26 @@ class HyperConnection(Connection):
 
 
 class ScaledSum(Connection):
-    """x += y * scale.  Parameters: ``hidden_size``.  The scale is held in float32."""
+    """x += y * scale * factor.  Parameters: ``hidden_size``, ``learned`` (False: no scale; default True), ``factor`` (a
+    constant, default 1).  The scale is held in float32."""
 
     def __init__(self, spec: PartSpec):
         super().__init__(spec)
         self.hidden = int(spec.params["hidden_size"])
+        self.learned, self.factor = bool(spec.params.get("learned", True)), float(spec.params.get("factor", 1.0))
         self.scale: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
-        return {"scale": ParamSpec((self.hidden,), init="ones", keep_float32=True)}
+        return {"scale": ParamSpec((self.hidden,), init="ones", keep_float32=True)} if self.learned else {}
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
-        self.scale = t["scale"].contiguous()
+        self.scale = t["scale"].contiguous() if self.learned else None
 
     def write(self, h: torch.Tensor, y) -> NormedSum:
         result = y if isinstance(y, NormedSum) else NormedSum(y)
         if result.scale is not None:
             raise ValueError("the result already carries a scale")
-        return replace(result, scale=self.scale)
+        return replace(result, scale=self.scale, factor=result.factor * self.factor)
 
     def capture_key(self, host):
         return None

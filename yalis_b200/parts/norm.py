@@ -15,7 +15,8 @@ from .base import Norm, NormedSum, ParamSpec, PendingWrite, ResidualStream, regi
 class RMSNorm(Norm):
     """Parameters: ``size`` (width of the stream), ``eps``, ``one_plus`` (the stored tensor w lies around
     zero and the scale is 1 + w; default False: the tensor is the scale), ``scalar`` (the stored tensor is one number,
-    the scale of every coordinate).  The scale is held in float32."""
+    the scale of every coordinate).  The scale is held in float32.  A stream kept in copies is read as their weighted sum,
+    after whatever write is pending, in the same pass that applies the write."""
 
     def __init__(self, spec: PartSpec):
         super().__init__(spec)
@@ -33,12 +34,21 @@ class RMSNorm(Norm):
         w = w.reshape(1).expand(self.size).contiguous() if self.scalar else w.contiguous()
         self.weight = (1.0 + w) if self.one_plus else w       # float32: the sum is exact to one rounding
 
-    def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None) -> torch.Tensor:
-        if stream.copies > 1:
-            raise ValueError("rms_norm reads a stream of one copy")
+    def forward(self, stream: ResidualStream, rows: Optional[torch.Tensor] = None,
+                in_weights: Optional[torch.Tensor] = None) -> torch.Tensor:
+        """``in_weights`` [copies]: the weights of the copies in the sum that is normed (None: the plain sum)."""
+        if stream.x.dim() == 3 or in_weights is not None or isinstance(stream.pending, PendingWrite):
+            from yalis_b200.ops.streams import stream_step
+            if isinstance(stream.pending, NormedSum):
+                stream.flush()
+            pending = stream.pending
+            write = pending.arguments() if isinstance(pending, PendingWrite) else ({"y": pending} if pending is not None else {})
+            h = stream_step(stream.x, rms=(self.weight, self.eps), in_weights=in_weights, rows=rows, out_dtype=stream.dtype,
+                            source=stream.take_source(stores=rows is None), **write)
+            if rows is None:
+                stream.pending = None   # the kernel has stored the written copies
+            return h
         stream.materialize()
-        if isinstance(stream.pending, PendingWrite):
-            stream.flush()
         if isinstance(stream.pending, NormedSum):      # a result with a bias or a norm of its own: the same single pass
             pend = stream.pending
             y = add_normed_rmsnorm(stream.x, pend.y, weight=self.weight, eps=self.eps, out_dtype=stream.dtype, rows=rows,

@@ -1,7 +1,8 @@
 """Mixers that keep a matrix per head instead of keys and values, and mixers side by side.
 
 ``retention``    S_t = d_h S_(t-1) + k_t v_t^T,  o_t = S_t^T q_t  with a fixed decay d_h per head; rotated q
-                 and k; the read-out of each head divided by its root mean square and gated.
+                 and k, the read-out of each head divided by its root mean square and gated; or (lightning attention)
+                 q, k and v through silu, all heads of the read-out normed together, and a sigmoid gate.
 ``gated_delta``  S <- g_t S;  u = beta_t (v_t - S^T k_t);  S <- S + k_t u^T;  o_t = S^T q_t  with q, k, v passed
                  through a short causal convolution and silu, q and k brought to unit length, a decay g_t
                  per head or per head and key channel computed from the input, and a normed, gated read-out.
@@ -71,8 +72,11 @@ class _ProjectedMixer(Mixer, Projected):
 
 class Retention(_ProjectedMixer):
     """Parameters: ``hidden_size``, ``heads``, ``dim`` (of q and k), ``vdim``, ``decay`` (one number per head),
-    ``rotary`` ({"dims", "theta"} or None), ``eps`` (of the read-out's norm), ``out_scale``.
-    Keys are multiplied by dim^(-1/2) after the rotation; the gate is silu."""
+    ``rotary`` ({"dims", "theta"} or None), ``eps`` (of the read-out's norm), ``out_scale``, ``k_scale`` (a factor on the
+    keys after the rotation; default dim^(-1/2)), ``gate`` (``silu``, the default, or ``sigmoid``), ``activation`` (``silu``: q,
+    k and v = silu(W x), without rotation and factor; None, the default: as projected), ``norm`` (``head``, the default: every
+    head's read-out divided by its own root mean square; ``all``: all heads by that of the whole row, times a learned
+    vector, the tensor ``norm``)."""
 
     def __init__(self, spec: PartSpec, position: Optional[PositionEncoding] = None):
         super().__init__(spec, position or position_part(spec.params))
@@ -82,18 +86,31 @@ class Retention(_ProjectedMixer):
         self.decay_values = [float(x) for x in p["decay"]]
         if len(self.decay_values) != self.h:
             raise ValueError(f"retention: {len(self.decay_values)} decays for {self.h} heads")
+        self.k_scale = float(p["k_scale"]) if p.get("k_scale") is not None else self.d ** -0.5
+        self.act, self.norm_kind = p.get("activation"), str(p.get("norm", "head"))
+        gates = {"silu": rec_ops.GATE_SILU, "sigmoid": rec_ops.GATE_SIGMOID}
+        if p.get("gate", "silu") not in gates or self.act not in (None, "silu") or self.norm_kind not in ("head", "all"):
+            raise ValueError(f"retention: gate {p.get('gate')!r}, activation {self.act!r} or norm {self.norm_kind!r} is unknown")
+        self.gate_kind = gates[p.get("gate", "silu")]
+        if self.act is not None and (self.position is not None or p.get("k_scale") is not None):
+            raise ValueError("retention: activated queries and keys are neither rotated nor scaled")
         self.layout = rec_ops.StateLayout(self.h, self.d, self.vd)
         self.hidden_width = self.h * self.vd
         self.decay: Optional[torch.Tensor] = None
 
     def param_specs(self) -> Dict[str, ParamSpec]:
         hd, hv = self.h * self.d, self.h * self.vd
-        return {"q_proj": ParamSpec((hd, self.hidden)), "k_proj": ParamSpec((hd, self.hidden)),
-                "v_proj": ParamSpec((hv, self.hidden)), "g_proj": ParamSpec((hv, self.hidden)),
-                "o_proj": ParamSpec((self.hidden, hv))}
+        specs = {"q_proj": ParamSpec((hd, self.hidden)), "k_proj": ParamSpec((hd, self.hidden)),
+                 "v_proj": ParamSpec((hv, self.hidden)), "g_proj": ParamSpec((hv, self.hidden)),
+                 "o_proj": ParamSpec((self.hidden, hv))}
+        if self.norm_kind == "all":
+            specs["norm"] = ParamSpec((hv,), init="ones", keep_float32=True)
+        return specs
 
     def load(self, t: Dict[str, torch.Tensor]) -> None:
-        self.w_in = torch.cat([t["q_proj"], t["k_proj"], t["v_proj"], t["g_proj"]], dim=0).contiguous()
+        # the gate's columns of the product start on a 16-byte boundary
+        self.w_in, (_, self.gate_span) = stack_rows([torch.cat([t["q_proj"], t["k_proj"], t["v_proj"]], dim=0), t["g_proj"]])
+        self.norm_w = t["norm"].contiguous() if self.norm_kind == "all" else None
         self.w_out = t["o_proj"].contiguous()
         self.decay = torch.tensor(self.decay_values, dtype=torch.float64).to(torch.float32).to(self.w_out.device)
 
@@ -105,13 +122,26 @@ class Retention(_ProjectedMixer):
 
     def mix(self, z: torch.Tensor, ctx, cache: SlotStateCache, y: torch.Tensor) -> None:
         hd, hv = self.h * self.d, self.h * self.vd
-        freq = self.position.rotary_frequencies(self.position.head_dim, z.device) if self.position is not None else None
-        q, k, v = qkv_prepare(z, (0, hd, 2 * hd), self.h, self.h, self.d, self.vd, ctx.positions, ctx.req_of_token,
-                              out_dtype=torch.float32, inv_freq=freq, k_scale=self.d ** -0.5)
+        gate = z[:, self.gate_span[0]:self.gate_span[1]]
+        if self.act is not None:
+            x = activation(z[:, :2 * hd + hv], self.act, out_dtype=torch.float32)
+            q, k, v = x[:, :hd], x[:, hd:2 * hd], x[:, 2 * hd:]
+        else:
+            q, k, v = self._rotated(z, ctx)
         o = rec_ops.state_scan(q, k, v, cache.state, self.layout, ctx.q_start, ctx.slots, kv_heads=self.h, decay=self.decay,
                                max_q_len=ctx.host.max_q_len)
-        rec_ops.head_norm_gate(o, self.h, self.vd, self.eps, ctx.req_of_token, y, gate=z[:, 2 * hd + hv:2 * hd + 2 * hv],
-                               gate_kind=rec_ops.GATE_SILU, out_scale=self.out_scale)
+        if self.norm_kind == "all":
+            rec_ops.gate_norm(o, gate, 1, self.norm_w, self.eps, ctx.req_of_token, y, out_scale=self.out_scale,
+                              gate_kind=self.gate_kind, after=True)
+        else:
+            rec_ops.head_norm_gate(o, self.h, self.vd, self.eps, ctx.req_of_token, y, gate=gate, gate_kind=self.gate_kind,
+                                   out_scale=self.out_scale)
+
+    def _rotated(self, z: torch.Tensor, ctx):
+        hd = self.h * self.d
+        freq = self.position.rotary_frequencies(self.position.head_dim, z.device) if self.position is not None else None
+        return qkv_prepare(z, (0, hd, 2 * hd), self.h, self.h, self.d, self.vd, ctx.positions, ctx.req_of_token,
+                           out_dtype=torch.float32, inv_freq=freq, k_scale=self.k_scale)
 
 
 class GatedDelta(_ProjectedMixer):
