@@ -10,6 +10,7 @@ Llama-3-8B shape (random weights, bfloat16, page size 16), batch 8, 1,024-token 
     python bench.py --workload mixers --family pametar          # Pametar beside the Vepivik shape of equal size
     python bench.py --workload mixers --family sazavik          # Sazavik beside the Vepivik shape of equal size
     python bench.py --workload mixers --family ludelorn         # Ludelorn beside the Tirezen shape of equal size
+    python bench.py --workload mixers --family lagulorn         # Lagulorn beside the Pametar shape of equal size
 
 A "step" is one decode step of the whole batch.  ``value`` is decoded tokens per second
 with the K steps timed on the device (CUDA events) and the chosen tokens fed back on
@@ -46,7 +47,9 @@ width, expert count and latent sizes.  ``--family sazavik`` runs the Sazavik pre
 sinks, gates and a distance bias, norms on both sides of every sub-layer, dense and routed feed-forwards) beside the
 Vepivik presets of the same width, head and expert counts.  ``--family ludelorn`` runs the Ludelorn presets (windowed
 attention beside a selective state space, a window with pooled blocks, a window with a bias per distance and a sink)
-beside the Tirezen presets of the same width, heads and feed-forward.
+beside the Tirezen presets of the same width, heads and feed-forward.  ``--family lagulorn`` runs the Lagulorn presets (a
+stream in four copies, lightning attention, differential attention over a window, experts chosen by groups beside identity
+experts) beside the Pametar presets of the same width, copies, heads and experts.
 """
 
 from __future__ import annotations
@@ -292,7 +295,7 @@ def run_mixers(args) -> int:
 
     peaks, peak_source = load_peaks()
     family = args.family
-    other_family = {"pametar": "vepivik", "sazavik": "vepivik", "ludelorn": "tirezen"}.get(family)
+    other_family = {"pametar": "vepivik", "sazavik": "vepivik", "ludelorn": "tirezen", "lagulorn": "pametar"}.get(family)
     beside = {"1b": "Llama-3.2-1B", "3b": "Llama-3.2-3B"} if other_family is None else {s: f"{other_family}-{s}" for s in ("1b", "3b")}
     pairs = {size: (f"{family}-{size}", other) for size, other in beside.items()}
     steps = args.steps or 64
@@ -361,7 +364,7 @@ def main() -> int:
     ap.add_argument("--impl", default="ours", choices=["ours", "reference"])
     ap.add_argument("--workload", default="decode-8b", choices=["decode-8b", "mixed-1b", "serve-3b", "mixers"])
     ap.add_argument("--sizes", default="1b,3b", help="for --workload mixers: which pairs of models to run")
-    ap.add_argument("--family", default="tirezen", choices=["tirezen", "vepivik", "pametar", "sazavik", "ludelorn"],
+    ap.add_argument("--family", default="tirezen", choices=["tirezen", "vepivik", "pametar", "sazavik", "ludelorn", "lagulorn"],
                     help="for --workload mixers: the family whose presets run beside the Llama shapes")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--page-size", type=int, default=None, help="tokens per cache page (default: 16 as the benchmark "

@@ -442,6 +442,81 @@ PRESETS["ludelorn-1b"] = _ludelorn_stack(2048, 32000, 4, 16, 8, 128, 8192)
 PRESETS["ludelorn-3b"] = _ludelorn_stack(3072, 32000, 6, 24, 8, 128, 8192)
 
 
+# ---- Lagulorn ------------------------------------------------------------------------------------------------------
+
+def _lg_lightning(heads, dim, vdim, decay, mlp):
+    return {"type": "lightning", "mixer": {"heads": heads, "dim": dim, "vdim": vdim, "decay": list(decay)}, "mlp": mlp}
+
+
+def _lg_attention(heads, kv_heads, dim, vdim, scale, diff, window, mlp):
+    return {"type": "attention", "mlp": mlp,
+            "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": scale, "diff": diff, "mask": {"size": window}}}
+
+
+def _lg_dense(ff):
+    return {"kind": "dense", "ff": ff}
+
+
+def _lg_moe(experts, top, ff, limit, identity=0, groups=None):
+    router = {"experts": experts, "top": top, "identity": identity}
+    if groups is not None:
+        router["groups"] = {"count": groups[0], "keep": groups[1]}
+    return {"kind": "moe", "expert": {"ff": ff, "limit": limit}, "router": router}
+
+
+def _lagulorn(width, vocab, streams, layers, embedding_scale=1.0, residual_mult=1.0, eps=1e-5) -> Dict[str, Any]:
+    """``layers``: entries, or numbers of earlier layers whose tensors run again."""
+    full = []
+    for layer in layers:
+        full.append({**deepcopy(full[layer]), "weights_of": layer} if isinstance(layer, int) else layer)
+    cfg = {"architecture": "Lagulorn", "embedding": {"scale": embedding_scale}, "layers": full, "norm": {"eps": eps},
+           "residual_mult": residual_mult, "vocab": vocab, "width": width}
+    if streams is not None:
+        cfg["streams"] = streams
+    return cfg
+
+
+def _lagulorn_stack(width, vocab, groups, streams, heads, kv_heads, dim, state_heads, state_dim, experts, identity, top, ff) -> Dict[str, Any]:
+    """``groups`` times (lightning, differential attention) at the sizes of a real model, every layer with experts."""
+    decay = [1.0 - 2.0 ** (-1.0 - 9.0 * h / state_heads) for h in range(state_heads)]
+    layers = []
+    for _ in range(groups):
+        mlp = _lg_moe(experts, top, ff, 7.0, identity, (4, 2))
+        layers.append(_lg_lightning(state_heads, state_dim, state_dim, decay, mlp))
+        layers.append(_lg_attention(heads, kv_heads, dim, 2 * dim, dim ** -0.5, 0.35, 1024, mlp))
+    return _lagulorn(width, vocab, streams, layers, embedding_scale=width ** 0.5)
+
+
+# Test shapes.  A: layers that run another's tensors (one of each mixer), a layer without feed-forward, groups and identity
+# experts, value and key sizes apart.  B: sizes that are multiples of nothing, one copy of the stream, a window of one
+# position, no groups, no identity experts, an expert whose limit always binds.  C: the head sizes of the tensor-core
+# kernels, four copies, one group kept of several, windows around a page.  D: no copies (the plain residual sum), windows
+# that never bind, more heads to a key head than a decode tile holds, every output chosen, a chain of shared tensors.
+PRESETS["lagulorn-tiny-A"] = _lagulorn(64, 96, 2, [
+    _lg_lightning(2, 16, 12, (0.5, 0.98), _lg_dense(80)),
+    _lg_attention(4, 2, 12, 20, 0.3, 0.2, 9, _lg_moe(6, 3, 16, 0.8, 2, (4, 2))),
+    0, 1,
+    _lg_lightning(3, 8, 10, (0.9, 0.0, 1.0), None)], embedding_scale=2.5, residual_mult=0.7)
+PRESETS["lagulorn-tiny-B"] = _lagulorn(37, 50, 1, [
+    _lg_attention(3, 1, 5, 7, 0.4, -0.3, 4, _lg_moe(5, 3, 9, 0.2)),
+    _lg_lightning(5, 9, 3, (0.3, 0.7, 0.95, 0.99, 0.9), _lg_dense(18)),
+    _lg_attention(2, 2, 6, 11, 0.5, 0.6, 1, None)], embedding_scale=1.3, residual_mult=0.5, eps=1e-4)
+PRESETS["lagulorn-tiny-C"] = _lagulorn(128, 160, 4, [
+    _lg_attention(6, 2, 32, 48, 0.17, 0.5, 33, _lg_moe(14, 4, 40, 2.0, 2, (4, 1))),
+    _lg_lightning(3, 48, 40, (0.8, 0.97, 0.995), _lg_dense(192)),
+    _lg_attention(8, 1, 16, 32, 0.25, 0.1, 70, _lg_moe(9, 2, 64, 1.0, 3, (3, 2))),
+    0,
+    _lg_attention(2, 1, 64, 128, 0.125, 0.8, 16, _lg_dense(256))], embedding_scale=3.0, residual_mult=0.4)
+PRESETS["lagulorn-tiny-D"] = _lagulorn(48, 64, None, [
+    _lg_attention(20, 1, 16, 24, 0.25, 0.25, 4096, _lg_moe(3, 5, 20, 1.2, 2)),
+    _lg_lightning(2, 6, 30, (0.97, 0.6), _lg_moe(4, 1, 24, 0.5, 4, (8, 3))),
+    0, 2], embedding_scale=0.7, residual_mult=1.5)
+# Sizes that resemble a real model's layers (random weights, for the benchmark): the widths, head and expert counts, expert
+# sizes and copies of the stream of the Pametar benchmark models.
+PRESETS["lagulorn-1b"] = _lagulorn_stack(2048, 32000, 8, 4, 16, 8, 64, 16, 128, 16, 4, 2, 1280)
+PRESETS["lagulorn-3b"] = _lagulorn_stack(3072, 32000, 12, 4, 24, 8, 64, 24, 128, 32, 8, 4, 1024)
+
+
 def preset(name: str) -> Dict[str, Any]:
     """A fresh copy of the named configuration dictionary."""
     for key in (name, name.split("/")[-1], name.split("/")[-1].replace("Meta-", "")):
