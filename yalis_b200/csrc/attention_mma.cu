@@ -41,7 +41,7 @@
 // wholly before the window.  The blocks have pools and a block table of their own; their tiles
 // come first, then those of the window, in one softmax.
 //
-// The form of two maps (FORM 4) has two queries per head and two keys per key/value head and position (side by side in a
+// The form of two maps (FORM 4 and 5) has two queries per head and two keys per key/value head and position (side by side in a
 // cached row of 2 d sizes) over one value: each map is a softmax of its own, and the result is the first map's minus
 // lambda times the second's, divided by its root mean square, times a factor.  A row is then a (token, head, map): a
 // block takes half as many pairs (token, head) as it has rows, the first half of its rows for the first map and the second
@@ -82,8 +82,8 @@ struct AttnParams {
   const __nv_bfloat16* gate;   // GEN: [N, gate_stride] the result is multiplied by sigmoid(gate[t, head, :]) (null: not)
   int gate_stride;
   int gate_per_head;           // GEN: the gate is [N, nh], one number per head
-  int map_dim;                 // FORM 4: d, the size of one map's query and key (hs = 2 d, a multiple of 32)
-  float lambda, diff_eps;      // FORM 4
+  int map_dim;                 // FORM 4, 5: d, the size of one map's query and key (hs = 2 d, a multiple of 32)
+  float lambda, diff_eps;      // FORM 4, 5
   int hs, vs;                  // FORM 2, 3, 4: sizes of a key and a value (multiples of 8, at most HS)
   const float* rel;            // FORM 2, 3: [nh, rel_len], rel[h][min(p - key, rel_len - 1)] is added to the scaled score (null: not)
   int rel_len;
@@ -93,7 +93,7 @@ struct AttnParams {
   const int32_t* pool_table;
   int pool_table_width, pool_page_size, pool_num_pages, pool_page_shift;
   int n_splits;
-  float* part_o;               // [N, nh, n_splits, HS] (split mode); FORM 4: [N, nh, 2, n_splits, HS]
+  float* part_o;               // [N, nh, n_splits, HS] (split mode); FORM 4, 5: [N, nh, 2, n_splits, HS]
   float* part_ml;              // the same places, 2 floats each
   int32_t* tickets;            // one per block of a split: zero before the launch and zero again after it (split mode)
 };
@@ -263,10 +263,11 @@ __device__ __forceinline__ float finish_factor(const AttnParams& p, float m, flo
 }
 
 // FORM: 0 plain, 1 general, 2 extended, 3 extended with sizes known at launch (HS is then the padded size; p.hs and p.vs
-// are the real ones), 4 two maps (sizes known at launch too; p.hs is that of both maps' keys together).
+// are the real ones), 4 two maps (sizes known at launch too; p.hs is that of both maps' keys together), 5 two maps whose
+// keys together and values both have size HS.
 template <int HS, bool DEC, int FORM>
 __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const AttnParams p) {
-  constexpr bool GEN = FORM >= 1, EXT = FORM >= 2, SIZED = FORM >= 3, MAPS = FORM == 4;
+  constexpr bool GEN = FORM >= 1, EXT = FORM >= 2 && FORM <= 4, SIZED = FORM == 3 || FORM == 4, MAPS = FORM >= 4;
   const int hs = SIZED ? p.hs : HS, vs = SIZED ? p.vs : HS;
   constexpr int LD = HS + 8;            // padded row: ldmatrix rows fall into distinct banks
   constexpr int KSTEPS = HS / 16;       // k-steps of Q K^T
@@ -297,7 +298,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
   const int wrow = DEC ? 0 : warp * 16;           // first row of this warp within the block's tile
   const int wkey = DEC ? warp * WKEYS : 0;        // first key of this warp within a key tile
   const int wcol = HALF ? (wrow / PB) * p.map_dim : 0;         // first column of this warp's queries and keys
-  const int wcols = HALF ? p.map_dim : hs;
+  const int wcols = HALF ? p.map_dim : hs;        // (looked at where sizes are known at launch)
   const int32_t* bt = p.block_table + (size_t)req * p.table_width;
 
   // Positions of the tile's first and last token bound the keys this block needs.
@@ -827,7 +828,7 @@ __global__ void __launch_bounds__(NWARPS * 32) paged_attention_mma_kernel(const 
 template <int HS, bool DEC, int FORM>
 int launch_mode(const AttnParams& args, int n_requests, int max_rows, cudaStream_t stream) {
   constexpr int LD = HS + 8;
-  constexpr int RB = DEC ? 16 : BM, PB = FORM == 4 ? RB / 2 : RB, NST = DEC ? 3 : 2;
+  constexpr int RB = DEC ? 16 : BM, PB = FORM >= 4 ? RB / 2 : RB, NST = DEC ? 3 : 2;
   constexpr size_t tiles = (size_t)(RB + 2 * NST * BN) * LD * sizeof(__nv_bfloat16);
   // what a staged table of biases may take without costing a resident block
   constexpr int rel_room = FORM == 2 || FORM == 3 ? (DEC ? 1024 : 4096) : 0;
@@ -867,6 +868,9 @@ int launch_extended(const AttnParams& p, int n_requests, int max_rows, cudaStrea
 
 template <int HS>
 int launch_maps(const AttnParams& p, int n_requests, int max_pairs, cudaStream_t stream) {
+  if (p.hs == HS && p.vs == HS)
+    return max_pairs <= 16 ? launch_mode<HS, true, 5>(p, n_requests, max_pairs, stream)
+                           : launch_mode<HS, false, 5>(p, n_requests, max_pairs, stream);
   return max_pairs <= 16 ? launch_mode<HS, true, 4>(p, n_requests, max_pairs, stream)
                          : launch_mode<HS, false, 4>(p, n_requests, max_pairs, stream);
 }

@@ -313,6 +313,77 @@ __global__ void __launch_bounds__(256, 5) qkv_prepare_kernel(const PrepParams p)
   }
 }
 
+// The same where nothing turns and nothing is averaged: heads that are normed one by one or not at all, biases aside.  L
+// lanes take a head, NV times four values each (4 L NV covers the widest head), so heads of few sizes do not leave most of
+// a warp idle; the values stay in registers.  Groups of lanes are dealt to (token, head) pairs in order.
+template <typename T, typename TO, int L, int NV>
+__global__ void __launch_bounds__(256) qkv_plain_kernel(const PrepParams p, int n_tokens) {
+  pdl_launch_dependents();
+  pdl_wait();
+  const int keys = p.nk * p.maps, heads = p.nq + keys + p.nk;
+  const unsigned at = blockIdx.x * (256u / L) + threadIdx.x / L;
+  const int n = (int)(at / (unsigned)heads), head = (int)(at - (unsigned)n * heads), sl = threadIdx.x % L;
+  const int req = n < n_tokens ? p.req_of_token[n] : -1;
+  const bool is_q = head < p.nq, is_v = head >= p.nq + keys;
+  const int hh = is_q ? head : (is_v ? head - p.nq - keys : head - p.nq);
+  const int width = is_v ? p.vdim : p.dim;
+  TO* dst = nullptr;
+  if (req >= 0) {
+    if (is_q) {
+      dst = reinterpret_cast<TO*>(p.q_out) + (size_t)n * p.q_out_stride + (size_t)hh * width;
+    } else if (p.k_pool != nullptr) {
+      const long long row = paged_row(p.block_table + (size_t)req * p.table_width, p.table_width, p.page_size, p.num_pages, p.nk,
+                                      is_v ? hh : hh / p.maps, p.positions[n]);
+      if (row < 0) {
+        if (sl == 0 && p.bad_page) atomicOr(p.bad_page, YALIS_FLAG_BAD_PAGE);
+      } else {
+        dst = is_v ? reinterpret_cast<TO*>(p.v_pool) + row * width
+                   : reinterpret_cast<TO*>(p.k_pool) + row * (p.maps * width) + hh % p.maps * width;
+      }
+    } else if (p.k_out != nullptr) {
+      dst = is_v ? reinterpret_cast<TO*>(p.v_out) + (size_t)n * p.v_out_stride + (size_t)hh * width
+                 : reinterpret_cast<TO*>(p.k_out) + (size_t)n * p.k_out_stride + (size_t)hh * width;
+    }
+  }
+  const T* src = reinterpret_cast<const T*>(p.src) + (size_t)(req >= 0 ? n : 0) * p.src_stride +
+                 (is_q ? p.q_off : (is_v ? p.v_off : p.k_off)) + (size_t)hh * width;
+  float4 x[NV];
+  float ss = 0.f;
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = (sl + i * L) * 4;
+    x[i] = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (dst != nullptr && d < width) x[i] = load4_f32(src + d);
+    ss += (x[i].x * x[i].x + x[i].y * x[i].y) + (x[i].z * x[i].z + x[i].w * x[i].w);
+  }
+#pragma unroll
+  for (int o = L / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+  if (dst == nullptr) return;
+  const float* nw = is_v ? nullptr : (is_q ? p.q_norm : p.k_norm);
+  const float r = (is_v ? 1.0f : (is_q ? p.q_scale : p.k_scale)) * (nw ? 1.0f / sqrtf(ss / (float)width + p.norm_eps) : 1.0f);
+#pragma unroll
+  for (int i = 0; i < NV; ++i) {
+    const int d = (sl + i * L) * 4;
+    if (d >= width) continue;
+    float4 w = make_float4(1.f, 1.f, 1.f, 1.f);
+    if (nw) w = load4_f32(nw + d);
+    store4(dst + d, make_float4(x[i].x * r * w.x, x[i].y * r * w.y, x[i].z * r * w.z, x[i].w * r * w.w));
+  }
+}
+
+template <typename T, typename TO>
+int launch_qkv_plain(const PrepParams& p, int n_tokens, cudaStream_t stream) {
+  const int narrow = p.dim < p.vdim ? p.dim : p.vdim, widest = p.dim < p.vdim ? p.vdim : p.dim;
+  const long long pairs = (long long)n_tokens * (p.nq + (p.maps + 1) * p.nk);
+  if (pairs >= 1LL << 31) return YALIS_ERR_SHAPE;
+  auto go = [&](auto kernel, int lanes) {
+    return yalis_launch(kernel, dim3((unsigned)((pairs * lanes + 255) / 256)), dim3(256), 0, stream, p, n_tokens);
+  };
+  if (narrow <= 32 && widest <= 64) return go(qkv_plain_kernel<T, TO, 8, 2>, 8);
+  if (narrow <= 64 && widest <= 128) return go(qkv_plain_kernel<T, TO, 16, 2>, 16);
+  return go(qkv_plain_kernel<T, TO, 32, 2>, 32);
+}
+
 template <typename T, typename TO>
 int launch_qkv_prepare(const PrepParams& p, dim3 grid, int warps, bool table, bool vec, cudaStream_t stream) {
   const int row_floats = ((p.dim > p.vdim ? p.dim : p.vdim) + 3) & ~3;
@@ -523,6 +594,12 @@ YALIS_API int yalis_qkv_prepare(const void* src, int dtype, int src_stride, int 
   const bool vec = ((dim | vdim | rot_dims | src_stride | q_off | k_off | v_off | q_out_stride | k_out_stride | v_out_stride) & 3) == 0 &&
                    (ptrs & 15) == 0;
   int st;
+  const bool plain = vec && !inv_freq && !norm_all && q_temp_every <= 0 && pool == 0 && !q_bias && !k_bias && !v_bias &&
+                     dim <= 256 && vdim <= 256;
+  if (plain && dtype == YALIS_F32 && out_dtype == YALIS_F32) return launch_qkv_plain<float, float>(p, n_tokens, stream);
+  if (plain && dtype == YALIS_BF16 && out_dtype == YALIS_BF16)
+    return launch_qkv_plain<__nv_bfloat16, __nv_bfloat16>(p, n_tokens, stream);
+  if (plain && dtype == YALIS_BF16 && out_dtype == YALIS_F32) return launch_qkv_plain<__nv_bfloat16, float>(p, n_tokens, stream);
   if (dtype == YALIS_F32 && out_dtype == YALIS_F32) st = launch_qkv_prepare<float, float>(p, grid, warps, table, vec, stream);
   else if (dtype == YALIS_BF16 && out_dtype == YALIS_BF16)
     st = launch_qkv_prepare<__nv_bfloat16, __nv_bfloat16>(p, grid, warps, table, vec, stream);
