@@ -278,7 +278,7 @@ __device__ __forceinline__ void load4(const __nv_bfloat16* p, float& a, float& b
 // the experts, and a row of the router read once serves all TOK tokens (each token's sum has the same order whatever
 // TOK is); then warp t chooses for token t.
 template <typename T, int TOK, bool RULES>
-__global__ void route_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ w, int E, int K, int top,
+__global__ void __launch_bounds__(512) route_kernel(const T* __restrict__ x, long x_stride, const float* __restrict__ w, int E, int K, int top,
                              float eps, float factor, const int32_t* __restrict__ req_of_token, int32_t* __restrict__ ids,
                              float* __restrict__ weights, int n_tokens, int sigmoid, const float* __restrict__ side,
                              float* __restrict__ side_out, const ChoiceRules rules) {
@@ -316,7 +316,7 @@ __global__ void route_kernel(const T* __restrict__ x, long x_stride, const float
 #pragma unroll
     for (int t = 0; t < TOK; ++t) acc[t] = 0.f;
     if (vec) {
-#pragma unroll 2
+#pragma unroll (TOK == 1 ? 8 : 2)
       for (int k = 4 * lane; k < K; k += 128) {
         const float4 wv = *reinterpret_cast<const float4*>(wr + k);
 #pragma unroll
@@ -384,7 +384,9 @@ int launch_route(const void* x, long x_stride, const float* w, int n_tokens, int
       return YALIS_ERR_LAUNCH;
     configured = smem;
   }
-  return yalis_launch(route_kernel<T, TOK, RULES>, dim3((n_tokens + TOK - 1) / TOK), dim3(256), smem, stream, (const T*)x, x_stride, w, E, K,
+  // one token a block: blocks are few, so sixteen warps share out the experts
+  const int threads = TOK == 1 && n_tokens <= 2 * yalis_sm_count() ? 512 : 256;
+  return yalis_launch(route_kernel<T, TOK, RULES>, dim3((n_tokens + TOK - 1) / TOK), dim3(threads), smem, stream, (const T*)x, x_stride, w, E, K,
                       top, eps, factor, req_of_token, ids, weights, n_tokens, sigmoid, side, side_out, rules);
 }
 
